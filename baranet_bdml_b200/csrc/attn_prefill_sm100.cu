@@ -54,17 +54,8 @@ struct PrefillWsLayout {
 
 static PrefillWsLayout prefill_layout(int B, int S, int Hkv) {
     PrefillWsLayout L;
-    auto up = [](size_t x) { return (x + 255) / 256 * 256; };
-    L.table = 256;                                               // after the header (error word)
-    L.kmax2 = L.table + up((size_t)S * (PF_D / 2) * sizeof(float2));   // [B][Hkv][key tiles of 128] largest |k|^2
-    L.krot = L.kmax2 + up((size_t)B * Hkv * ((S + PF_BN - 1) / PF_BN) * sizeof(float));
-    L.total = L.krot + up((size_t)B * S * Hkv * PF_D * sizeof(__nv_bfloat16));
+    prefill_bf16_workspace_layout(B, S, Hkv, &L.table, &L.kmax2, &L.krot, &L.total);
     return L;
-}
-
-void prefill_bf16_workspace_layout(int B, int S, int Hkv, size_t* table, size_t* kmax2, size_t* krot, size_t* total) {
-    const PrefillWsLayout L = prefill_layout(B, S, Hkv);
-    *table = L.table; *kmax2 = L.kmax2; *krot = L.krot; *total = L.total;
 }
 
 // the cos/sin table alone (for a caller that produces the rotated K itself): [S][32] of position s + position_offset

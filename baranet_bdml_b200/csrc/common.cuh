@@ -49,7 +49,13 @@ inline void launch_dependent(void (*kernel)(P...), unsigned grid, unsigned block
 
 // Byte offsets inside the scratch buffer of bn_attn_prefill_bf16 (cos/sin table, per-tile key norms, rotated K) and
 // its size: the fused q/k/v projection writes the last two itself.
-void prefill_bf16_workspace_layout(int B, int S, int Hkv, size_t* table, size_t* kmax2, size_t* krot, size_t* total);
+inline void prefill_bf16_workspace_layout(int B, int S, int Hkv, size_t* table, size_t* kmax2, size_t* krot, size_t* total) {
+    auto up = [](size_t x) { return (x + 255) / 256 * 256; };
+    *table = 256;                                                        // after the header (error word)
+    *kmax2 = *table + up((size_t)S * 32 * sizeof(float2));               // [B][Hkv][key tiles of 128] largest |k|^2
+    *krot = *kmax2 + up((size_t)B * Hkv * ((S + 127) / 128) * sizeof(float));
+    *total = *krot + up((size_t)B * S * Hkv * 64 * sizeof(__nv_bfloat16));
+}
 
 // The RoPE frequency of pair i, with the reference's exact arithmetic
 // (src/ops/op_rope.cuh:82): fp32 exponent, fp32 pow, reciprocal taken in

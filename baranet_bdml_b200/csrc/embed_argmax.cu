@@ -10,8 +10,41 @@
 //       it is element 0.  The reference runs ONE THREAD per row; here a CTA per row.
 // Both are HBM-bound copies / reductions: 16-byte accesses, consecutive threads on consecutive addresses.
 #include "common.cuh"
+#include "hybrid.cuh"
 
 namespace bn {
+
+// A bf16 table: rows to fp32 (a residual stream), to bf16 (an operand of a product), or to both
+__global__ void __launch_bounds__(256)
+embedding_gather_bf16_kernel(const __nv_bfloat16* __restrict__ table, int64_t table_rs, const uint32_t* __restrict__ ids,
+                             float* __restrict__ out32, int64_t rs32, __nv_bfloat16* __restrict__ out16, int64_t rs16,
+                             int n_ids, int hidden, int vocab, int* __restrict__ error_word) {
+    const bool vec = (hidden | table_rs | rs32 | rs16) % 4 == 0 &&
+                     ((reinterpret_cast<uintptr_t>(table) | reinterpret_cast<uintptr_t>(out32) | reinterpret_cast<uintptr_t>(out16)) & 15) == 0;
+    for (int i = blockIdx.x; i < n_ids; i += gridDim.x) {
+        const uint32_t id = ids[i];
+        const bool valid = id < (uint32_t)vocab;
+        if (!valid && threadIdx.x == 0 && error_word) atomicExch(error_word, BN_ERR_INVALID_ARG);
+        const __nv_bfloat16* src = table + (int64_t)(valid ? id : 0) * table_rs;
+        const float keep = valid ? 1.f : 0.f;
+        if (vec) {
+            for (int c = threadIdx.x * 4; c < hidden; c += blockDim.x * 4) {
+                float v[4];
+                load4(src + c, v);
+#pragma unroll
+                for (int e = 0; e < 4; ++e) v[e] *= keep;
+                if (out32) store4(out32 + i * rs32 + c, v);
+                if (out16) store4(out16 + i * rs16 + c, v);
+            }
+        } else {
+            for (int c = threadIdx.x; c < hidden; c += blockDim.x) {
+                const float v = to_f(src[c]) * keep;
+                if (out32) out32[i * rs32 + c] = v;
+                if (out16) out16[i * rs16 + c] = from_f<__nv_bfloat16>(v);
+            }
+        }
+    }
+}
 
 __global__ void __launch_bounds__(256)
 embedding_gather_kernel(const float* __restrict__ table, int64_t table_rs, const uint32_t* __restrict__ ids,
@@ -106,6 +139,24 @@ extern "C" int bn_embedding_gather_f32(const float* table, int64_t table_rs, con
     embedding_gather_kernel<<<(unsigned)(n_ids < cap ? n_ids : cap), 256, 0, as_stream(stream)>>>(
         table, table_rs, ids, out, out_rs, n_ids, hidden, vocab, error_word);
     return launch_status("bn_embedding_gather_f32");
+}
+
+extern "C" int bn_embedding_gather_bf16(const void* table, int64_t table_rs, const uint32_t* ids, float* out_f32, int64_t rs_f32,
+                                        void* out_bf16, int64_t rs_bf16, int n_ids, int hidden, int vocab, int* error_word,
+                                        bn_stream_t stream) {
+    const char* what = "bn_embedding_gather_bf16";
+    if (!table || !ids || (!out_f32 && !out_bf16)) return fail(BN_ERR_INVALID_ARG, "%s: null pointer", what);
+    if (n_ids < 0 || hidden < 0 || vocab <= 0) return fail(BN_ERR_INVALID_ARG, "%s: bad shape n_ids=%d hidden=%d vocab=%d", what, n_ids, hidden, vocab);
+    if (int rc = require_sm100()) return rc;
+    if (n_ids == 0 || hidden == 0) return BN_OK;
+    int dev = 0, sms = 0;
+    cudaGetDevice(&dev);
+    cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
+    const long long cap = (long long)sms * 8;
+    embedding_gather_bf16_kernel<<<(unsigned)(n_ids < cap ? n_ids : cap), 256, 0, as_stream(stream)>>>(
+        static_cast<const __nv_bfloat16*>(table), table_rs, ids, out_f32, rs_f32, static_cast<__nv_bfloat16*>(out_bf16), rs_bf16,
+        n_ids, hidden, vocab, error_word);
+    return launch_status(what);
 }
 
 extern "C" int bn_argmax_rows_f32(const float* x, int64_t x_rs, int64_t x_cs, uint32_t* out, int rows, int cols,

@@ -12,12 +12,15 @@
 // Output tile 128 x 256; the fp32 accumulator (256 TMEM columns) is double buffered, so the epilogue of one tile
 // runs under the main loop of the next.  Tiles are walked N-panel by N-panel with M fastest, so the CTAs that run
 // together share their Bt panel in L2.  Edges: TMA zero-fills loads beyond M, N, K; stores are bounds-checked.
-// Epilogue variants: plain (C = the accumulator as bf16) and SwiGLU (`MLP.__call__`, mygrad/llama/llama_layers.py:217-232,
-// SiLU as op_silu.cuh:7-15): Bt holds, per 256-row tile, 128 rows of the gate weight followed by the 128 rows of the up
-// weight for the same intermediate indices, so one thread finds gate and up of an output element in the same
-// accumulator row and writes silu(gate) * up -- the two GEMMs, the activation and the product in one launch.
+// Epilogue variants: plain (C = the accumulator as bf16), fp32 (the accumulator itself), the accumulator's activation
+// times a matrix given by the caller, and the gated linear unit (SwiGLU in `MLP.__call__`,
+// mygrad/llama/llama_layers.py:217-232, SiLU as op_silu.cuh:7-15; GELU for other models): Bt holds, per 256-row tile, 128
+// rows of the gate weight followed by the 128 rows of the up weight for the same intermediate indices, so one thread finds
+// gate and up of an output element in the same accumulator row and writes act(gate) * up -- the two GEMMs, the activation
+// and the product in one launch.
 // Every mbarrier wait is bounded; on expiry the kernel raises the caller's error word, frees TMEM and returns.
 #include "common.cuh"
+#include "hybrid.cuh"
 #include "ptx.cuh"
 #include "tcgen05.cuh"
 #include "tma.cuh"
@@ -53,16 +56,21 @@ struct QkvEpilogue {
     int max_pages, S, NQ, NK, Hkv, n_ktiles, position_offset;
 };
 
-constexpr int EPI_PLAIN = 0, EPI_SWIGLU = 1, EPI_PARTIAL = 2, EPI_QKV = 3;
+// EPI_GLU + activation: one instantiation per activation keeps the choice out of the epilogue's loop
+constexpr int EPI_PLAIN = 0, EPI_PARTIAL = 2, EPI_QKV = 3, EPI_F32 = 4, EPI_ACTMUL = 5, EPI_GLU = 16;
+constexpr int EPI_GLU_SILU = EPI_GLU + BN_ACT_SILU, EPI_GLU_GELU = EPI_GLU + BN_ACT_GELU_TANH;
 
 struct GemmParams {
     __nv_bfloat16* c;
     int* error_word;       // optional
     int M, N, K;           // N = rows of Bt
-    int n_out;             // columns of C: N (plain) or the intermediate size (SwiGLU)
+    int n_out;             // columns of C: N (plain) or the intermediate size (GLU)
     float* partial;        // EPI_PARTIAL: [split][M][N] fp32
     int splits, k_per_split;   // EPI_PARTIAL: K steps are cut into `splits` ranges of k_per_split steps
     QkvEpilogue qkv;       // EPI_QKV
+    const __nv_bfloat16* mul;  // EPI_ACTMUL: (M, mul_ld), C = act(accumulator) * mul
+    long long mul_ld;
+    int act;
 };
 
 
@@ -300,8 +308,35 @@ gemm_bf16_nt_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
                         }
                     }
                 }
-            } else if (EPI == EPI_PARTIAL) {
-                // the fp32 partial sum of this K range; the ranges are added in order by the reduce kernel
+            } else if (EPI == EPI_ACTMUL) {
+                __nv_bfloat16* crow = p.c + (size_t)gm * p.n_out + n0;
+                const __nv_bfloat16* mrow = p.mul + (size_t)gm * p.mul_ld + n0;
+#pragma unroll 1
+                for (int c = 0; c < GM_BN / 32; ++c) {
+                    uint32_t r[32];
+                    tc::ld32(tmem + lane_base + acc * GM_BN + c * 32, r);
+                    tc::wait_ld(r);
+                    if (gm < p.M) {
+#pragma unroll
+                        for (int v = 0; v < 4; ++v) {
+                            const int col = n0 + c * 32 + v * 8;
+                            if (col < p.n_out) {
+                                const uint4 m4 = *reinterpret_cast<const uint4*>(mrow + c * 32 + v * 8);
+                                const uint32_t* mw = reinterpret_cast<const uint32_t*>(&m4);
+                                uint4 o4;
+                                uint32_t* ow = reinterpret_cast<uint32_t*>(&o4);
+#pragma unroll
+                                for (int e = 0; e < 4; ++e)
+                                    ow[e] = pack_bf16(activation_fast(p.act, __uint_as_float(r[v * 8 + 2 * e])) * bf16_lo(mw[e]),
+                                                      activation_fast(p.act, __uint_as_float(r[v * 8 + 2 * e + 1])) * bf16_hi(mw[e]));
+                                *reinterpret_cast<uint4*>(crow + c * 32 + v * 8) = o4;
+                            }
+                        }
+                    }
+                }
+            } else if (EPI == EPI_PARTIAL || EPI == EPI_F32) {
+                // the accumulator in fp32: the result itself (EPI_F32), or the partial sum of this K range; the ranges
+                // are added in order by the reduce kernel
                 float* prow = p.partial + ((size_t)(t / (tiles_m * tiles_n)) * p.M + gm) * p.N + n0;
 #pragma unroll 1
                 for (int c = 0; c < GM_BN / 32; ++c) {
@@ -339,8 +374,7 @@ gemm_bf16_nt_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
 #pragma unroll
                                 for (int e = 0; e < 8; ++e) {
                                     const float gv = __uint_as_float(g[v * 8 + e]);
-                                    // silu(g) * up, silu(g) = g / (1 + exp(-g))
-                                    h[e] = __fdividef(gv, 1.f + __expf(-gv)) * __uint_as_float(u[v * 8 + e]);
+                                    h[e] = activation_fast(EPI - EPI_GLU, gv) * __uint_as_float(u[v * 8 + e]);
                                 }
                                 uint4 o4;
                                 o4.x = pack_bf16(h[0], h[1]);
@@ -374,9 +408,11 @@ gemm_bf16_nt_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
 
 using namespace bn;
 
-// sum of the split-K partials, in split order (deterministic), rounded once to bf16
+// sum of the split-K partials, in split order (deterministic), rounded once to bf16, or kept in fp32 (c32), or its
+// activation times `mul`
 __global__ void __launch_bounds__(256)
-gemm_splitk_reduce_kernel(const float* __restrict__ partial, __nv_bfloat16* __restrict__ c, long long mn4, int splits) {
+gemm_splitk_reduce_kernel(const float* __restrict__ partial, __nv_bfloat16* __restrict__ c, long long mn4, int splits,
+                          float* __restrict__ c32, const __nv_bfloat16* __restrict__ mul, long long mul_ld, int N, int act) {
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;     // one group of 4 outputs
     if (i >= mn4) return;
     const float4* p4 = reinterpret_cast<const float4*>(partial);
@@ -384,6 +420,18 @@ gemm_splitk_reduce_kernel(const float* __restrict__ partial, __nv_bfloat16* __re
     for (int s = 1; s < splits; ++s) {
         const float4 v = __ldcg(p4 + (long long)s * mn4 + i);
         acc.x += v.x; acc.y += v.y; acc.z += v.z; acc.w += v.w;
+    }
+    if (c32) {
+        reinterpret_cast<float4*>(c32)[i] = acc;
+        return;
+    }
+    if (mul) {
+        const long long row = i * 4 / N, col = i * 4 - row * N;
+        const uint2 m = *reinterpret_cast<const uint2*>(mul + row * mul_ld + col);
+        acc.x = activation_fast(act, acc.x) * bf16_lo(m.x);
+        acc.y = activation_fast(act, acc.y) * bf16_hi(m.x);
+        acc.z = activation_fast(act, acc.z) * bf16_lo(m.y);
+        acc.w = activation_fast(act, acc.w) * bf16_hi(m.y);
     }
     reinterpret_cast<uint2*>(c)[i] = make_uint2(pack_bf16(acc.x, acc.y), pack_bf16(acc.z, acc.w));
 }
@@ -414,17 +462,23 @@ static int gemm_configure(int dev) {
 
 static int gemm_launch(const void* a, const void* bt, void* c, int M, int N, int K, int n_out, int epi, int* error_word,
                        bn_stream_t stream, const char* what, float* partial = nullptr, int splits = 1,
-                       int k_per_split = 0, const QkvEpilogue* qkv = nullptr) {
-    if (!a || !bt || !c) return fail(BN_ERR_INVALID_ARG, "%s: null pointer", what);
+                       int k_per_split = 0, const QkvEpilogue* qkv = nullptr, float* c32 = nullptr,
+                       const void* mul = nullptr, long long mul_ld = 0, int act = BN_ACT_NONE) {
+    if (!a || !bt || (!c && !c32)) return fail(BN_ERR_INVALID_ARG, "%s: null pointer", what);
     if (M < 0 || N < 0 || K < 0 || n_out < 0) return fail(BN_ERR_INVALID_ARG, "%s: bad shape M=%d N=%d K=%d", what, M, N, K);
     if (n_out % 8 || K % 8)
         return fail(BN_ERR_UNSUPPORTED, "%s: N=%d and K=%d must be multiples of 8 (16-byte rows)", what, n_out, K);
-    if ((reinterpret_cast<uintptr_t>(a) | reinterpret_cast<uintptr_t>(bt) | reinterpret_cast<uintptr_t>(c)) & 15)
+    if ((reinterpret_cast<uintptr_t>(a) | reinterpret_cast<uintptr_t>(bt) | reinterpret_cast<uintptr_t>(c) |
+         reinterpret_cast<uintptr_t>(c32) | reinterpret_cast<uintptr_t>(mul)) & 15)
         return fail(BN_ERR_INVALID_ARG, "%s: a/bt/c must be 16-byte aligned", what);
+    if (mul && (mul_ld < n_out || mul_ld % 8))
+        return fail(BN_ERR_INVALID_ARG, "%s: row stride %lld of the factor (a multiple of 8, at least %d)", what, mul_ld, n_out);
+    if (act < 0 || act > BN_ACT_LAST) return fail(BN_ERR_INVALID_ARG, "%s: activation %d", what, act);
     if (int rc = require_sm100()) return rc;
     if (M == 0 || n_out == 0) return BN_OK;
     if (K == 0) {
-        cudaError_t e = cudaMemsetAsync(c, 0, (size_t)M * n_out * 2, as_stream(stream));
+        cudaError_t e = c32 ? cudaMemsetAsync(c32, 0, (size_t)M * n_out * 4, as_stream(stream))
+                            : cudaMemsetAsync(c, 0, (size_t)M * n_out * 2, as_stream(stream));
         return e == cudaSuccess ? BN_OK : fail(BN_ERR_CUDA, "%s: %s", what, cudaGetErrorString(e));
     }
     const int bn = epi == EPI_PARTIAL ? 64 : 256;
@@ -447,16 +501,27 @@ static int gemm_launch(const void* a, const void* bt, void* c, int M, int N, int
     cudaGetDevice(&dev);
     cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
     const long long n_items = (long long)((M + GM_BM - 1) / GM_BM) * ((N + bn - 1) / bn) * splits;
-    GemmParams p{static_cast<__nv_bfloat16*>(c), error_word, M, N, K, n_out, partial, splits, k_per_split, QkvEpilogue{}};
+    GemmParams p{static_cast<__nv_bfloat16*>(c), error_word, M, N, K, n_out, partial, splits, k_per_split, QkvEpilogue{},
+                 static_cast<const __nv_bfloat16*>(mul), mul_ld, act};
+    if (epi == EPI_F32) p.partial = c32;
     if (qkv) p.qkv = *qkv;
     const unsigned grid = (unsigned)(n_items < sms ? n_items : sms);
     cudaStream_t st = as_stream(stream);
     if (epi == EPI_PLAIN) {
         if (int rc = gemm_configure<EPI_PLAIN, 256>(dev)) return rc;
         gemm_bf16_nt_kernel<EPI_PLAIN, 256><<<grid, GM_THREADS, GemmShape<256>::SMEM_BYTES, st>>>(tmap_a, tmap_b, p);
-    } else if (epi == EPI_SWIGLU) {
-        if (int rc = gemm_configure<EPI_SWIGLU, 256>(dev)) return rc;
-        gemm_bf16_nt_kernel<EPI_SWIGLU, 256><<<grid, GM_THREADS, GemmShape<256>::SMEM_BYTES, st>>>(tmap_a, tmap_b, p);
+    } else if (epi == EPI_GLU_SILU) {
+        if (int rc = gemm_configure<EPI_GLU_SILU, 256>(dev)) return rc;
+        gemm_bf16_nt_kernel<EPI_GLU_SILU, 256><<<grid, GM_THREADS, GemmShape<256>::SMEM_BYTES, st>>>(tmap_a, tmap_b, p);
+    } else if (epi == EPI_GLU_GELU) {
+        if (int rc = gemm_configure<EPI_GLU_GELU, 256>(dev)) return rc;
+        gemm_bf16_nt_kernel<EPI_GLU_GELU, 256><<<grid, GM_THREADS, GemmShape<256>::SMEM_BYTES, st>>>(tmap_a, tmap_b, p);
+    } else if (epi == EPI_F32) {
+        if (int rc = gemm_configure<EPI_F32, 256>(dev)) return rc;
+        gemm_bf16_nt_kernel<EPI_F32, 256><<<grid, GM_THREADS, GemmShape<256>::SMEM_BYTES, st>>>(tmap_a, tmap_b, p);
+    } else if (epi == EPI_ACTMUL) {
+        if (int rc = gemm_configure<EPI_ACTMUL, 256>(dev)) return rc;
+        gemm_bf16_nt_kernel<EPI_ACTMUL, 256><<<grid, GM_THREADS, GemmShape<256>::SMEM_BYTES, st>>>(tmap_a, tmap_b, p);
     } else if (epi == EPI_QKV) {
         if (int rc = gemm_configure<EPI_QKV, 256>(dev)) return rc;
         gemm_bf16_nt_kernel<EPI_QKV, 256><<<grid, GM_THREADS, GemmShape<256>::SMEM_BYTES, st>>>(tmap_a, tmap_b, p);
@@ -466,7 +531,7 @@ static int gemm_launch(const void* a, const void* bt, void* c, int M, int N, int
         if (int rc = launch_status(what)) return rc;
         const long long mn4 = (long long)M * N / 4;
         gemm_splitk_reduce_kernel<<<(unsigned)((mn4 + 255) / 256), 256, 0, st>>>(partial, static_cast<__nv_bfloat16*>(c),
-                                                                             mn4, splits);
+                                                                             mn4, splits, c32, p.mul, mul_ld, N, act);
     }
     return launch_status(what);
 }
@@ -480,7 +545,27 @@ extern "C" int bn_gemm_swiglu_bf16_nt(const void* x, const void* gate_up_t, void
                                       int* error_word, bn_stream_t stream) {
     if (inter < 0) return fail(BN_ERR_INVALID_ARG, "bn_gemm_swiglu_bf16_nt: bad shape inter=%d", inter);
     const int n_rows = (inter + 127) / 128 * 256;      // rows of the packed gate/up weight
-    return gemm_launch(x, gate_up_t, h, M, n_rows, K, inter, EPI_SWIGLU, error_word, stream, "bn_gemm_swiglu_bf16_nt");
+    return gemm_launch(x, gate_up_t, h, M, n_rows, K, inter, EPI_GLU_SILU, error_word, stream, "bn_gemm_swiglu_bf16_nt");
+}
+
+extern "C" int bn_gemm_glu_bf16_nt(const void* x, const void* gate_up_t, void* h, int M, int inter, int K, int act,
+                                   int* error_word, bn_stream_t stream) {
+    const char* what = "bn_gemm_glu_bf16_nt";
+    if (inter < 0) return fail(BN_ERR_INVALID_ARG, "%s: bad shape inter=%d", what, inter);
+    if (act != BN_ACT_SILU && act != BN_ACT_GELU_TANH) return fail(BN_ERR_UNSUPPORTED, "%s: activation %d", what, act);
+    return gemm_launch(x, gate_up_t, h, M, (inter + 127) / 128 * 256, K, inter, EPI_GLU + act, error_word, stream, what);
+}
+
+extern "C" int bn_gemm_bf16_nt_f32(const void* a, const void* bt, float* c, int M, int N, int K, int* error_word,
+                                   bn_stream_t stream) {
+    return gemm_launch(a, bt, nullptr, M, N, K, N, EPI_F32, error_word, stream, "bn_gemm_bf16_nt_f32", nullptr, 1, 0, nullptr, c);
+}
+
+extern "C" int bn_gemm_act_mul_bf16_nt(const void* a, const void* bt, const void* mul, int64_t mul_ld, void* c, int M, int N,
+                                       int K, int act, int* error_word, bn_stream_t stream) {
+    if (!mul) return fail(BN_ERR_INVALID_ARG, "bn_gemm_act_mul_bf16_nt: null pointer");
+    return gemm_launch(a, bt, c, M, N, K, N, EPI_ACTMUL, error_word, stream, "bn_gemm_act_mul_bf16_nt", nullptr, 1, 0, nullptr,
+                       nullptr, mul, mul_ld, act);
 }
 
 extern "C" size_t bn_gemm_bf16_nt_small_m_workspace_bytes(int M, int N, int K) {
@@ -493,21 +578,42 @@ extern "C" size_t bn_gemm_bf16_nt_small_m_workspace_bytes(int M, int N, int K) {
     return (size_t)splits * M * N * sizeof(float);
 }
 
-extern "C" int bn_gemm_bf16_nt_small_m(const void* a, const void* bt, void* c, int M, int N, int K, void* workspace,
-                                       size_t workspace_bytes, int* error_word, bn_stream_t stream) {
+static int small_m_launch(const void* a, const void* bt, void* c, float* c32, const void* mul, int64_t mul_ld, int act, int M,
+                          int N, int K, void* workspace, size_t workspace_bytes, int* error_word, bn_stream_t stream,
+                          const char* what) {
+    int splits = 1, per = 0;
     if (M > 0 && N > 0 && K > 0) {
         if (!workspace || (reinterpret_cast<uintptr_t>(workspace) & 15))
-            return fail(BN_ERR_WORKSPACE, "bn_gemm_bf16_nt_small_m: workspace missing or not 16-byte aligned");
-        int dev = 0, sms = 0, splits = 1, per = 0;
+            return fail(BN_ERR_WORKSPACE, "%s: workspace missing or not 16-byte aligned", what);
+        int dev = 0, sms = 0;
         cudaGetDevice(&dev);
         cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
         splitk_plan(M, N, K, sms, &splits, &per);
         if (workspace_bytes < (size_t)splits * M * N * sizeof(float))
-            return fail(BN_ERR_WORKSPACE, "bn_gemm_bf16_nt_small_m: workspace of %zu bytes is too small", workspace_bytes);
-        return gemm_launch(a, bt, c, M, N, K, N, EPI_PARTIAL, error_word, stream, "bn_gemm_bf16_nt_small_m",
-                           static_cast<float*>(workspace), splits, per);
+            return fail(BN_ERR_WORKSPACE, "%s: workspace of %zu bytes is too small", what, workspace_bytes);
     }
-    return gemm_launch(a, bt, c, M, N, K, N, EPI_PARTIAL, error_word, stream, "bn_gemm_bf16_nt_small_m");
+    return gemm_launch(a, bt, c, M, N, K, N, EPI_PARTIAL, error_word, stream, what, static_cast<float*>(workspace), splits, per,
+                       nullptr, c32, mul, mul_ld, act);
+}
+
+extern "C" int bn_gemm_bf16_nt_small_m(const void* a, const void* bt, void* c, int M, int N, int K, void* workspace,
+                                       size_t workspace_bytes, int* error_word, bn_stream_t stream) {
+    return small_m_launch(a, bt, c, nullptr, nullptr, 0, BN_ACT_NONE, M, N, K, workspace, workspace_bytes, error_word, stream,
+                          "bn_gemm_bf16_nt_small_m");
+}
+
+extern "C" int bn_gemm_bf16_nt_small_m_f32(const void* a, const void* bt, float* c, int M, int N, int K, void* workspace,
+                                           size_t workspace_bytes, int* error_word, bn_stream_t stream) {
+    return small_m_launch(a, bt, nullptr, c, nullptr, 0, BN_ACT_NONE, M, N, K, workspace, workspace_bytes, error_word, stream,
+                          "bn_gemm_bf16_nt_small_m_f32");
+}
+
+extern "C" int bn_gemm_act_mul_bf16_nt_small_m(const void* a, const void* bt, const void* mul, int64_t mul_ld, void* c, int M,
+                                               int N, int K, int act, void* workspace, size_t workspace_bytes,
+                                               int* error_word, bn_stream_t stream) {
+    if (!mul) return fail(BN_ERR_INVALID_ARG, "bn_gemm_act_mul_bf16_nt_small_m: null pointer");
+    return small_m_launch(a, bt, c, nullptr, mul, mul_ld, act, M, N, K, workspace, workspace_bytes, error_word, stream,
+                          "bn_gemm_act_mul_bf16_nt_small_m");
 }
 
 extern "C" int bn_gemm_qkv_rope_bf16(const void* x, const void* wqkv_t, void* q_out, void* v_out, int B, int S, int hidden,

@@ -15,10 +15,12 @@
 //   The 8 warps' partial sums (16 x 8 fp32) are added through shared memory in warp order (deterministic).
 // Variants: up to three column ranges of one concatenated weight written to separate outputs (q, k, v of the layer in one
 // launch); the same with the K and V ranges rotated / appended to the paged cache by the epilogue instead (what
-// bn_kv_append would do with them, mygrad/llama/llama_layers.py:161-171 for the new token); and the SwiGLU pair (two weights, h = silu(x Wg) * (x Wu), op_silu.cuh:7-15).
-// K must be a multiple of 256 (a warp's eighth is a whole number of 32-wide steps) and at most 8192; N a multiple
-// of 8.  Anything else belongs to bn_gemm_bf16_nt_small_m.
+// bn_kv_append would do with them, mygrad/llama/llama_layers.py:161-171 for the new token); and the gated pair (two weights, h = act(x Wg) * (x Wu); SwiGLU: op_silu.cuh:7-15);
+// an fp32 output; and the result's activation times a matrix given by the caller.
+// K is a multiple of 8 and at most 8192, N a multiple of 8.  When K is a multiple of 256 a warp's eighth is a whole number
+// of 32-wide steps; otherwise (RAGGED) the eighths are rounded up and pieces beyond K read as zero.  Anything else belongs to bn_gemm_bf16_nt_small_m.
 #include "common.cuh"
+#include "hybrid.cuh"
 #include "ptx.cuh"
 
 namespace bn {
@@ -35,7 +37,11 @@ struct SkinnyParams {
     __nv_bfloat16* out[3];              // outputs of the column ranges
     int n_end[3];                       // range r covers columns [n_end[r-1], n_end[r])
     int ld[3];                          // row stride of out[r] in elements
-    int M, N, K, steps;                 // steps = K / (8 * 32)
+    int M, N, K, steps;                 // steps = K / (8 * 32), rounded up
+    float* out32;                       // when set, the (single) output range in fp32 instead of out[0]
+    const __nv_bfloat16* mul;           // when set, out[0] = act(x W) * mul, mul (M, mul_ld)
+    long long mul_ld;
+    int act;                            // of the gated pair, or of `mul`
     // APPEND: columns from n_end[0] on are the K and V projections of one new token per row and go to the paged cache
     // instead of out[1] / out[2] (arguments as bn_kv_append)
     __nv_bfloat16* pool;
@@ -50,7 +56,7 @@ struct SkinnyParams {
 // CH = K steps whose loads a lane keeps in flight at once.  More of them cover more latency per warp; fewer leave
 // registers for more CTAs per SM (8: two, 2: four), which matters when the grid would otherwise need a second, nearly
 // empty wave.
-template <bool SWIGLU, int CH, bool APPEND = false>
+template <bool SWIGLU, int CH, bool APPEND = false, bool RAGGED = false>
 __global__ void __launch_bounds__(SK_WARPS * 32)
 gemm_skinny_kernel(const SkinnyParams p) {
     __shared__ float s_part[SK_WARPS][2][16][8 + 1];
@@ -69,13 +75,16 @@ gemm_skinny_kernel(const SkinnyParams p) {
     // before it uses any of them - a launch of this kernel is one or two memory round trips long, and a load issued after
     // a wait would add its whole latency to that.
     const uint4 z = make_uint4(0, 0, 0, 0);
+    // whether this lane's 8 elements of step s lie inside K
+    auto inside = [&](int s) { return !RAGGED || kbase + (size_t)s * 32 < (size_t)p.K; };
     uint4 wv[CH], wv2[SWIGLU ? CH : 1], al[CH], ah[CH];
     auto load_weights = [&](int s0) {
 #pragma unroll
         for (int s = 0; s < CH; ++s)
             if (s0 + s < p.steps) {
-                wv[s] = __ldcs(bw + (size_t)(s0 + s) * 4);              // 32 K positions = 64 B = 4 x 16 B per row and step
-                if (SWIGLU) wv2[s] = __ldcs(bw2 + (size_t)(s0 + s) * 4);
+                // 32 K positions = 64 B = 4 x 16 B per row and step
+                wv[s] = inside(s0 + s) ? __ldcs(bw + (size_t)(s0 + s) * 4) : z;
+                if (SWIGLU) wv2[s] = inside(s0 + s) ? __ldcs(bw2 + (size_t)(s0 + s) * 4) : z;
             }
     };
     // The warp's whole slice of the 8 weight rows is requested into L2 at once (a 128-byte line is two steps of a
@@ -84,6 +93,7 @@ gemm_skinny_kernel(const SkinnyParams p) {
     // kernel before this one in the stream is still running - the weights do not depend on it, the activations do,
     // and nothing is READ before the wait (L2 is the point of coherence, so a line prefetched early cannot go stale).
     for (int s = 0; s < p.steps; s += 2) {
+        if (!inside(s)) break;
         asm volatile("prefetch.global.L2 [%0];" ::"l"(bw + (size_t)s * 4));
         if (SWIGLU) asm volatile("prefetch.global.L2 [%0];" ::"l"(bw2 + (size_t)s * 4));
     }
@@ -94,8 +104,8 @@ gemm_skinny_kernel(const SkinnyParams p) {
 #pragma unroll
         for (int s = 0; s < CH; ++s)
             if (s0 + s < p.steps) {
-                al[s] = lo_ok ? __ldg(a_lo + (size_t)(s0 + s) * 4) : z;
-                ah[s] = hi_ok ? __ldg(a_hi + (size_t)(s0 + s) * 4) : z;
+                al[s] = lo_ok && inside(s0 + s) ? __ldg(a_lo + (size_t)(s0 + s) * 4) : z;
+                ah[s] = hi_ok && inside(s0 + s) ? __ldg(a_hi + (size_t)(s0 + s) * 4) : z;
             }
 #pragma unroll
         for (int s = 0; s < CH; ++s)
@@ -131,7 +141,7 @@ gemm_skinny_kernel(const SkinnyParams p) {
                 v += s_part[w][0][row][col];
                 if (SWIGLU) u += s_part[w][1][row][col];
             }
-            if (SWIGLU) v = __fdividef(v, 1.f + __expf(-v)) * u;          // silu(gate) * up
+            if (SWIGLU) v = activation_fast(p.act, v) * u;                // act(gate) * up
         }
         const int n = n0 + col;
         if (APPEND && n >= p.n_end[0]) {       // the same for the CTA's 8 columns: the ranges are multiples of 8
@@ -160,7 +170,10 @@ gemm_skinny_kernel(const SkinnyParams p) {
                     }
                 }
             }
+        } else if (row < p.M && p.out32) {
+            p.out32[(size_t)row * p.N + n] = v;
         } else if (row < p.M) {
+            if (p.mul) v = activation_fast(p.act, v) * __bfloat162float(p.mul[row * p.mul_ld + n]);
             // selects, not indexed parameter arrays (an index known only at run time would copy them to local memory)
             __nv_bfloat16* o = p.out[0];
             int ld = p.ld[0], first = 0;
@@ -175,11 +188,25 @@ static int skinny_check(const char* what, const void* a, const void* bt, int M, 
     if (!a || !bt) return fail(BN_ERR_INVALID_ARG, "%s: null pointer", what);
     if (M <= 0 || M > 16) return fail(BN_ERR_UNSUPPORTED, "%s: M=%d (1..16 rows)", what, M);
     if (N <= 0 || N % 8) return fail(BN_ERR_UNSUPPORTED, "%s: N=%d must be a positive multiple of 8", what, N);
-    if (K <= 0 || K % 256 || K > SK_WARPS * 32 * SK_MAX_STEPS)
-        return fail(BN_ERR_UNSUPPORTED, "%s: K=%d must be a multiple of 256, at most %d", what, K, SK_WARPS * 32 * SK_MAX_STEPS);
+    if (K <= 0 || K % 8 || K > SK_WARPS * 32 * SK_MAX_STEPS)
+        return fail(BN_ERR_UNSUPPORTED, "%s: K=%d must be a multiple of 8, at most %d", what, K, SK_WARPS * 32 * SK_MAX_STEPS);
     if ((reinterpret_cast<uintptr_t>(a) | reinterpret_cast<uintptr_t>(bt)) & 15)
         return fail(BN_ERR_INVALID_ARG, "%s: a/bt must be 16-byte aligned", what);
     return require_sm100();
+}
+
+// Measured on the decode step's shapes: 256 CTAs (o, down) run fastest two per SM with 8 steps in flight, 320 (q/k/v in
+// one launch) four per SM with 2; the gated pair holds two weights and runs with 2.
+template <bool GLU, bool APPEND>
+static int skinny_launch(const SkinnyParams& p, cudaStream_t st, const char* what) {
+    int dev = 0, sms = 148;
+    cudaGetDevice(&dev);
+    cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
+    const bool deep = !GLU && p.N / 8 <= 2 * sms;
+    if (p.K % (SK_WARPS * 32)) launch_dependent(gemm_skinny_kernel<GLU, 2, APPEND, true>, p.N / 8, SK_WARPS * 32, 0, st, p);
+    else if (deep) launch_dependent(gemm_skinny_kernel<GLU, GLU ? 2 : 8, APPEND>, p.N / 8, SK_WARPS * 32, 0, st, p);
+    else launch_dependent(gemm_skinny_kernel<GLU, 2, APPEND>, p.N / 8, SK_WARPS * 32, 0, st, p);
+    return launch_status(what);
 }
 
 }  // namespace bn
@@ -202,33 +229,60 @@ extern "C" int bn_gemm_bf16_nt_skinny(const void* a, const void* bt, int M, int 
     p.out[2] = static_cast<__nv_bfloat16*>(out2);
     p.n_end[0] = n0; p.n_end[1] = n0 + n1; p.n_end[2] = N;
     p.ld[0] = n0; p.ld[1] = n1; p.ld[2] = N - n0 - n1;
-    p.M = M; p.N = N; p.K = K; p.steps = K / (SK_WARPS * 32);
-    // measured on the decode step's shapes: 256 CTAs (o, down) run fastest two per SM with 8 steps in flight, 320 (q/k/v
-    // in one launch) four per SM with 2
-    int dev = 0, sms = 148;
-    cudaGetDevice(&dev);
-    cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
-    if (N / 8 <= 2 * sms) launch_dependent(gemm_skinny_kernel<false, 8>, N / 8, SK_WARPS * 32, 0, as_stream(stream), p);
-    else launch_dependent(gemm_skinny_kernel<false, 2>, N / 8, SK_WARPS * 32, 0, as_stream(stream), p);
-    return launch_status(what);
+    p.M = M; p.N = N; p.K = K; p.steps = (K + SK_WARPS * 32 - 1) / (SK_WARPS * 32);
+    return skinny_launch<false, false>(p, as_stream(stream), what);
 }
 
-extern "C" int bn_gemm_swiglu_bf16_nt_skinny(const void* x, const void* gate_t, const void* up_t, void* h, int M, int inter,
-                                             int K, bn_stream_t stream) {
-    const char* what = "bn_gemm_swiglu_bf16_nt_skinny";
+extern "C" int bn_gemm_bf16_nt_skinny_f32(const void* a, const void* bt, int M, int N, int K, float* out, bn_stream_t stream) {
+    const char* what = "bn_gemm_bf16_nt_skinny_f32";
+    if (int rc = skinny_check(what, a, bt, M, N, K)) return rc;
+    if (!out) return fail(BN_ERR_INVALID_ARG, "%s: null pointer", what);
+    SkinnyParams p{};
+    p.a = static_cast<const __nv_bfloat16*>(a);
+    p.bt = static_cast<const __nv_bfloat16*>(bt);
+    p.out32 = out;
+    p.n_end[0] = p.n_end[1] = p.n_end[2] = N;
+    p.M = M; p.N = N; p.K = K; p.steps = (K + SK_WARPS * 32 - 1) / (SK_WARPS * 32);
+    return skinny_launch<false, false>(p, as_stream(stream), what);
+}
+
+extern "C" int bn_gemm_act_mul_bf16_nt_skinny(const void* a, const void* bt, const void* mul, int64_t mul_ld, void* out, int M,
+                                              int N, int K, int act, bn_stream_t stream) {
+    const char* what = "bn_gemm_act_mul_bf16_nt_skinny";
+    if (int rc = skinny_check(what, a, bt, M, N, K)) return rc;
+    if (!mul || !out || mul_ld < N || act < 0 || act > BN_ACT_LAST) return fail(BN_ERR_INVALID_ARG, "%s: bad argument", what);
+    SkinnyParams p{};
+    p.a = static_cast<const __nv_bfloat16*>(a);
+    p.bt = static_cast<const __nv_bfloat16*>(bt);
+    p.out[0] = static_cast<__nv_bfloat16*>(out);
+    p.n_end[0] = p.n_end[1] = p.n_end[2] = N;
+    p.ld[0] = N;
+    p.mul = static_cast<const __nv_bfloat16*>(mul); p.mul_ld = mul_ld; p.act = act;
+    p.M = M; p.N = N; p.K = K; p.steps = (K + SK_WARPS * 32 - 1) / (SK_WARPS * 32);
+    return skinny_launch<false, false>(p, as_stream(stream), what);
+}
+
+extern "C" int bn_gemm_glu_bf16_nt_skinny(const void* x, const void* gate_t, const void* up_t, void* h, int M, int inter,
+                                          int K, int act, bn_stream_t stream) {
+    const char* what = "bn_gemm_glu_bf16_nt_skinny";
     if (int rc = skinny_check(what, x, gate_t, M, inter, K)) return rc;
     if (!up_t || !h || (reinterpret_cast<uintptr_t>(up_t) & 15)) return fail(BN_ERR_INVALID_ARG, "%s: null or misaligned pointer", what);
+    if (act < 0 || act > BN_ACT_LAST) return fail(BN_ERR_INVALID_ARG, "%s: activation %d", what, act);
     SkinnyParams p{};
     p.a = static_cast<const __nv_bfloat16*>(x);
     p.bt = static_cast<const __nv_bfloat16*>(gate_t);
     p.bt2 = static_cast<const __nv_bfloat16*>(up_t);
     p.out[0] = static_cast<__nv_bfloat16*>(h);
-    p.out[1] = p.out[2] = nullptr;
     p.n_end[0] = p.n_end[1] = p.n_end[2] = inter;
-    p.ld[0] = inter; p.ld[1] = p.ld[2] = 0;
-    p.M = M; p.N = inter; p.K = K; p.steps = K / (SK_WARPS * 32);
-    launch_dependent(gemm_skinny_kernel<true, 2>, inter / 8, SK_WARPS * 32, 0, as_stream(stream), p);
-    return launch_status(what);
+    p.ld[0] = inter;
+    p.act = act;
+    p.M = M; p.N = inter; p.K = K; p.steps = (K + SK_WARPS * 32 - 1) / (SK_WARPS * 32);
+    return skinny_launch<true, false>(p, as_stream(stream), what);
+}
+
+extern "C" int bn_gemm_swiglu_bf16_nt_skinny(const void* x, const void* gate_t, const void* up_t, void* h, int M, int inter,
+                                             int K, bn_stream_t stream) {
+    return bn_gemm_glu_bf16_nt_skinny(x, gate_t, up_t, h, M, inter, K, BN_ACT_SILU, stream);
 }
 
 extern "C" int bn_gemm_qkv_append_bf16_skinny(const void* x, const void* wqkv_t, int M, int hidden, int Hq, int Hkv, int D,
@@ -248,14 +302,9 @@ extern "C" int bn_gemm_qkv_append_bf16_skinny(const void* x, const void* wqkv_t,
     p.out[0] = static_cast<__nv_bfloat16*>(q_out);
     p.n_end[0] = Hq * D; p.n_end[1] = (Hq + Hkv) * D; p.n_end[2] = N;
     p.ld[0] = Hq * D;
-    p.M = M; p.N = N; p.K = hidden; p.steps = hidden / (SK_WARPS * 32);
+    p.M = M; p.N = N; p.K = hidden; p.steps = (hidden + SK_WARPS * 32 - 1) / (SK_WARPS * 32);
     p.pool = static_cast<__nv_bfloat16*>(pool);
     p.page_table = page_table; p.seq_ids = seq_ids; p.positions = positions;
     p.pool_pages = pool_pages; p.max_pages = max_pages; p.Hkv = Hkv; p.D = D; p.theta = theta;
-    int dev = 0, sms = 148;
-    cudaGetDevice(&dev);
-    cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
-    if (N / 8 <= 2 * sms) launch_dependent(gemm_skinny_kernel<false, 8, true>, N / 8, SK_WARPS * 32, 0, as_stream(stream), p);
-    else launch_dependent(gemm_skinny_kernel<false, 2, true>, N / 8, SK_WARPS * 32, 0, as_stream(stream), p);
-    return launch_status(what);
+    return skinny_launch<false, true>(p, as_stream(stream), what);
 }

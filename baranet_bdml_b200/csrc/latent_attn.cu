@@ -1,0 +1,597 @@
+// Latent attention with a sliding window: keys and values of a token are expanded from one normalised latent vector c
+// (kv_rank wide) plus one rotated key part (rot wide) that all heads share, so those two are all that is cached.
+//
+//   prompt portions   the latents of the window before the portion are gathered from the cache in front of the
+//                     portion's own, both are expanded by ONE product to per-head keys and values, and attention runs
+//                     over those rows                               (bn_latent_prep, bn_latent_gather, bn_attn_window)
+//   one new token     the key expansion moves to the query side, q_c = W_uk^T q, so scores are taken against the cached
+//                     latents themselves; the weighted sum of latents is expanded once at the end
+//                                                     (bn_latent_absorb_q, bn_latent_decode, bn_latent_expand_out)
+//
+// Cache: ring[slot][ring_tokens][c: kv_ld | rotated key part: rot_ld], the token of position p at row p % ring_tokens,
+// ring_tokens >= window: what the window has passed is overwritten.  kv_ld and rot_ld are kv_rank and rot rounded up to
+// multiples of 8; the columns in between hold zeros, in the ring and in every buffer of the same shape, so products and
+// dot products may run over them.
+//
+// The kernels of this file take any sizes, in fp32 and in bf16; the tensor-core forms for the common sizes are in
+// latent_prefill_sm100.cu and latent_decode.cu.
+#include "common.cuh"
+#include "hybrid.cuh"
+#include "latent.cuh"
+
+namespace bn {
+
+// ---------------------------------------------------------------------------------------------------------------
+// One row of the down projections [c_q: q_rank | c: kv_rank | k_rot: rot] -> normalised c_q, normalised c, rotated
+// k_rot, and the last two into the cache
+// ---------------------------------------------------------------------------------------------------------------
+struct LatentPrepParams {
+    const void* proj;
+    int64_t proj_ld;
+    const float *q_norm, *kv_norm;
+    const double* freq;
+    const int32_t *seq_ids, *positions;
+    void *cq, *c, *krot, *ring;
+    int64_t cq_ld;
+    int rows, S, q_rank, kv_rank, rot, kv_ld, rot_ld, rows_per_seq, row_offset, ring_tokens;
+    float eps;
+};
+
+constexpr int LP_THREADS = 128;
+
+template <typename T>
+__global__ void __launch_bounds__(LP_THREADS)
+latent_prep_kernel(const LatentPrepParams p) {
+    __shared__ float sh[2][LP_THREADS / 32];
+    ptx::grid_dependency_wait();
+    ptx::grid_launch_dependents();
+    for (int r = blockIdx.x; r < p.rows; r += gridDim.x) {
+        const int b = r / p.S, s = r - b * p.S;
+        const T* in = static_cast<const T*>(p.proj) + (int64_t)r * p.proj_ld;
+        float sq = 0.f, sk = 0.f;
+        for (int i = threadIdx.x; i < p.q_rank; i += LP_THREADS) { const float v = to_f(in[i]); sq = fmaf(v, v, sq); }
+        for (int i = threadIdx.x; i < p.kv_rank; i += LP_THREADS) { const float v = to_f(in[p.q_rank + i]); sk = fmaf(v, v, sk); }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            sq += __shfl_xor_sync(0xffffffffu, sq, o);
+            sk += __shfl_xor_sync(0xffffffffu, sk, o);
+        }
+        __syncthreads();
+        if (threadIdx.x % 32 == 0) { sh[0][threadIdx.x / 32] = sq; sh[1][threadIdx.x / 32] = sk; }
+        __syncthreads();
+        sq = sk = 0.f;
+#pragma unroll
+        for (int w = 0; w < LP_THREADS / 32; ++w) { sq += sh[0][w]; sk += sh[1][w]; }
+        const float inv_q = rsqrtf(sq / (float)p.q_rank + p.eps), inv_k = rsqrtf(sk / (float)p.kv_rank + p.eps);
+
+        T* cq = static_cast<T*>(p.cq) + (int64_t)r * p.cq_ld;
+        for (int i = threadIdx.x; i < p.cq_ld; i += LP_THREADS)
+            cq[i] = from_f<T>(i < p.q_rank ? to_f(in[i]) * inv_q * p.q_norm[i] : 0.f);
+
+        const int pos = p.positions[b] + s;
+        const int64_t out_row = (int64_t)b * p.rows_per_seq + p.row_offset + s;
+        T* c = p.c ? static_cast<T*>(p.c) + out_row * p.kv_ld : nullptr;
+        T* kr = p.krot ? static_cast<T*>(p.krot) + out_row * p.rot_ld : nullptr;
+        // of a portion longer than the ring only the last ring_tokens rows are kept, so no ring row is written twice
+        T* ring = nullptr;
+        if (p.ring && s >= p.S - p.ring_tokens) {
+            const int slot = p.seq_ids ? p.seq_ids[b] : b;
+            ring = static_cast<T*>(p.ring) + ((int64_t)slot * p.ring_tokens + pos % p.ring_tokens) * (p.kv_ld + p.rot_ld);
+        }
+        for (int i = threadIdx.x; i < p.kv_ld; i += LP_THREADS) {
+            const T v = from_f<T>(i < p.kv_rank ? to_f(in[p.q_rank + i]) * inv_k * p.kv_norm[i] : 0.f);
+            if (c) c[i] = v;
+            if (ring) ring[i] = v;
+        }
+        const T* rin = in + p.q_rank + p.kv_rank;
+        for (int i = threadIdx.x; i < p.rot_ld / 2; i += LP_THREADS) {
+            T lo = from_f<T>(0.f), hi = lo;
+            if (2 * i < p.rot) {
+                const float u = to_f(rin[2 * i]), v = to_f(rin[2 * i + 1]);
+                float cs, sn;
+                rotation(pos, p.freq[i], &cs, &sn);
+                lo = from_f<T>(u * cs - v * sn);
+                hi = from_f<T>(v * cs + u * sn);
+            }
+            if (kr) { kr[2 * i] = lo; kr[2 * i + 1] = hi; }
+            if (ring) { ring[p.kv_ld + 2 * i] = lo; ring[p.kv_ld + 2 * i + 1] = hi; }
+        }
+    }
+}
+
+// the `n_old` tokens before the portion, out of the ring, to rows 0 .. n_old - 1 of each sequence's block of rows
+template <typename T>
+__global__ void __launch_bounds__(128)
+latent_gather_kernel(const T* ring, int ring_tokens, int kv_ld, int rot_ld, const int32_t* seq_ids, const int32_t* positions,
+                     int B, int n_old, T* c, T* krot, int rows_per_seq) {
+    ptx::grid_dependency_wait();
+    ptx::grid_launch_dependents();
+    for (int r = blockIdx.x; r < B * n_old; r += gridDim.x) {
+        const int b = r / n_old, i = r - b * n_old;
+        const int pos = positions[b] - n_old + i;
+        if (pos < 0) continue;                         // the host sized n_old by the same positions
+        const int slot = seq_ids ? seq_ids[b] : b;
+        const T* src = ring + ((int64_t)slot * ring_tokens + pos % ring_tokens) * (kv_ld + rot_ld);
+        T* cd = c + ((int64_t)b * rows_per_seq + i) * kv_ld;
+        T* kd = krot + ((int64_t)b * rows_per_seq + i) * rot_ld;
+        for (int j = threadIdx.x; j < kv_ld; j += 128) cd[j] = src[j];
+        for (int j = threadIdx.x; j < rot_ld; j += 128) kd[j] = src[kv_ld + j];
+    }
+}
+
+// rotates, in place, the last `rot` of each head's `dim + rot` columns
+template <typename T>
+__global__ void __launch_bounds__(256)
+rope_heads_kernel(T* q, int64_t q_ld, long long n, int S, int H, int dim, int rot, const double* freq, const int32_t* positions) {
+    ptx::grid_dependency_wait();
+    ptx::grid_launch_dependents();
+    const int half = rot / 2;
+    for (long long i = (long long)blockIdx.x * 256 + threadIdx.x; i < n; i += (long long)gridDim.x * 256) {
+        // n = rows * half pairs: a thread turns one pair of one row in every head, with one sine and cosine
+        const int64_t r = i / half;
+        const int j = (int)(i - r * half);
+        float cs, sn;
+        rotation(positions[r / S] + (int)(r % S), freq[j], &cs, &sn);
+        T* x = q + r * q_ld + dim + 2 * j;
+        for (int h = 0; h < H; ++h, x += dim + rot) {
+            const float u = to_f(x[0]), v = to_f(x[1]);
+            x[0] = from_f<T>(u * cs - v * sn);
+            x[1] = from_f<T>(v * cs + u * sn);
+        }
+    }
+}
+
+// ---------------------------------------------------------------------------------------------------------------
+// Windowed attention over expanded keys, any sizes: a warp per (query row, head); 32 keys at a time, a lane per key for
+// the scores, then a lane per value column.  Scores, weights and sums in fp32.
+// ---------------------------------------------------------------------------------------------------------------
+constexpr int AW_WARPS = 4, AW_MAXV = 16;      // vdim <= 512
+
+template <typename T>
+__global__ void __launch_bounds__(AW_WARPS * 32)
+attn_window_kernel(const AttnWindowParams p) {
+    extern __shared__ float q_smem[];
+    ptx::grid_dependency_wait();
+    ptx::grid_launch_dependents();
+    const int warp = threadIdx.x / 32, lane = threadIdx.x % 32;
+    const int E = p.dim + p.rot;
+    float* qs = q_smem + warp * E;
+    const long long n = (long long)p.B * p.S * p.H;
+    for (long long item = (long long)blockIdx.x * AW_WARPS + warp; item < n; item += (long long)gridDim.x * AW_WARPS) {
+        const int h = (int)(item % p.H);
+        const long long row = item / p.H;
+        const int b = (int)(row / p.S), s = (int)(row - (long long)b * p.S);
+        const T* q = static_cast<const T*>(p.q) + row * p.q_ld + h * E;
+        __syncwarp();
+        for (int e = lane; e < E; e += 32) qs[e] = to_f(q[e]);
+        __syncwarp();
+        const int last = p.n_old + s, first = max(0, last - p.window + 1);
+        const int64_t seq_row = (int64_t)b * p.rows_per_seq;
+        float m = -INFINITY, l = 0.f, acc[AW_MAXV];
+#pragma unroll
+        for (int v = 0; v < AW_MAXV; ++v) acc[v] = 0.f;
+        for (int k0 = first; k0 <= last; k0 += 32) {
+            const int k = k0 + lane;
+            float sc = -INFINITY;
+            if (k <= last) {
+                const T* kn = static_cast<const T*>(p.k) + (seq_row + k) * p.kv_ld + h * p.dim;
+                const T* kr = static_cast<const T*>(p.krot) + (seq_row + k) * p.krot_ld;
+                float d = 0.f;
+                for (int e = 0; e < p.dim; ++e) d = fmaf(qs[e], to_f(kn[e]), d);
+                for (int e = 0; e < p.rot; ++e) d = fmaf(qs[p.dim + e], to_f(kr[e]), d);
+                sc = d * p.scale;
+            }
+            float mx = sc;
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+            const float m_new = fmaxf(m, mx);
+            const float shrink = expf(m - m_new);      // 0 at the first keys (m = -inf)
+            const float w = expf(sc - m_new);
+            float sum = w;
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+            l = l * shrink + sum;
+            m = m_new;
+#pragma unroll
+            for (int v = 0; v < AW_MAXV; ++v) acc[v] *= shrink;
+            const int nk = min(32, last - k0 + 1);
+            for (int j = 0; j < nk; ++j) {
+                const float wj = __shfl_sync(0xffffffffu, w, j);
+                const T* vr = static_cast<const T*>(p.v) + (seq_row + k0 + j) * p.kv_ld + h * p.vdim;
+#pragma unroll
+                for (int v = 0; v < AW_MAXV; ++v)
+                    if (v * 32 + lane < p.vdim) acc[v] = fmaf(wj, to_f(vr[v * 32 + lane]), acc[v]);
+            }
+        }
+        T* out = static_cast<T*>(p.out) + row * p.out_ld + h * p.vdim;
+#pragma unroll
+        for (int v = 0; v < AW_MAXV; ++v)
+            if (v * 32 + lane < p.vdim) out[v * 32 + lane] = from_f<T>(acc[v] / l);
+        if (h == p.H - 1)                                   // the padding columns behind the last head
+            for (int i = p.H * p.vdim + lane; i < p.out_ld; i += 32)
+                static_cast<T*>(p.out)[row * p.out_ld + i] = from_f<T>(0.f);
+    }
+}
+
+// ---------------------------------------------------------------------------------------------------------------
+// One new token per row: the query moved into latent space.  Block (n tile, head); the last n tile is the rotation.
+//   q_abs[b][h][0..kv_ld) = sum_i q[b][h][i] W_uk[h * dim + i][:]      q_abs[b][h][kv_ld..) = rotated part
+// ---------------------------------------------------------------------------------------------------------------
+constexpr int LA_N = 128, LA_B = 8;
+
+template <typename T>
+__global__ void __launch_bounds__(LA_N)
+latent_absorb_kernel(const T* q, int64_t q_ld, const T* wuk, const double* freq, const int32_t* positions, T* q_abs, int B, int H,
+                     int dim, int rot, int kv_ld, int rot_ld) {
+    extern __shared__ float q_smem[];                   // [LA_B][dim]
+    ptx::grid_dependency_wait();
+    ptx::grid_launch_dependents();
+    const int h = blockIdx.x % H, tile = blockIdx.x / H, n_tiles = (kv_ld + LA_N - 1) / LA_N;
+    const int width = kv_ld + rot_ld;
+    if (tile == n_tiles) {
+        for (int i = threadIdx.x; i < B * (rot_ld / 2); i += LA_N) {
+            const int b = i / (rot_ld / 2), j = i % (rot_ld / 2);
+            T lo = from_f<T>(0.f), hi = lo;
+            if (2 * j < rot) {
+                const T* x = q + b * q_ld + h * (dim + rot) + dim + 2 * j;
+                const float u = to_f(x[0]), v = to_f(x[1]);
+                float cs, sn;
+                rotation(positions[b], freq[j], &cs, &sn);
+                lo = from_f<T>(u * cs - v * sn);
+                hi = from_f<T>(v * cs + u * sn);
+            }
+            T* o = q_abs + ((int64_t)b * H + h) * width + kv_ld + 2 * j;
+            o[0] = lo;
+            o[1] = hi;
+        }
+        return;
+    }
+    const int n = tile * LA_N + threadIdx.x;
+    for (int b0 = 0; b0 < B; b0 += LA_B) {
+        const int nb = min(LA_B, B - b0);
+        __syncthreads();
+        for (int i = threadIdx.x; i < LA_B * dim; i += LA_N) {
+            const int b = i / dim, e = i - b * dim;
+            q_smem[i] = b < nb ? to_f(q[(b0 + b) * q_ld + h * (dim + rot) + e]) : 0.f;
+        }
+        __syncthreads();
+        if (n < kv_ld) {
+            float acc[LA_B];
+#pragma unroll
+            for (int b = 0; b < LA_B; ++b) acc[b] = 0.f;
+            const T* w = wuk + (int64_t)h * dim * kv_ld + n;
+#pragma unroll 8
+            for (int e = 0; e < dim; ++e) {
+                const float wv = to_f(w[(int64_t)e * kv_ld]);
+#pragma unroll
+                for (int b = 0; b < LA_B; ++b) acc[b] = fmaf(q_smem[b * dim + e], wv, acc[b]);
+            }
+#pragma unroll
+            for (int b = 0; b < LA_B; ++b)
+                if (b < nb) q_abs[((int64_t)(b0 + b) * H + h) * width + n] = from_f<T>(acc[b]);
+        }
+    }
+}
+
+// ---------------------------------------------------------------------------------------------------------------
+// Scores and weighted latent sum over the ring, any sizes.  Block (row, head, split); warps take 32 keys at a time.
+// The partial result of a split is the normalised sum and its log-sum-exp.
+// ---------------------------------------------------------------------------------------------------------------
+constexpr int LD_WARPS = 4, LD_MAXN = 32;              // kv_ld <= 1024
+
+template <typename T>
+__global__ void __launch_bounds__(LD_WARPS * 32)
+latent_decode_any_kernel(const LatentDecodeParams p) {
+    extern __shared__ float smem[];
+    ptx::grid_dependency_wait();
+    ptx::grid_launch_dependents();
+    const int warp = threadIdx.x / 32, lane = threadIdx.x % 32;
+    const int width = p.kv_ld + p.rot_ld;
+    float* qs = smem;                                   // [width]
+    float* s_acc = smem + width;                        // [LD_WARPS][kv_ld]
+    float* s_ml = s_acc + LD_WARPS * p.kv_ld;           // [LD_WARPS][2]
+    const int split = blockIdx.x % p.splits, h = (blockIdx.x / p.splits) % p.H, b = blockIdx.x / (p.splits * p.H);
+    const int pos = p.positions[b], slot = p.seq_ids ? p.seq_ids[b] : b;
+    const T* q = static_cast<const T*>(p.q_abs) + ((int64_t)b * p.H + h) * width;
+    for (int e = threadIdx.x; e < width; e += blockDim.x) qs[e] = to_f(q[e]);
+    __syncthreads();
+    const int first = max(0, pos - p.window + 1), count = pos - first + 1;
+    const int per = ((count + p.splits - 1) / p.splits + 31) / 32 * 32;
+    const int k_begin = first + split * per, k_end = min(pos + 1, k_begin + per);
+    const T* ring = static_cast<const T*>(p.ring) + (int64_t)slot * p.ring_tokens * width;
+    float m = -INFINITY, l = 0.f, acc[LD_MAXN];
+#pragma unroll
+    for (int v = 0; v < LD_MAXN; ++v) acc[v] = 0.f;
+    for (int k0 = k_begin + warp * 32; k0 < k_end; k0 += LD_WARPS * 32) {
+        const int k = k0 + lane;
+        float sc = -INFINITY;
+        if (k < k_end) {
+            const T* row = ring + (int64_t)(k % p.ring_tokens) * width;
+            float d = 0.f;
+            for (int e = 0; e < width; ++e) d = fmaf(qs[e], to_f(row[e]), d);
+            sc = d * p.scale;
+        }
+        float mx = sc;
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+        const float m_new = fmaxf(m, mx), shrink = expf(m - m_new), w = expf(sc - m_new);
+        float sum = w;
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+        l = l * shrink + sum;
+        m = m_new;
+#pragma unroll
+        for (int v = 0; v < LD_MAXN; ++v) acc[v] *= shrink;
+        const int nk = min(32, k_end - k0);
+        for (int j = 0; j < nk; ++j) {
+            const float wj = __shfl_sync(0xffffffffu, w, j);
+            const T* row = ring + (int64_t)((k0 + j) % p.ring_tokens) * width;
+#pragma unroll
+            for (int v = 0; v < LD_MAXN; ++v)
+                if (v * 32 + lane < p.kv_ld) acc[v] = fmaf(wj, to_f(row[v * 32 + lane]), acc[v]);
+        }
+    }
+    for (int v = 0; v < LD_MAXN; ++v)
+        if (v * 32 + lane < p.kv_ld) s_acc[warp * p.kv_ld + v * 32 + lane] = acc[v];
+    if (lane == 0) { s_ml[warp * 2] = m; s_ml[warp * 2 + 1] = l; }
+    __syncthreads();
+    float M = -INFINITY;
+#pragma unroll
+    for (int w = 0; w < LD_WARPS; ++w) M = fmaxf(M, s_ml[w * 2]);
+    float L = 0.f, f[LD_WARPS];
+#pragma unroll
+    for (int w = 0; w < LD_WARPS; ++w) {
+        f[w] = M == -INFINITY ? 0.f : expf(s_ml[w * 2] - M);
+        L = fmaf(s_ml[w * 2 + 1], f[w], L);
+    }
+    const int64_t part = ((int64_t)b * p.H + h) * p.splits + split;
+    for (int i = threadIdx.x; i < p.kv_ld; i += blockDim.x) {
+        float o = 0.f;
+#pragma unroll
+        for (int w = 0; w < LD_WARPS; ++w) o = fmaf(s_acc[w * p.kv_ld + i], f[w], o);
+        p.partial[part * p.kv_ld + i] = L > 0.f ? o / L : 0.f;
+    }
+    if (threadIdx.x == 0) p.lse[part] = L > 0.f ? M + logf(L) : -INFINITY;
+}
+
+// ---------------------------------------------------------------------------------------------------------------
+// Merges the splits and expands the latent sum to the head's values: out[b][h][v] = sum_n W_uv[h * vdim + v][n] o[n].
+// Block (value tile of LO_V rows, head, group of LO_B rows); a warp per value row.
+// ---------------------------------------------------------------------------------------------------------------
+constexpr int LO_WARPS = 8, LO_V = 32, LO_B = 4;
+
+template <typename T>
+__global__ void __launch_bounds__(LO_WARPS * 32)
+latent_expand_out_kernel(const float* partial, const float* lse, int splits, const T* wuv, T* out, int64_t out_ld, int B, int H,
+                         int vdim, int kv_ld) {
+    extern __shared__ float o_smem[];                   // [LO_B][kv_ld]
+    ptx::grid_dependency_wait();
+    ptx::grid_launch_dependents();
+    const int v_tiles = (vdim + LO_V - 1) / LO_V;
+    const int vt = blockIdx.x % v_tiles, h = (blockIdx.x / v_tiles) % H, b0 = blockIdx.x / (v_tiles * H) * LO_B;
+    const int warp = threadIdx.x / 32, lane = threadIdx.x % 32, nb = min(LO_B, B - b0);
+    for (int b = 0; b < LO_B; ++b) {
+        if (b >= nb) {
+            for (int i = threadIdx.x; i < kv_ld; i += blockDim.x) o_smem[b * kv_ld + i] = 0.f;
+            continue;
+        }
+        const int64_t part = ((int64_t)(b0 + b) * H + h) * splits;
+        float M = -INFINITY;
+        for (int s = 0; s < splits; ++s) M = fmaxf(M, lse[part + s]);
+        float L = 0.f;
+        for (int s = 0; s < splits; ++s) L += expf(lse[part + s] - M);
+        const float inv = 1.f / L;
+        for (int i = threadIdx.x; i < kv_ld; i += blockDim.x) {
+            float o = 0.f;
+            for (int s = 0; s < splits; ++s) o = fmaf(partial[(part + s) * kv_ld + i], expf(lse[part + s] - M), o);
+            o_smem[b * kv_ld + i] = o * inv;
+        }
+    }
+    __syncthreads();
+    for (int v = vt * LO_V + warp; v < min(vdim, (vt + 1) * LO_V); v += LO_WARPS) {
+        const T* w = wuv + ((int64_t)h * vdim + v) * kv_ld;
+        float acc[LO_B];
+#pragma unroll
+        for (int b = 0; b < LO_B; ++b) acc[b] = 0.f;
+#pragma unroll 4
+        for (int i = lane; i < kv_ld; i += 32) {
+            const float wv = to_f(w[i]);
+#pragma unroll
+            for (int b = 0; b < LO_B; ++b) acc[b] = fmaf(wv, o_smem[b * kv_ld + i], acc[b]);
+        }
+#pragma unroll
+        for (int b = 0; b < LO_B; ++b) {
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) acc[b] += __shfl_xor_sync(0xffffffffu, acc[b], o);
+            if (lane == 0 && b < nb) out[(b0 + b) * out_ld + h * vdim + v] = from_f<T>(acc[b]);
+        }
+    }
+    if (h == H - 1 && vt == 0)                          // the padding columns behind the last head
+        for (int b = 0; b < nb; ++b)
+            for (int i = H * vdim + threadIdx.x; i < out_ld; i += blockDim.x) out[(b0 + b) * out_ld + i] = from_f<T>(0.f);
+}
+
+static int sm_count() {
+    int dev = 0, sms = 148;
+    cudaGetDevice(&dev);
+    cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
+    return sms;
+}
+
+template <typename K>
+static int allow_smem(K kernel, size_t bytes, const char* what) {
+    if (bytes <= 48 * 1024) return BN_OK;
+    if (bytes > 200 * 1024) return fail(BN_ERR_UNSUPPORTED, "%s: %zu bytes of shared memory", what, bytes);
+    cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
+    return e == cudaSuccess ? BN_OK : fail(BN_ERR_CUDA, "%s: %s", what, cudaGetErrorString(e));
+}
+
+}  // namespace bn
+
+using namespace bn;
+
+extern "C" int bn_latent_prep(const void* proj, int64_t proj_ld, const float* q_norm, const float* kv_norm, float eps,
+                              const double* freq, const int32_t* seq_ids, const int32_t* positions, int B, int S, int q_rank,
+                              int kv_rank, int rot, void* cq, int64_t cq_ld, void* c, void* krot, int rows_per_seq,
+                              int row_offset, void* ring, int ring_tokens, int dtype, bn_stream_t stream) {
+    const char* what = "bn_latent_prep";
+    if (!proj || !q_norm || !kv_norm || !freq || !positions || !cq || (!c) != (!krot)) return fail(BN_ERR_INVALID_ARG, "%s: null pointer", what);
+    if (B < 0 || S < 0 || q_rank <= 0 || kv_rank <= 0 || rot < 0 || rot % 2 || (ring && ring_tokens <= 0) || (dtype & ~1))
+        return fail(BN_ERR_INVALID_ARG, "%s: bad shape B=%d S=%d q_rank=%d kv_rank=%d rot=%d", what, B, S, q_rank, kv_rank, rot);
+    if (int rc = require_sm100()) return rc;
+    if (B == 0 || S == 0) return BN_OK;
+    LatentPrepParams p{proj, proj_ld, q_norm, kv_norm, freq, seq_ids, positions, cq, c, krot, ring, cq_ld, B * S, S, q_rank,
+                       kv_rank, rot, round8(kv_rank), round8(rot), rows_per_seq, row_offset, ring_tokens, eps};
+    const int cap = sm_count() * 16;
+    const unsigned grid = (unsigned)(B * S < cap ? B * S : cap);
+    if (dtype == 0) launch_dependent(latent_prep_kernel<float>, grid, LP_THREADS, 0, as_stream(stream), p);
+    else launch_dependent(latent_prep_kernel<__nv_bfloat16>, grid, LP_THREADS, 0, as_stream(stream), p);
+    return launch_status(what);
+}
+
+extern "C" int bn_latent_gather(const void* ring, int ring_tokens, int kv_rank, int rot, const int32_t* seq_ids,
+                                const int32_t* positions, int B, int n_old, void* c, void* krot, int rows_per_seq, int dtype,
+                                bn_stream_t stream) {
+    const char* what = "bn_latent_gather";
+    if (!ring || !positions || !c || !krot) return fail(BN_ERR_INVALID_ARG, "%s: null pointer", what);
+    if (B < 0 || n_old < 0 || n_old > ring_tokens || n_old > rows_per_seq || (dtype & ~1))
+        return fail(BN_ERR_INVALID_ARG, "%s: bad shape B=%d n_old=%d ring_tokens=%d", what, B, n_old, ring_tokens);
+    if (int rc = require_sm100()) return rc;
+    if (B == 0 || n_old == 0) return BN_OK;
+    const long long n = (long long)B * n_old, cap = (long long)sm_count() * 16;
+    const unsigned grid = (unsigned)(n < cap ? n : cap);
+    const int kl = round8(kv_rank), rl = round8(rot);
+    if (dtype == 0)
+        launch_dependent(latent_gather_kernel<float>, grid, 128, 0, as_stream(stream), static_cast<const float*>(ring), ring_tokens,
+                         kl, rl, seq_ids, positions, B, n_old, static_cast<float*>(c), static_cast<float*>(krot), rows_per_seq);
+    else
+        launch_dependent(latent_gather_kernel<__nv_bfloat16>, grid, 128, 0, as_stream(stream), static_cast<const __nv_bfloat16*>(ring),
+                         ring_tokens, kl, rl, seq_ids, positions, B, n_old, static_cast<__nv_bfloat16*>(c),
+                         static_cast<__nv_bfloat16*>(krot), rows_per_seq);
+    return launch_status(what);
+}
+
+extern "C" int bn_rope_heads(void* q, int64_t q_ld, int B, int S, int H, int dim, int rot, const double* freq,
+                             const int32_t* positions, int dtype, bn_stream_t stream) {
+    const char* what = "bn_rope_heads";
+    if (!q || !freq || !positions) return fail(BN_ERR_INVALID_ARG, "%s: null pointer", what);
+    if (B < 0 || S < 0 || H <= 0 || dim < 0 || rot < 0 || rot % 2 || (dtype & ~1)) return fail(BN_ERR_INVALID_ARG, "%s: bad shape", what);
+    if (int rc = require_sm100()) return rc;
+    const long long n = (long long)B * S * (rot / 2);
+    if (n == 0) return BN_OK;
+    const long long blocks = (n + 255) / 256, cap = (long long)sm_count() * 32;
+    const unsigned grid = (unsigned)(blocks < cap ? blocks : cap);
+    if (dtype == 0)
+        launch_dependent(rope_heads_kernel<float>, grid, 256, 0, as_stream(stream), static_cast<float*>(q), q_ld, n, S, H, dim, rot,
+                         freq, positions);
+    else
+        launch_dependent(rope_heads_kernel<__nv_bfloat16>, grid, 256, 0, as_stream(stream), static_cast<__nv_bfloat16*>(q), q_ld, n,
+                         S, H, dim, rot, freq, positions);
+    return launch_status(what);
+}
+
+extern "C" int bn_attn_window(const void* q, int64_t q_ld, const void* k, const void* v, int64_t kv_ld, const void* krot,
+                              int64_t krot_ld, void* out, int64_t out_ld, int B, int S, int n_old, int rows_per_seq, int H,
+                              int dim, int rot, int vdim, int window, float scale, int* error_word, int dtype,
+                              bn_stream_t stream) {
+    const char* what = "bn_attn_window";
+    if (!q || !k || !v || !krot || !out) return fail(BN_ERR_INVALID_ARG, "%s: null pointer", what);
+    if (B < 0 || S < 0 || n_old < 0 || n_old + S > rows_per_seq || H <= 0 || dim <= 0 || rot < 0 || vdim <= 0 || window <= 0 || (dtype & ~1))
+        return fail(BN_ERR_INVALID_ARG, "%s: bad shape B=%d S=%d n_old=%d H=%d dim=%d rot=%d vdim=%d window=%d", what, B, S, n_old,
+                    H, dim, rot, vdim, window);
+    if (int rc = require_sm100()) return rc;
+    if (B == 0 || S == 0) return BN_OK;
+    AttnWindowParams p{q, k, v, krot, out, q_ld, kv_ld, krot_ld, out_ld, B, S, n_old, rows_per_seq, H, dim, rot, vdim, window, scale,
+                       error_word};
+    if (dtype == 1 && attn_window_sm100_ok(p)) return attn_window_sm100(p, as_stream(stream));
+    if (vdim > AW_MAXV * 32) return fail(BN_ERR_UNSUPPORTED, "%s: vdim=%d (at most %d)", what, vdim, AW_MAXV * 32);
+    const size_t smem = (size_t)AW_WARPS * (dim + rot) * sizeof(float);
+    const long long blocks = ((long long)B * S * H + AW_WARPS - 1) / AW_WARPS, cap = (long long)sm_count() * 64;
+    const unsigned grid = (unsigned)(blocks < cap ? blocks : cap);
+    if (dtype == 0) {
+        if (int rc = allow_smem(attn_window_kernel<float>, smem, what)) return rc;
+        launch_dependent(attn_window_kernel<float>, grid, AW_WARPS * 32, smem, as_stream(stream), p);
+    } else {
+        if (int rc = allow_smem(attn_window_kernel<__nv_bfloat16>, smem, what)) return rc;
+        launch_dependent(attn_window_kernel<__nv_bfloat16>, grid, AW_WARPS * 32, smem, as_stream(stream), p);
+    }
+    return launch_status(what);
+}
+
+extern "C" int bn_latent_absorb_q(const void* q, int64_t q_ld, const void* wuk, const double* freq, const int32_t* positions,
+                                  void* q_abs, int B, int H, int dim, int rot, int kv_rank, int dtype, bn_stream_t stream) {
+    const char* what = "bn_latent_absorb_q";
+    if (!q || !wuk || !freq || !positions || !q_abs) return fail(BN_ERR_INVALID_ARG, "%s: null pointer", what);
+    if (B < 0 || H <= 0 || dim <= 0 || rot < 0 || rot % 2 || kv_rank <= 0 || (dtype & ~1)) return fail(BN_ERR_INVALID_ARG, "%s: bad shape", what);
+    if (int rc = require_sm100()) return rc;
+    if (B == 0) return BN_OK;
+    const int kl = round8(kv_rank), rl = round8(rot);
+    const unsigned grid = (unsigned)(H * ((kl + LA_N - 1) / LA_N + 1));
+    const size_t smem = (size_t)LA_B * dim * sizeof(float);
+    if (dtype == 0) {
+        if (int rc = allow_smem(latent_absorb_kernel<float>, smem, what)) return rc;
+        launch_dependent(latent_absorb_kernel<float>, grid, LA_N, smem, as_stream(stream), static_cast<const float*>(q), q_ld,
+                         static_cast<const float*>(wuk), freq, positions, static_cast<float*>(q_abs), B, H, dim, rot, kl, rl);
+    } else {
+        if (int rc = allow_smem(latent_absorb_kernel<__nv_bfloat16>, smem, what)) return rc;
+        launch_dependent(latent_absorb_kernel<__nv_bfloat16>, grid, LA_N, smem, as_stream(stream), static_cast<const __nv_bfloat16*>(q),
+                         q_ld, static_cast<const __nv_bfloat16*>(wuk), freq, positions, static_cast<__nv_bfloat16*>(q_abs), B, H, dim,
+                         rot, kl, rl);
+    }
+    return launch_status(what);
+}
+
+extern "C" int bn_latent_decode_splits(int B, int H, int kv_rank, int rot, int window, int dtype) {
+    if (B <= 0 || H <= 0 || window <= 0) return 0;
+    if (dtype == 1 && latent_decode_mma_ok(H, round8(kv_rank), round8(rot))) return latent_decode_mma_splits(B, H, window, sm_count());
+    long long want = (2LL * sm_count() + (long long)B * H - 1) / ((long long)B * H);
+    const long long most = (window + 127) / 128;
+    if (want > most) want = most;
+    return (int)(want < 1 ? 1 : want);
+}
+
+extern "C" int bn_latent_decode(const void* q_abs, const void* ring, int ring_tokens, const int32_t* seq_ids,
+                                const int32_t* positions, float* partial, float* lse, int splits, int B, int H, int kv_rank, int rot,
+                                int window, float scale, int dtype, bn_stream_t stream) {
+    const char* what = "bn_latent_decode";
+    if (!q_abs || !ring || !positions || !partial || !lse) return fail(BN_ERR_INVALID_ARG, "%s: null pointer", what);
+    if (B < 0 || H <= 0 || kv_rank <= 0 || rot < 0 || window <= 0 || ring_tokens < window || splits <= 0 || (dtype & ~1))
+        return fail(BN_ERR_INVALID_ARG, "%s: bad shape B=%d H=%d kv_rank=%d window=%d ring_tokens=%d", what, B, H, kv_rank, window, ring_tokens);
+    if (int rc = require_sm100()) return rc;
+    if (B == 0) return BN_OK;
+    LatentDecodeParams p{q_abs, ring, seq_ids, positions, partial, lse, B, H, round8(kv_rank), round8(rot), ring_tokens, window, splits, scale};
+    if (dtype == 1 && latent_decode_mma_ok(H, p.kv_ld, p.rot_ld)) return latent_decode_mma(p, as_stream(stream));
+    if (p.kv_ld > LD_MAXN * 32) return fail(BN_ERR_UNSUPPORTED, "%s: kv_rank=%d (at most %d)", what, kv_rank, LD_MAXN * 32);
+    const size_t smem = (size_t)(p.kv_ld + p.rot_ld + LD_WARPS * p.kv_ld + LD_WARPS * 2) * sizeof(float);
+    const unsigned grid = (unsigned)((long long)B * H * splits);
+    if (dtype == 0) {
+        if (int rc = allow_smem(latent_decode_any_kernel<float>, smem, what)) return rc;
+        launch_dependent(latent_decode_any_kernel<float>, grid, LD_WARPS * 32, smem, as_stream(stream), p);
+    } else {
+        if (int rc = allow_smem(latent_decode_any_kernel<__nv_bfloat16>, smem, what)) return rc;
+        launch_dependent(latent_decode_any_kernel<__nv_bfloat16>, grid, LD_WARPS * 32, smem, as_stream(stream), p);
+    }
+    return launch_status(what);
+}
+
+extern "C" int bn_latent_expand_out(const float* partial, const float* lse, int splits, const void* wuv, void* out, int64_t out_ld,
+                                    int B, int H, int vdim, int kv_rank, int dtype, bn_stream_t stream) {
+    const char* what = "bn_latent_expand_out";
+    if (!partial || !lse || !wuv || !out) return fail(BN_ERR_INVALID_ARG, "%s: null pointer", what);
+    if (B < 0 || H <= 0 || vdim <= 0 || kv_rank <= 0 || splits <= 0 || (dtype & ~1)) return fail(BN_ERR_INVALID_ARG, "%s: bad shape", what);
+    if (int rc = require_sm100()) return rc;
+    if (B == 0) return BN_OK;
+    const int kl = round8(kv_rank);
+    const unsigned grid = (unsigned)(((vdim + LO_V - 1) / LO_V) * H * ((B + LO_B - 1) / LO_B));
+    const size_t smem = (size_t)LO_B * kl * sizeof(float);
+    if (dtype == 0) {
+        if (int rc = allow_smem(latent_expand_out_kernel<float>, smem, what)) return rc;
+        launch_dependent(latent_expand_out_kernel<float>, grid, LO_WARPS * 32, smem, as_stream(stream), partial, lse, splits,
+                         static_cast<const float*>(wuv), static_cast<float*>(out), out_ld, B, H, vdim, kl);
+    } else {
+        if (int rc = allow_smem(latent_expand_out_kernel<__nv_bfloat16>, smem, what)) return rc;
+        launch_dependent(latent_expand_out_kernel<__nv_bfloat16>, grid, LO_WARPS * 32, smem, as_stream(stream), partial, lse, splits,
+                         static_cast<const __nv_bfloat16*>(wuv), static_cast<__nv_bfloat16*>(out), out_ld, B, H, vdim, kl);
+    }
+    return launch_status(what);
+}

@@ -97,3 +97,76 @@ class PagedKVCache:
             lse.data_ptr() if lse is not None else None, B, Hq, self.num_kv_heads, D, float(scale), self.theta,
             int(bool(rope_q)), int(max_seq_len), int(chunk_tokens), ws.ptr, ws.nbytes, _stream()))
         return out if out is not None else out_f32
+
+
+class LatentRingCache:
+    """What latent attention keeps of a sequence's last tokens: the normalised latent and the rotated key part that all
+    heads share.  A token's row is position % ring_tokens, so a sliding-window layer holds a constant amount per sequence
+    however long the sequence gets: ring_tokens is the window, rounded up to whole pages of PAGE_TOKENS.
+
+    ring[slot][ring_tokens][round8(kv_rank) | round8(rot_dim)], zeros behind the values of each part."""
+
+    def __init__(self, num_seqs: int, window: int, kv_rank: int, rot_dim: int, dtype=torch.bfloat16, device="cuda"):
+        from .ops import round8
+        self.num_seqs, self.window, self.kv_rank, self.rot_dim, self.dtype = num_seqs, window, kv_rank, rot_dim, dtype
+        self.kv_ld, self.rot_ld = round8(kv_rank), round8(rot_dim)
+        self.ring_tokens = (window + PAGE_TOKENS - 1) // PAGE_TOKENS * PAGE_TOKENS
+        self.ring = torch.zeros((num_seqs, self.ring_tokens, self.kv_ld + self.rot_ld), dtype=dtype, device=device)
+
+    def reset(self, slot: int) -> None:
+        """Nothing to clear: a row is read only for positions that the sequence itself has written."""
+
+    def tensors(self):
+        return [self.ring]
+
+    def gather(self, seq_ids, positions, n_old: int, latents: torch.Tensor, keys: torch.Tensor, rows_per_seq: int) -> None:
+        """The n_old tokens before `positions` to the first rows of each sequence's block of `latents` / `keys`."""
+        from .ops import _dt
+        _lib.check(_lib.load().bn_latent_gather(
+            self.ring.data_ptr(), self.ring_tokens, self.kv_rank, self.rot_dim, seq_ids.data_ptr(), positions.data_ptr(),
+            seq_ids.numel(), n_old, latents.data_ptr(), keys.data_ptr(), rows_per_seq, _dt(self.dtype), _stream()))
+
+
+class RecurrentState:
+    """What a Mamba-2 layer keeps of a sequence: its state matrices, fp32, and the convolution's last inputs in a ring
+    (the input of position p in row p % taps)."""
+
+    def __init__(self, num_seqs: int, heads: int, vdim: int, state: int, channels: int, taps: int, dtype=torch.bfloat16,
+                 device="cuda"):
+        self.num_seqs = num_seqs
+        self.state = torch.zeros((num_seqs, heads, vdim, state), dtype=torch.float32, device=device)
+        self.conv = torch.zeros((num_seqs, taps, channels), dtype=dtype, device=device)
+
+    def reset(self, slot: int) -> None:
+        self.state[slot].zero_()
+        self.conv[slot].zero_()
+
+    def tensors(self):
+        return [self.state, self.conv]
+
+
+class SequenceSlots:
+    """Which slot of the per-layer caches and states a live sequence has, and how many tokens it has seen.  A slot is reset
+    in every layer when it is taken, so what an earlier sequence left never reaches the next one."""
+
+    def __init__(self, num_seqs: int, states, device="cuda"):
+        self.num_seqs, self.states = num_seqs, list(states)
+        self.lens = torch.zeros((num_seqs,), dtype=torch.int32, device=device)
+        self.free = list(range(num_seqs - 1, -1, -1))
+
+    def acquire(self) -> int:
+        if not self.free:
+            raise RuntimeError(f"all {self.num_seqs} sequence slots are in use")
+        slot = self.free.pop()
+        self.lens[slot] = 0
+        for s in self.states:
+            s.reset(slot)
+        return slot
+
+    def release(self, slot: int) -> None:
+        if slot in self.free or not 0 <= slot < self.num_seqs:
+            raise RuntimeError(f"slot {slot} is not in use")
+        self.free.append(slot)
+
+    def tensors(self):
+        return [self.lens] + [t for s in self.states for t in s.tensors()]

@@ -1,4 +1,5 @@
-"""LLaMAModel on the bf16 path with a paged KV cache: `generate()` without whole-sequence recomputation.
+"""Generation over a cached model (`CausalLM`), and LLaMAModel on the bf16 path with a paged KV cache: `generate()` without
+whole-sequence recomputation.
 
 Mirror of mygrad/llama/llama_model.py (`LLaMAModel`: embed_tokens, layers, norm, lm_head; `__call__`, `generate`),
 composed from the rows of this package: device-side embedding gather, `LLaMADecoderLayerBF16` blocks for the prompt,
@@ -19,7 +20,82 @@ from .kv_cache import PAGE_TOKENS, PagedKVCache
 from .layers import LLaMAConfig, LLaMADecoderLayerBF16
 
 
-class LLaMAModelBF16:
+class CausalLM:
+    """Generation over a cached model: what every model family here shares.  A family supplies `config` (with
+    eos_token_id, or None), `prefill(prompts, max_len)` and `decode_step(token_ids, check)`, both returning fp32 logits of
+    one row per sequence, `seq_lens`, and `state_tensors()`, all that a decode step changes and a repeated step would not
+    put right by itself."""
+
+    ragged_prompts = False            # whether prompts of different lengths may share a batch
+
+    def argmax(self, logits: torch.Tensor) -> torch.Tensor:
+        rows, cols = logits.shape
+        out = torch.zeros((rows,), dtype=torch.int32, device="cuda")
+        _lib.check(_lib.load().bn_argmax_rows_f32(logits.data_ptr(), logits.stride(0), logits.stride(1), out.data_ptr(),
+                                                  rows, cols, torch.cuda.current_stream().cuda_stream))
+        return out
+
+    def capture_decode_step(self):
+        """Captures `decode_step` + argmax for the current batch into a CUDA graph: a step is tens of launches that
+        Python issues one by one (the host, not the GPU, bounds it); replayed from a graph they are one submission.
+        Returns step(token_ids) -> (logits, next_ids), both static buffers overwritten by the next call.  Lengths (and
+        states) advance inside the graph, so every replay is the next position."""
+        B = self.seq_lens.numel()
+        static_tok = torch.zeros((B,), dtype=torch.int32, device="cuda")
+        saved = [t.clone() for t in self.state_tensors()]
+        side = torch.cuda.Stream()
+        side.wait_stream(torch.cuda.current_stream())
+        with torch.cuda.stream(side):                      # warm-up outside the capture (workspaces, attributes)
+            self.decode_step(static_tok, check=False)
+        torch.cuda.current_stream().wait_stream(side)
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(graph):
+            logits = self.decode_step(static_tok, check=False)
+            nxt = self.argmax(logits)
+        torch.cuda.synchronize()
+        for t, v in zip(self.state_tensors(), saved):      # warm-up and capture must not count as positions
+            t.copy_(v)
+
+        def step(token_ids: torch.Tensor):
+            static_tok.copy_(token_ids)
+            graph.replay()
+            return logits, nxt
+
+        step.graph = graph
+        return step
+
+    def generate(self, input_ids, max_new_tokens: int = 50) -> List[List[int]]:
+        """Greedy `generate` (llama_model.py:112-168 with temperature -> 0): prompts (B, S) of equal length, or, where the
+        family takes them (`ragged_prompts`), a list of id lists of any lengths."""
+        rows = [np.asarray(r, dtype=np.int32).reshape(-1) for r in (input_ids if np.ndim(input_ids[0]) else [input_ids])]
+        if any(len(r) == 0 for r in rows):
+            raise ValueError("generate: empty prompt")
+        longest, B = max(len(r) for r in rows), len(rows)
+        if all(len(r) == longest for r in rows):
+            prompts = torch.from_numpy(np.ascontiguousarray(np.stack(rows))).cuda()
+        elif self.ragged_prompts:
+            prompts = rows
+        else:
+            raise ValueError("generate: this model takes prompts of equal length")
+        logits = self.prefill(prompts, longest + max_new_tokens)
+        out = [list(map(int, r)) for r in rows]
+        done = [False] * B
+        for n in range(max_new_tokens):
+            nxt = self.argmax(logits)
+            host = nxt.cpu().numpy()
+            for b in range(B):
+                if not done[b]:
+                    if self.config.eos_token_id is not None and int(host[b]) == self.config.eos_token_id:
+                        done[b] = True
+                    else:
+                        out[b].append(int(host[b]))
+            if all(done) or n + 1 == max_new_tokens:
+                break
+            logits = self.decode_step(nxt)
+        return out
+
+
+class LLaMAModelBF16(CausalLM):
     def __init__(self, config: LLaMAConfig, is_cuda: bool = True):
         if not is_cuda:
             raise RuntimeError("LLaMAModelBF16: only GPU implementation available")
@@ -52,13 +128,6 @@ class LLaMAModelBF16:
         """final norm of (residual + pending), lm_head: (rows, hidden) -> (rows, vocab) fp32"""
         _, normed = ops.add_rmsnorm_bf16(residual, pending, self.norm_weight, self.config.rms_norm_eps, want_sum=False)
         return ops.gemm_bf16_nt(normed, self.lm_head).float()
-
-    def argmax(self, logits: torch.Tensor) -> torch.Tensor:
-        rows, cols = logits.shape
-        out = torch.zeros((rows,), dtype=torch.int32, device="cuda")
-        _lib.check(_lib.load().bn_argmax_rows_f32(logits.data_ptr(), logits.stride(0), logits.stride(1), out.data_ptr(),
-                                                  rows, cols, torch.cuda.current_stream().cuda_stream))
-        return out
 
     # ----------------------------------------------------------------- forward
     def __call__(self, input_ids: torch.Tensor, position_offset: int = 0, use_causal_mask: bool = True) -> torch.Tensor:
@@ -134,56 +203,9 @@ class LLaMAModelBF16:
             h, pending = residual, layer.mlp(normed, few_rows=True)
         return self._logits(h, pending)
 
-    def capture_decode_step(self):
-        """Captures `decode_step` + argmax for the current batch into a CUDA graph: a step is about 30 launches that
-        Python issues one by one (the host, not the GPU, bounds it); replayed from a graph they are one submission.
-        Returns step(token_ids) -> (logits, next_ids), both static buffers overwritten by the next call.  The caches'
-        lengths advance inside the graph, so every replay is the next position."""
-        B = self.caches[0].num_seqs
-        static_tok = torch.zeros((B,), dtype=torch.int32, device="cuda")
-        saved = self.seq_lens.clone()
-        side = torch.cuda.Stream()
-        side.wait_stream(torch.cuda.current_stream())
-        with torch.cuda.stream(side):                      # warm-up outside the capture (workspaces, attributes)
-            self.decode_step(static_tok, check=False)
-        torch.cuda.current_stream().wait_stream(side)
-        graph = torch.cuda.CUDAGraph()
-        with torch.cuda.graph(graph):
-            logits = self.decode_step(static_tok, check=False)
-            nxt = self.argmax(logits)
-        torch.cuda.synchronize()
-        self.seq_lens.copy_(saved)                         # warm-up and capture must not count as positions
-
-        def step(token_ids: torch.Tensor):
-            static_tok.copy_(token_ids)
-            graph.replay()
-            return logits, nxt
-
-        step.graph = graph
-        return step
-
-    def generate(self, input_ids: np.ndarray, max_new_tokens: int = 50) -> List[List[int]]:
-        """Greedy `generate` (llama_model.py:112-168 with temperature -> 0): prompts (B, S) of equal length."""
-        ids = torch.from_numpy(np.ascontiguousarray(input_ids, dtype=np.int32)).cuda()
-        if ids.dim() == 1:
-            ids = ids[None]
-        B, S = ids.shape
-        logits = self.prefill(ids, S + max_new_tokens)
-        out = [list(map(int, row)) for row in ids.cpu().numpy()]
-        done = [False] * B
-        for _ in range(max_new_tokens):
-            nxt = self.argmax(logits)
-            host = nxt.cpu().numpy()
-            for b in range(B):
-                if not done[b]:
-                    if int(host[b]) == self.config.eos_token_id:
-                        done[b] = True
-                    else:
-                        out[b].append(int(host[b]))
-            if all(done):
-                break
-            logits = self.decode_step(nxt)
-        return out
+    def state_tensors(self):
+        """A step that ran by mistake is undone by its lengths alone: what it appended lies behind every valid token."""
+        return [self.seq_lens]
 
     def status(self) -> None:
         """Raises if any kernel of the model gave up a bounded wait since the last check (attention scratch of every
@@ -191,6 +213,24 @@ class LLaMAModelBF16:
         for c in self.caches or []:
             c.status()
         ops.gemm_status()
+
+    def load_weights(self, w) -> None:
+        """Weights from a checkpoint (checkpoint.Weights), named as the reference's attributes and stored (out, in)."""
+        cfg = self.config
+        H, inter, kv = cfg.hidden_size, cfg.intermediate_size, cfg.num_key_value_heads * cfg.head_dim
+        put = lambda name, *shape: w(name, *shape).to(device="cuda", dtype=torch.bfloat16).contiguous()      # noqa: E731
+        self.embed_tokens = w("embed_tokens", cfg.vocab_size, H).to(device="cuda", dtype=torch.float32).contiguous()
+        for i, layer in enumerate(self.layers):
+            p, at, mlp = f"layers.{i}.", layer.self_attn, layer.mlp
+            at.q_proj, at.k_proj = put(p + "self_attn.q_proj", H, H), put(p + "self_attn.k_proj", kv, H)
+            at.v_proj, at.o_proj = put(p + "self_attn.v_proj", kv, H), put(p + "self_attn.o_proj", H, H)
+            mlp.gate_proj, mlp.up_proj = put(p + "mlp.gate_proj", inter, H), put(p + "mlp.up_proj", inter, H)
+            mlp.down_proj = put(p + "mlp.down_proj", H, inter)
+            mlp._gate_up = ops.pack_gate_up(mlp.gate_proj, mlp.up_proj)
+            layer.input_layernorm_weight = put(p + "input_layernorm", H)
+            layer.post_attention_layernorm_weight = put(p + "post_attention_layernorm", H)
+        self.norm_weight = put("norm", H)
+        self.lm_head = put("lm_head", cfg.vocab_size, H)
 
     def parameters(self):
         p = [self.embed_tokens]

@@ -159,6 +159,15 @@ def gemm_bf16_nt(a: torch.Tensor, bt: torch.Tensor, *, out: Optional[torch.Tenso
 _small_m_ws = {}
 
 
+def _small_m_scratch(device, M: int, N: int, K: int):
+    n = int(_lib.load().bn_gemm_bf16_nt_small_m_workspace_bytes(M, N, K))
+    key = (device, n)
+    ws = _small_m_ws.get(key)
+    if ws is None:
+        ws = _small_m_ws[key] = torch.empty(max(n, 16), dtype=torch.uint8, device=device)
+    return ws, n
+
+
 def gemm_bf16_nt_small_m(a: torch.Tensor, bt: torch.Tensor, *, out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """a (M,K) @ bt (N,K)^T for few rows (a decode step: one token per sequence): the weight stream is spread over
     all SMs (64-wide N tiles, K split, partial sums added in a fixed order).  The fp32 scratch is kept per
@@ -169,23 +178,29 @@ def gemm_bf16_nt_small_m(a: torch.Tensor, bt: torch.Tensor, *, out: Optional[tor
         raise RuntimeError(f"MatMul: inner dimensions mismatch {tuple(a.shape)} x {tuple(bt.shape)}^T")
     M, K = a.shape
     N = bt.shape[0]
-    lib = _lib.load()
-    n = int(lib.bn_gemm_bf16_nt_small_m_workspace_bytes(M, N, K))
-    key = (a.device, n)
-    ws = _small_m_ws.get(key)
-    if ws is None:
-        ws = _small_m_ws[key] = torch.empty(max(n, 16), dtype=torch.uint8, device=a.device)
+    ws, n = _small_m_scratch(a.device, M, N, K)
     if out is None:
         out = torch.empty((M, N), dtype=torch.bfloat16, device=a.device)
     _need(out, torch.bfloat16, "gemm_bf16_nt_small_m(out)")
-    _lib.check(lib.bn_gemm_bf16_nt_small_m(a.data_ptr(), bt.data_ptr(), out.data_ptr(), M, N, K, ws.data_ptr(), n,
-                                           _gemm_error_ptr(a.device, None), _stream()))
+    _lib.check(_lib.load().bn_gemm_bf16_nt_small_m(a.data_ptr(), bt.data_ptr(), out.data_ptr(), M, N, K, ws.data_ptr(), n,
+                                                   _gemm_error_ptr(a.device, None), _stream()))
     return out
 
 
 def skinny_ok(rows: int, n_out: int, k: int) -> bool:
+    """Shapes the weight-streaming kernel for at most 16 rows was tuned for."""
+    return skinny_any_k(rows, n_out, k) and k % 256 == 0
+
+
+def skinny_any_k(rows: int, n_out: int, k: int) -> bool:
     """Shapes the weight-streaming kernel for at most 16 rows takes."""
-    return 0 < rows <= 16 and n_out % 8 == 0 and k % 256 == 0 and 0 < k <= 8192
+    return 0 < rows <= 16 and n_out % 8 == 0 and k % 8 == 0 and 0 < k <= 8192
+
+
+def small_m_ok(rows: int, n_out: int) -> bool:
+    """Few rows and too few 256-wide output tiles to occupy the GPU (measured cross-over: fewer than half as many tiles as
+    SMs): the split-K form."""
+    return rows <= 128 and (n_out + 255) // 256 < 74
 
 
 def gemm_bf16_nt_skinny(x: torch.Tensor, weight_t: torch.Tensor, splits: Optional[Tuple[int, ...]] = None):
@@ -246,12 +261,11 @@ def gemm_swiglu_bf16_nt_skinny(x: torch.Tensor, gate_t: torch.Tensor, up_t: torc
 
 def linear_bf16(x: torch.Tensor, weight_t: torch.Tensor) -> torch.Tensor:
     """x (rows, in) @ weight_t (out, in)^T, choosing the kernel by shape: at most 16 rows -> the weight-streaming
-    kernel; few rows and too few 256-wide output tiles to occupy the GPU (measured cross-over: fewer than half as many
-    tiles as SMs) -> the split-K small-M form; otherwise the large-tile kernel."""
+    kernel; few rows and few output tiles -> the split-K small-M form; otherwise the large-tile kernel."""
     rows, n_out = x.shape[0], weight_t.shape[0]
-    if skinny_ok(rows, n_out, x.shape[1]):
+    if skinny_any_k(rows, n_out, x.shape[1]):
         return gemm_bf16_nt_skinny(x, weight_t)
-    if rows <= 128 and (n_out + 255) // 256 < 74:
+    if small_m_ok(rows, n_out):
         return gemm_bf16_nt_small_m(x, weight_t)
     return gemm_bf16_nt(x, weight_t)
 
@@ -390,3 +404,219 @@ def lse_combine(outs: torch.Tensor, lses: torch.Tensor, *, out_dtype=torch.float
                                                o32.data_ptr() if o32 is not None else None,
                                                o16.data_ptr() if o16 is not None else None, lse.data_ptr(), _stream()))
     return (o32 if o32 is not None else o16), lse
+
+
+# ---------------------------------------------------------------------------------------------------------------------
+# Operators that exist in fp32 and in bf16 (dtype of the activations decides); row strides may exceed the row, so that
+# rows of any width start on 16-byte boundaries.
+# ---------------------------------------------------------------------------------------------------------------------
+ACTIVATIONS = {"none": _lib.BN_ACT_NONE, "silu": _lib.BN_ACT_SILU, "gelu_tanh": _lib.BN_ACT_GELU_TANH}
+
+
+def round8(n: int) -> int:
+    return (n + 7) // 8 * 8
+
+
+def _dt(dtype) -> int:
+    if dtype not in (torch.float32, torch.bfloat16):
+        raise RuntimeError(f"dtype {dtype}: float32 or bfloat16")
+    return 0 if dtype == torch.float32 else 1
+
+
+def _ptr(t: Optional[torch.Tensor]):
+    return None if t is None else t.data_ptr()
+
+
+def _rows(t: torch.Tensor, what: str) -> torch.Tensor:
+    if not t.is_cuda:
+        raise RuntimeError(f"{what}: only GPU implementation available")
+    if t.dim() != 2 or t.stride(1) != 1:
+        raise RuntimeError(f"{what}: expected rows of contiguous elements")
+    return t
+
+
+class Linear:
+    """y = x W^T for a weight (out, in): bf16 on the tensor cores, or true fp32 (`bn_mm_f32`).  Both sizes are rounded up to
+    multiples of 8 with zeros, so x may be passed with its padding columns (which must be finite) and y has them."""
+
+    def __init__(self, weight: torch.Tensor, dtype, device="cuda"):
+        self.out_features, self.in_features = weight.shape
+        self.dtype = dtype
+        self.n, self.k = round8(self.out_features), round8(self.in_features)
+        self.weight = torch.zeros((self.n, self.k), dtype=dtype, device=device)
+        self.weight[:self.out_features, :self.in_features] = weight.to(device)
+
+    def _operand(self, x: torch.Tensor) -> torch.Tensor:
+        _rows(x, "linear(x)")
+        if x.dtype != self.dtype:
+            raise RuntimeError(f"linear: {x.dtype} rows for a {self.dtype} weight")
+        if x.shape[1] == self.k and x.stride(0) == self.k:
+            return x
+        if x.shape[1] not in (self.k, self.in_features):
+            raise RuntimeError(f"MatMul: inner dimensions mismatch {tuple(x.shape)} x {tuple(self.weight.shape)}^T")
+        out = torch.zeros((x.shape[0], self.k), dtype=x.dtype, device=x.device)
+        out[:, :x.shape[1]] = x
+        return out
+
+    def _mm_f32(self, x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+        w = self.weight
+        _lib.check(_lib.load().bn_mm_f32(x.data_ptr(), x.stride(0), 1, w.data_ptr(), 1, w.stride(0), out.data_ptr(),
+                                         out.stride(0), 1, x.shape[0], self.k, self.n, _stream()))
+        return out
+
+    def __call__(self, x: torch.Tensor, f32_out: bool = False) -> torch.Tensor:
+        """(rows, in) -> (rows, out rounded up to a multiple of 8); `f32_out`: the fp32 accumulators themselves."""
+        x = self._operand(x)
+        rows = x.shape[0]
+        if self.dtype == torch.float32:
+            return self._mm_f32(x, torch.empty((rows, self.n), dtype=torch.float32, device=x.device))
+        if not f32_out:
+            return linear_bf16(x, self.weight)
+        out = torch.empty((rows, self.n), dtype=torch.float32, device=x.device)
+        lib = _lib.load()
+        if skinny_any_k(rows, self.n, self.k):
+            _lib.check(lib.bn_gemm_bf16_nt_skinny_f32(x.data_ptr(), self.weight.data_ptr(), rows, self.n, self.k,
+                                                      out.data_ptr(), _stream()))
+        elif small_m_ok(rows, self.n):
+            ws, n = _small_m_scratch(x.device, rows, self.n, self.k)
+            _lib.check(lib.bn_gemm_bf16_nt_small_m_f32(x.data_ptr(), self.weight.data_ptr(), out.data_ptr(), rows, self.n,
+                                                       self.k, ws.data_ptr(), n, _gemm_error_ptr(x.device, None), _stream()))
+        else:
+            _lib.check(lib.bn_gemm_bf16_nt_f32(x.data_ptr(), self.weight.data_ptr(), out.data_ptr(), rows, self.n, self.k,
+                                               _gemm_error_ptr(x.device, None), _stream()))
+        return out
+
+    def act_mul(self, x: torch.Tensor, mul: torch.Tensor, act: str) -> torch.Tensor:
+        """act(x W^T) * mul, mul (rows, >= out rounded up) with any row stride that is a multiple of 8."""
+        x = self._operand(x)
+        rows, a = x.shape[0], ACTIVATIONS[act]
+        _rows(mul, "act_mul(mul)")
+        if mul.shape[0] != rows or mul.shape[1] < self.n or mul.dtype != self.dtype:
+            raise RuntimeError("act_mul: the factor must have the product's rows, columns and dtype")
+        out = torch.empty((rows, self.n), dtype=self.dtype, device=x.device)
+        lib = _lib.load()
+        if self.dtype == torch.float32:
+            self._mm_f32(x, out)
+            _lib.check(lib.bn_act_mul_f32(out.data_ptr(), self.n, mul.data_ptr(), mul.stride(0), out.data_ptr(), self.n, rows,
+                                          self.n, a, _stream()))
+        elif skinny_any_k(rows, self.n, self.k):
+            _lib.check(lib.bn_gemm_act_mul_bf16_nt_skinny(x.data_ptr(), self.weight.data_ptr(), mul.data_ptr(), mul.stride(0),
+                                                          out.data_ptr(), rows, self.n, self.k, a, _stream()))
+        elif small_m_ok(rows, self.n):
+            ws, n = _small_m_scratch(x.device, rows, self.n, self.k)
+            _lib.check(lib.bn_gemm_act_mul_bf16_nt_small_m(x.data_ptr(), self.weight.data_ptr(), mul.data_ptr(), mul.stride(0),
+                                                           out.data_ptr(), rows, self.n, self.k, a, ws.data_ptr(), n,
+                                                           _gemm_error_ptr(x.device, None), _stream()))
+        else:
+            _lib.check(lib.bn_gemm_act_mul_bf16_nt(x.data_ptr(), self.weight.data_ptr(), mul.data_ptr(), mul.stride(0),
+                                                   out.data_ptr(), rows, self.n, self.k, a, _gemm_error_ptr(x.device, None),
+                                                   _stream()))
+        return out
+
+
+class GatedLinear:
+    """act(x Wgate^T) * (x Wup^T): one launch in bf16, three in fp32."""
+
+    def __init__(self, gate: torch.Tensor, up: torch.Tensor, act: str, dtype, device="cuda"):
+        if gate.shape != up.shape:
+            raise RuntimeError("gate and up weights must have the same (inter, K) shape")
+        self.act, self.dtype = act, dtype
+        self.gate, self.up = Linear(gate, dtype, device), Linear(up, dtype, device)
+        self.inter, self.k = self.gate.n, self.gate.k
+        self._packed = pack_gate_up(self.gate.weight, self.up.weight) if dtype == torch.bfloat16 else None
+
+    def __call__(self, x: torch.Tensor) -> torch.Tensor:
+        x = self.gate._operand(x)
+        rows, a = x.shape[0], ACTIVATIONS[self.act]
+        out = torch.empty((rows, self.inter), dtype=self.dtype, device=x.device)
+        lib = _lib.load()
+        if self.dtype == torch.float32:
+            g, u = self.gate(x), self.up(x)
+            _lib.check(lib.bn_act_mul_f32(g.data_ptr(), g.stride(0), u.data_ptr(), u.stride(0), out.data_ptr(), self.inter, rows,
+                                          self.inter, a, _stream()))
+        elif skinny_any_k(rows, self.inter, self.k):
+            _lib.check(lib.bn_gemm_glu_bf16_nt_skinny(x.data_ptr(), self.gate.weight.data_ptr(), self.up.weight.data_ptr(),
+                                                      out.data_ptr(), rows, self.inter, self.k, a, _stream()))
+        else:
+            _lib.check(lib.bn_gemm_glu_bf16_nt(x.data_ptr(), self._packed.data_ptr(), out.data_ptr(), rows, self.inter, self.k, a,
+                                               _gemm_error_ptr(x.device, None), _stream()))
+        return out
+
+
+def embedding_rows(table: torch.Tensor, ids: torch.Tensor, *, out_f32: Optional[torch.Tensor] = None,
+                   out_bf16: Optional[torch.Tensor] = None, error_word: Optional[torch.Tensor] = None) -> None:
+    """Rows `ids` (int32) of an fp32 or bf16 table into out_f32 and/or (bf16 tables) out_bf16; an id outside the table gives
+    a zero row and raises error_word."""
+    _rows(table, "embedding_rows(table)")
+    _need(ids, torch.int32, "embedding_rows(ids)")
+    n, (vocab, hidden) = ids.numel(), table.shape
+    if table.dtype == torch.float32:
+        _lib.check(_lib.load().bn_embedding_gather_f32(table.data_ptr(), table.stride(0), ids.data_ptr(), out_f32.data_ptr(),
+                                                       out_f32.stride(0), n, hidden, vocab, _ptr(error_word), _stream()))
+    else:
+        _lib.check(_lib.load().bn_embedding_gather_bf16(
+            table.data_ptr(), table.stride(0), ids.data_ptr(), _ptr(out_f32), 0 if out_f32 is None else out_f32.stride(0),
+            _ptr(out_bf16), 0 if out_bf16 is None else out_bf16.stride(0), n, hidden, vocab, _ptr(error_word), _stream()))
+
+
+class NormWeight:
+    """Weight and bias of a layer norm (bias given) or an RMS norm, fp32 on the GPU."""
+
+    def __init__(self, weight: torch.Tensor, bias: Optional[torch.Tensor], eps: float, device="cuda"):
+        self.weight = weight.to(device=device, dtype=torch.float32).contiguous()
+        self.bias = None if bias is None else bias.to(device=device, dtype=torch.float32).contiguous()
+        self.center = bias is not None
+        self.eps = float(eps)
+
+
+class Pending:
+    """A sublayer's output that has not been added to the residual stream yet: the next residual_norm adds it, as it is or
+    RMS-normed with a weight of its own."""
+
+    def __init__(self, rows: torch.Tensor, norm: Optional[NormWeight] = None):
+        self.rows, self.norm = _rows(rows, "pending"), norm
+
+    def select(self, index: torch.Tensor) -> "Pending":
+        return Pending(self.rows.index_select(0, index), self.norm)
+
+
+def residual_norm(x: Optional[torch.Tensor], pending: Optional[Pending], dtype, hidden: int, *, row: Optional[torch.Tensor] = None,
+                  norm: Optional[NormWeight] = None, keep_sum: bool = True, cast: Optional[torch.Tensor] = None,
+                  lo_offset: int = 0):
+    """x (rows, hidden) fp32 + pending + row -> (the fp32 sum, its norm in `dtype`); either may be None when not asked for.
+    `cast` receives the sum rounded to `dtype` (and, lo_offset columns on, the remainder of that rounding)."""
+    src = x if x is not None else pending.rows
+    rows = src.shape[0]
+    dev = src.device
+    if x is not None:
+        _need(x, torch.float32, "residual_norm(x)")
+    d = None if pending is None else pending.rows
+    dn = None if pending is None else pending.norm
+    changed = d is not None or row is not None
+    total = torch.empty((rows, hidden), dtype=torch.float32, device=dev) if keep_sum and changed else None
+    y = None
+    if norm is not None:
+        y = torch.empty((rows, round8(hidden)), dtype=dtype, device=dev)
+        if y.shape[1] != hidden:
+            y[:, hidden:] = 0
+    if total is None and y is None and cast is None:
+        return x, None
+    _lib.check(_lib.load().bn_residual_norm(
+        _ptr(x), _ptr(d), 0 if d is None else d.stride(0), 1 if d is not None and d.dtype == torch.bfloat16 else 0,
+        None if dn is None else dn.weight.data_ptr(), 0.0 if dn is None else dn.eps, _ptr(row), _ptr(total), _ptr(cast),
+        0 if cast is None else cast.stride(0), lo_offset, None if norm is None else norm.weight.data_ptr(),
+        None if norm is None or norm.bias is None else norm.bias.data_ptr(), _ptr(y), 0 if y is None else y.stride(0),
+        int(norm is not None and norm.center), _dt(dtype), rows, hidden, 0.0 if norm is None else norm.eps, _stream()))
+    return (total if changed else x), y
+
+
+def rotation_frequencies(rot_dim: int, base: float, device="cuda") -> torch.Tensor:
+    """base ** (-2 i / rot_dim) for the rot_dim / 2 pairs, fp64."""
+    i = torch.arange(0, rot_dim, 2, dtype=torch.float64)
+    return torch.pow(torch.tensor(float(base), dtype=torch.float64), -i / rot_dim).to(device)
+
+
+def status_word(device) -> torch.Tensor:
+    """The int32 per device that launches report a bounded wait that ran out into (read by `gemm_status`)."""
+    _gemm_error_ptr(device, None)
+    return _gemm_err[torch.device(device).index if torch.device(device).index is not None else torch.cuda.current_device()]

@@ -52,6 +52,12 @@ extern "C" {
 /* tokens per KV-cache page */
 #define BN_PAGE_TOKENS 16
 
+/* activations of the fused products */
+#define BN_ACT_NONE 0
+#define BN_ACT_SILU 1
+#define BN_ACT_GELU_TANH 2
+#define BN_ACT_LAST 2
+
 typedef void* bn_stream_t; /* a cudaStream_t */
 
 /* exported symbol (the library is built with hidden default visibility) */
@@ -365,6 +371,109 @@ BN_API int bn_exchange_combine(bn_exchange_t* x, const float* partial, float* ou
                                bn_stream_t stream);
 BN_API int bn_exchange_status(bn_exchange_t* x, bn_stream_t stream);
 BN_API void bn_exchange_destroy(bn_exchange_t* x);
+
+/* ------------------------------------------------------------------------
+ * Further forms of the products (operands and limits as their plain forms above): the gated linear unit with a choice
+ * of activation, an fp32 result, and act(a bt^T) * mul with `mul` (M, mul_ld) bf16.
+ * ------------------------------------------------------------------------ */
+BN_API int bn_gemm_glu_bf16_nt(const void* x, const void* gate_up_t, void* h, int M, int inter, int K, int act,
+                               int* error_word, bn_stream_t stream);
+BN_API int bn_gemm_bf16_nt_f32(const void* a, const void* bt, float* c, int M, int N, int K, int* error_word,
+                               bn_stream_t stream);
+BN_API int bn_gemm_act_mul_bf16_nt(const void* a, const void* bt, const void* mul, int64_t mul_ld, void* c, int M, int N,
+                                   int K, int act, int* error_word, bn_stream_t stream);
+BN_API int bn_gemm_bf16_nt_small_m_f32(const void* a, const void* bt, float* c, int M, int N, int K, void* workspace,
+                                       size_t workspace_bytes, int* error_word, bn_stream_t stream);
+BN_API int bn_gemm_act_mul_bf16_nt_small_m(const void* a, const void* bt, const void* mul, int64_t mul_ld, void* c, int M,
+                                           int N, int K, int act, void* workspace, size_t workspace_bytes,
+                                           int* error_word, bn_stream_t stream);
+BN_API int bn_gemm_glu_bf16_nt_skinny(const void* x, const void* gate_t, const void* up_t, void* h, int M, int inter, int K,
+                                      int act, bn_stream_t stream);
+BN_API int bn_gemm_bf16_nt_skinny_f32(const void* a, const void* bt, int M, int N, int K, float* out, bn_stream_t stream);
+BN_API int bn_gemm_act_mul_bf16_nt_skinny(const void* a, const void* bt, const void* mul, int64_t mul_ld, void* out, int M,
+                                          int N, int K, int act, bn_stream_t stream);
+BN_API int bn_act_mul_f32(const float* a, int64_t a_ld, const float* b, int64_t b_ld, float* out, int64_t out_ld, int rows,
+                          int cols, int act, bn_stream_t stream);
+BN_API int bn_embedding_gather_bf16(const void* table, int64_t table_rs, const uint32_t* ids, float* out_f32,
+                                    int64_t rs_f32, void* out_bf16, int64_t rs_bf16, int n_ids, int hidden, int vocab,
+                                    int* error_word, bn_stream_t stream);
+
+/* ------------------------------------------------------------------------
+ * The fp32 residual stream.  dtype of an argument below: 0 = fp32, 1 = bf16; `dtype` is that of cast and y.
+ *   d = delta, or its RMS norm with weight delta_w;  x' = x + d + row (each optional)
+ *   x_out = x' (fp32);  cast = x' rounded, and lo_offset columns on (0: not wanted) the rounding's remainder, rounded
+ *   y = layer norm (center) or RMS norm of x' with weight w and bias b (w null: not wanted)
+ * ------------------------------------------------------------------------ */
+BN_API int bn_residual_norm(const float* x, const void* delta, int64_t delta_ld, int delta_dtype, const float* delta_w,
+                            float delta_eps, const float* row, float* x_out, void* cast, int64_t cast_ld, int lo_offset,
+                            const float* w, const float* b, void* y, int64_t y_ld, int center, int dtype, int rows,
+                            int hidden, float eps, bn_stream_t stream);
+
+/* ------------------------------------------------------------------------
+ * Latent attention with a sliding window (fp32 or bf16).  Rows are B sequences x S new tokens; sequence b occupies slot
+ * seq_ids[b] (null: b) and its first new token has position positions[b].  freq: rot / 2 rotation frequencies in fp64;
+ * pair (2i, 2i+1) of a rotated part turns by position * freq[i].  A latent row has round8(kv_rank) columns, a rotated
+ * key part round8(rot), zeros behind the values; ring[slot][ring_tokens][latent | rotated part], ring_tokens >= window,
+ * holds the token of position p in row p % ring_tokens.
+ * ------------------------------------------------------------------------ */
+/* proj row [q_rank | kv_rank | rot] -> cq = normalised query latent (cq_ld columns, zeros behind q_rank); latent and
+ * rotated part to row b * rows_per_seq + row_offset + s of c / krot (may be null) and into the ring (may be null) */
+BN_API int bn_latent_prep(const void* proj, int64_t proj_ld, const float* q_norm, const float* kv_norm, float eps,
+                          const double* freq, const int32_t* seq_ids, const int32_t* positions, int B, int S, int q_rank,
+                          int kv_rank, int rot, void* cq, int64_t cq_ld, void* c, void* krot, int rows_per_seq,
+                          int row_offset, void* ring, int ring_tokens, int dtype, bn_stream_t stream);
+/* the n_old tokens before positions[b], from the ring to rows b * rows_per_seq + 0 .. n_old - 1 of c and krot */
+BN_API int bn_latent_gather(const void* ring, int ring_tokens, int kv_rank, int rot, const int32_t* seq_ids,
+                            const int32_t* positions, int B, int n_old, void* c, void* krot, int rows_per_seq, int dtype,
+                            bn_stream_t stream);
+/* rotates the last rot of each head's dim + rot columns of q (B*S, q_ld), in place */
+BN_API int bn_rope_heads(void* q, int64_t q_ld, int B, int S, int H, int dim, int rot, const double* freq,
+                         const int32_t* positions, int dtype, bn_stream_t stream);
+/* softmax(scale (q_unrotated k + q_rotated krot)) v over the `window` keys that end at the query's own; key row
+ * b * rows_per_seq + n_old + s belongs to query s of sequence b.  k (rows, H * dim) and v (rows, H * vdim) share the row
+ * stride kv_ld.  error_word (may be null) receives BN_ERR_TIMEOUT if a bounded wait runs out. */
+BN_API int bn_attn_window(const void* q, int64_t q_ld, const void* k, const void* v, int64_t kv_ld, const void* krot,
+                          int64_t krot_ld, void* out, int64_t out_ld, int B, int S, int n_old, int rows_per_seq, int H,
+                          int dim, int rot, int vdim, int window, float scale, int* error_word, int dtype,
+                          bn_stream_t stream);
+/* one new token per row: q (B, q_ld) -> q_abs (B, H, latent | rotated part), the query against cached latents.
+ * wuk (H * dim, round8(kv_rank)) */
+BN_API int bn_latent_absorb_q(const void* q, int64_t q_ld, const void* wuk, const double* freq, const int32_t* positions,
+                              void* q_abs, int B, int H, int dim, int rot, int kv_rank, int dtype, bn_stream_t stream);
+/* how many parts bn_latent_decode cuts a window into (a size, 0 for a bad shape): partial holds
+ * B * H * splits * round8(kv_rank) floats and lse B * H * splits */
+BN_API int bn_latent_decode_splits(int B, int H, int kv_rank, int rot, int window, int dtype);
+BN_API int bn_latent_decode(const void* q_abs, const void* ring, int ring_tokens, const int32_t* seq_ids,
+                            const int32_t* positions, float* partial, float* lse, int splits, int B, int H, int kv_rank,
+                            int rot, int window, float scale, int dtype, bn_stream_t stream);
+/* merges the parts and expands the latent sum: out (B, out_ld), column h * vdim + v; wuv (H * vdim, round8(kv_rank)) */
+BN_API int bn_latent_expand_out(const float* partial, const float* lse, int splits, const void* wuv, void* out,
+                                int64_t out_ld, int B, int H, int vdim, int kv_rank, int dtype, bn_stream_t stream);
+
+/* ------------------------------------------------------------------------
+ * Mamba-2 mixer (fp32 or bf16).  proj row [z: H*P | x: H*P | B: G*N | C: G*N | dt: H]; conv_w [channels][taps], last tap
+ * the current token's; ring[slot][taps][channels] the last inputs of the convolution (position p in row p % taps);
+ * state[slot][H][P][N] fp32, zero for a new sequence.  taps <= 16, N <= 512.
+ * ------------------------------------------------------------------------ */
+/* convolution + silu -> xbc (B*S, xbc_ld) = [x | B | C]; dt = softplus(dt + dt_bias), a = -exp(a_log) dt, (B*S, H) each;
+ * updates the ring */
+BN_API int bn_mamba2_conv(const void* proj, int64_t proj_ld, const float* conv_w, const float* conv_b,
+                          const float* dt_bias, const float* a_log, void* ring, const int32_t* seq_ids,
+                          const int32_t* positions, int B, int S, int H, int P, int G, int N, int taps, void* xbc,
+                          int64_t xbc_ld, float* dt, float* a, int dtype, bn_stream_t stream);
+/* the recurrence over S tokens from the slot's state, which it advances: y (B*S, y_ld) = S^T C + D x */
+BN_API int bn_ssm_scan(const void* xbc, int64_t xbc_ld, const float* dt, const float* a, const float* D, float* state,
+                       const int32_t* seq_ids, int B, int S, int H, int P, int G, int N, void* y, int64_t y_ld, int dtype,
+                       bn_stream_t stream);
+/* one new token per row, everything between the two products but the norm: gated (B, H*P) = (y + D x) silu(z) */
+BN_API int bn_mamba2_step(const void* proj, int64_t proj_ld, const float* conv_w, const float* conv_b,
+                          const float* dt_bias, const float* a_log, const float* D, void* ring, float* state,
+                          const int32_t* seq_ids, const int32_t* positions, int B, int H, int P, int G, int N, int taps,
+                          float* gated, int dtype, bn_stream_t stream);
+/* out = w * RMS norm, in `groups` equal parts, of y * silu(z) (z null: of y) */
+BN_API int bn_gated_group_norm(const void* y, int64_t y_ld, int y_dtype, const void* z, int64_t z_ld, const float* w,
+                               void* out, int64_t out_ld, int rows, int width, int groups, float eps, int dtype,
+                               bn_stream_t stream);
 
 #ifdef __cplusplus
 }
