@@ -82,7 +82,7 @@ SIGNATURES = {
                             _i, _p]),
     "bn_latent_absorb_q": (_i, [_p, _i64, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _p]),
     "bn_latent_decode_splits": (_i, [_i, _i, _i, _i, _i, _i]),
-    "bn_latent_decode": (_i, [_p, _p, _i, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _f, _i, _p]),
+    "bn_latent_decode": (_i, [_p, _p, _i, _i, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _f, _i, _p]),
     "bn_latent_expand_out": (_i, [_p, _p, _i, _p, _p, _i64, _i, _i, _i, _i, _i, _p]),
     "bn_mamba2_conv": (_i, [_p, _i64, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _i, _p, _i64, _p, _p, _i,
                             _p]),

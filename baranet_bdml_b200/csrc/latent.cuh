@@ -22,7 +22,7 @@ struct LatentDecodeParams {
     const void *q_abs, *ring;
     const int32_t *seq_ids, *positions;
     float *partial, *lse;             // [B][H][splits][kv_ld], [B][H][splits]
-    int B, H, kv_ld, rot_ld, ring_tokens, window, splits;
+    int B, H, kv_ld, rot_ld, num_slots, ring_tokens, window, splits;
     float scale;
 };
 

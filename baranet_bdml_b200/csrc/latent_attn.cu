@@ -214,7 +214,8 @@ attn_window_kernel(const AttnWindowParams p) {
 }
 
 // ---------------------------------------------------------------------------------------------------------------
-// One new token per row: the query moved into latent space.  Block (n tile, head); the last n tile is the rotation.
+// One new token per row: the query moved into latent space.  Block (row group, n tile, head); the last n tile is the
+// rotation.
 //   q_abs[b][h][0..kv_ld) = sum_i q[b][h][i] W_uk[h * dim + i][:]      q_abs[b][h][kv_ld..) = rotated part
 // ---------------------------------------------------------------------------------------------------------------
 constexpr int LA_N = 128, LA_B = 8;
@@ -223,14 +224,16 @@ template <typename T>
 __global__ void __launch_bounds__(LA_N)
 latent_absorb_kernel(const T* q, int64_t q_ld, const T* wuk, const double* freq, const int32_t* positions, T* q_abs, int B, int H,
                      int dim, int rot, int kv_ld, int rot_ld) {
-    extern __shared__ float q_smem[];                   // [LA_B][dim]
+    extern __shared__ __align__(16) float qa_smem[];    // [dim][LA_B]
+    float* q_smem = qa_smem;
     ptx::grid_dependency_wait();
     ptx::grid_launch_dependents();
-    const int h = blockIdx.x % H, tile = blockIdx.x / H, n_tiles = (kv_ld + LA_N - 1) / LA_N;
+    const int n_tiles = (kv_ld + LA_N - 1) / LA_N, h = blockIdx.x % H, tile = blockIdx.x / H % (n_tiles + 1);
+    const int b0 = blockIdx.x / (H * (n_tiles + 1)) * LA_B, nb = min(LA_B, B - b0);
     const int width = kv_ld + rot_ld;
     if (tile == n_tiles) {
-        for (int i = threadIdx.x; i < B * (rot_ld / 2); i += LA_N) {
-            const int b = i / (rot_ld / 2), j = i % (rot_ld / 2);
+        for (int i = threadIdx.x; i < nb * (rot_ld / 2); i += LA_N) {
+            const int b = b0 + i / (rot_ld / 2), j = i % (rot_ld / 2);
             T lo = from_f<T>(0.f), hi = lo;
             if (2 * j < rot) {
                 const T* x = q + b * q_ld + h * (dim + rot) + dim + 2 * j;
@@ -247,30 +250,28 @@ latent_absorb_kernel(const T* q, int64_t q_ld, const T* wuk, const double* freq,
         return;
     }
     const int n = tile * LA_N + threadIdx.x;
-    for (int b0 = 0; b0 < B; b0 += LA_B) {
-        const int nb = min(LA_B, B - b0);
-        __syncthreads();
-        for (int i = threadIdx.x; i < LA_B * dim; i += LA_N) {
-            const int b = i / dim, e = i - b * dim;
-            q_smem[i] = b < nb ? to_f(q[(b0 + b) * q_ld + h * (dim + rot) + e]) : 0.f;
-        }
-        __syncthreads();
-        if (n < kv_ld) {
-            float acc[LA_B];
-#pragma unroll
-            for (int b = 0; b < LA_B; ++b) acc[b] = 0.f;
-            const T* w = wuk + (int64_t)h * dim * kv_ld + n;
-#pragma unroll 8
-            for (int e = 0; e < dim; ++e) {
-                const float wv = to_f(w[(int64_t)e * kv_ld]);
-#pragma unroll
-                for (int b = 0; b < LA_B; ++b) acc[b] = fmaf(q_smem[b * dim + e], wv, acc[b]);
-            }
-#pragma unroll
-            for (int b = 0; b < LA_B; ++b)
-                if (b < nb) q_abs[((int64_t)(b0 + b) * H + h) * width + n] = from_f<T>(acc[b]);
-        }
+    for (int i = threadIdx.x; i < LA_B * dim; i += LA_N) {
+        const int b = i / dim, e = i - b * dim;
+        q_smem[e * LA_B + b] = b < nb ? to_f(q[(b0 + b) * q_ld + h * (dim + rot) + e]) : 0.f;
     }
+    __syncthreads();
+    if (n >= kv_ld) return;
+    float acc[LA_B];
+#pragma unroll
+    for (int b = 0; b < LA_B; ++b) acc[b] = 0.f;
+    const T* w = wuk + (int64_t)h * dim * kv_ld + n;
+#pragma unroll 16
+    for (int e = 0; e < dim; ++e) {
+        const float wv = to_f(w[(int64_t)e * kv_ld]);
+        float q8[LA_B];
+        load4(q_smem + e * LA_B, *reinterpret_cast<float(*)[4]>(q8));
+        load4(q_smem + e * LA_B + 4, *reinterpret_cast<float(*)[4]>(q8 + 4));
+#pragma unroll
+        for (int b = 0; b < LA_B; ++b) acc[b] = fmaf(q8[b], wv, acc[b]);
+    }
+#pragma unroll
+    for (int b = 0; b < LA_B; ++b)
+        if (b < nb) q_abs[((int64_t)(b0 + b) * H + h) * width + n] = from_f<T>(acc[b]);
 }
 
 // ---------------------------------------------------------------------------------------------------------------
@@ -526,7 +527,7 @@ extern "C" int bn_latent_absorb_q(const void* q, int64_t q_ld, const void* wuk, 
     if (int rc = require_sm100()) return rc;
     if (B == 0) return BN_OK;
     const int kl = round8(kv_rank), rl = round8(rot);
-    const unsigned grid = (unsigned)(H * ((kl + LA_N - 1) / LA_N + 1));
+    const unsigned grid = (unsigned)(H * ((kl + LA_N - 1) / LA_N + 1) * ((B + LA_B - 1) / LA_B));
     const size_t smem = (size_t)LA_B * dim * sizeof(float);
     if (dtype == 0) {
         if (int rc = allow_smem(latent_absorb_kernel<float>, smem, what)) return rc;
@@ -550,16 +551,16 @@ extern "C" int bn_latent_decode_splits(int B, int H, int kv_rank, int rot, int w
     return (int)(want < 1 ? 1 : want);
 }
 
-extern "C" int bn_latent_decode(const void* q_abs, const void* ring, int ring_tokens, const int32_t* seq_ids,
+extern "C" int bn_latent_decode(const void* q_abs, const void* ring, int num_slots, int ring_tokens, const int32_t* seq_ids,
                                 const int32_t* positions, float* partial, float* lse, int splits, int B, int H, int kv_rank, int rot,
                                 int window, float scale, int dtype, bn_stream_t stream) {
     const char* what = "bn_latent_decode";
     if (!q_abs || !ring || !positions || !partial || !lse) return fail(BN_ERR_INVALID_ARG, "%s: null pointer", what);
-    if (B < 0 || H <= 0 || kv_rank <= 0 || rot < 0 || window <= 0 || ring_tokens < window || splits <= 0 || (dtype & ~1))
+    if (B < 0 || H <= 0 || kv_rank <= 0 || rot < 0 || window <= 0 || num_slots <= 0 || ring_tokens < window || splits <= 0 || (dtype & ~1))
         return fail(BN_ERR_INVALID_ARG, "%s: bad shape B=%d H=%d kv_rank=%d window=%d ring_tokens=%d", what, B, H, kv_rank, window, ring_tokens);
     if (int rc = require_sm100()) return rc;
     if (B == 0) return BN_OK;
-    LatentDecodeParams p{q_abs, ring, seq_ids, positions, partial, lse, B, H, round8(kv_rank), round8(rot), ring_tokens, window, splits, scale};
+    LatentDecodeParams p{q_abs, ring, seq_ids, positions, partial, lse, B, H, round8(kv_rank), round8(rot), num_slots, ring_tokens, window, splits, scale};
     if (dtype == 1 && latent_decode_mma_ok(H, p.kv_ld, p.rot_ld)) return latent_decode_mma(p, as_stream(stream));
     if (p.kv_ld > LD_MAXN * 32) return fail(BN_ERR_UNSUPPORTED, "%s: kv_rank=%d (at most %d)", what, kv_rank, LD_MAXN * 32);
     const size_t smem = (size_t)(p.kv_ld + p.rot_ld + LD_WARPS * p.kv_ld + LD_WARPS * 2) * sizeof(float);

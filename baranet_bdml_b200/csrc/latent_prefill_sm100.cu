@@ -1,6 +1,430 @@
+// Windowed attention of a prompt portion on the 5th-generation tensor cores: per-head keys of dim unrotated columns plus
+// one rotated part shared by all heads, values of another width, a sliding window, and keys that start before the
+// portion's first query (bn_attn_window's fast path, bf16).
+//
+// Persistent, one CTA per SM, ten warps.  Work unit = (sequence, head, PAIR of 128-row query tiles); a unit walks the
+// 64-key tiles from the first key that the pair's first row sees to the last row's own key:
+//   warps 0-3 / 4-7   softmax of query tile 0 / 1: thread = TMEM lane = query row, 64 scores of a step in registers
+//   warp 8            MMA issuer (one elected thread)
+//   warp 9            TMA producer
+// Shared memory holds blocks of 64 columns (128-byte swizzled rows): Q of both tiles, and a ring of K and V stages.  A
+// query or key row is ceil(dim / 64) unrotated blocks and ceil(rot / 64) rotated ones; the tensor maps end at dim (keys)
+// and at dim + rot (queries), so what a block holds beyond its part meets zeros on the other side.
+// Tensor memory: scores of tile 0 / 1 at columns [0, 64) / [64, 128), the bf16 weights written over the scores they came
+// from; outputs at [128, 320) / [320, 512), at most 192 value columns.
+// Step (tile u, key tile j): S = Q K^T, softmax with a running maximum that rescales O only when it has grown by 2^8,
+// O += P V.  The issuer's order is  PV(0,j) QK(0,j+1) PV(1,j) QK(1,j+1):  the tensor pipe executes in issue order, so new
+// scores never overtake the read of the weights they replace, and while one tile's softmax runs the other tile's products
+// do.  A commit covers everything issued before it, so the scores' barrier of step j also says that PV of step j - 1 has
+// landed and O may be rescaled.
+// A key tile that a query tile does not see at all is skipped for that tile.  Masks are applied only by warps that have an
+// edge (a row's own key, or the window's far end) inside the key tile.
+// Every wait is bounded; on expiry the kernel raises the caller's error word, frees TMEM and returns.
 #include "common.cuh"
 #include "latent.cuh"
+#include "ptx.cuh"
+#include "tcgen05.cuh"
+#include "tma.cuh"
+
 namespace bn {
-bool attn_window_sm100_ok(const AttnWindowParams&) { return false; }
-int attn_window_sm100(const AttnWindowParams&, cudaStream_t) { return fail(BN_ERR_UNSUPPORTED, "not built"); }
+
+using namespace ptx;
+
+constexpr int WA_BM = 128, WA_BN = 64;
+constexpr int WA_THREADS = 320;
+constexpr int WA_QBLK = WA_BM * 128, WA_KBLK = WA_BN * 128;      // bytes of a 64-column block
+constexpr int WA_MAXSTAGE = 4;
+constexpr uint32_t WA_TMEM_COLS = 512, WA_COL_O = 128, WA_O_STRIDE = 192;
+constexpr int WA_MAXVB = 3;                                      // value blocks of 64 columns
+constexpr int WA_SMEM_LIMIT = 226 * 1024;
+constexpr float WA_LOG2E = 1.4426950408889634f;
+constexpr float WA_RESCALE_THRESHOLD = 8.0f;                     // log2 units
+
+struct WaParams {
+    __nv_bfloat16* out;
+    int64_t out_ld;
+    int* error_word;
+    int B, S, n_old, H, dim, rot, vdim, window;
+    int nb_dim, nb_rot, nb_v, stages;        // 64-column blocks of the unrotated / rotated key parts and of the values
+    int n_pairs, n_units;
+    float scale_log2;
+};
+
+struct WaUnit {
+    int b, h, i0;                            // first query row of the pair
+    int key0, n;                             // first key of key tile 0; key tiles
+    int first[2], last[2];                   // key tiles that query tile u needs (last < first: none)
+};
+
+__device__ __forceinline__ WaUnit wa_unit(const WaParams& p, int k) {
+    WaUnit w;
+    const int bh = k % (p.B * p.H);
+    w.i0 = (p.n_pairs - 1 - k / (p.B * p.H)) * 2 * WA_BM;          // late rows see the most keys: they come first
+    w.b = bh / p.H;
+    w.h = bh - w.b * p.H;
+    w.key0 = max(0, p.n_old + w.i0 - p.window + 1);
+    w.n = 0;
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+        const int r0 = w.i0 + u * WA_BM;
+        if (r0 >= p.S) { w.first[u] = 0; w.last[u] = -1; continue; }
+        const int lo = max(0, p.n_old + r0 - p.window + 1), hi = p.n_old + min(r0 + WA_BM, p.S) - 1;
+        w.first[u] = (lo - w.key0) / WA_BN;
+        w.last[u] = (hi - w.key0) / WA_BN;
+        w.n = w.last[u] + 1;                                       // tile 1's last key is never before tile 0's
+    }
+    return w;
 }
+
+// units are dealt in snake order, so that the CTAs' sums of a descending sequence stay close
+__device__ __forceinline__ int wa_unit_index(int round, int n_units) {
+    const int G = gridDim.x, c = blockIdx.x;
+    const int k = round * G + ((round & 1) ? G - 1 - c : c);
+    return k < n_units ? k : -1;
+}
+
+__global__ void __launch_bounds__(WA_THREADS, 1)
+attn_window_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
+                         const __grid_constant__ CUtensorMap tmap_r, const __grid_constant__ CUtensorMap tmap_v,
+                         const WaParams p) {
+    extern __shared__ uint8_t smem_raw[];
+    __shared__ __align__(8) uint64_t bar_q[2], bar_qfree[2], bar_s[2], bar_p[2], bar_o[2];
+    __shared__ __align__(8) uint64_t bar_kfull[WA_MAXSTAGE], bar_kempty[WA_MAXSTAGE], bar_vfull[WA_MAXSTAGE], bar_vempty[WA_MAXSTAGE];
+    __shared__ uint32_t s_tmem_base;
+    __shared__ int s_abort;
+
+    const int tid = threadIdx.x, warp = tid / 32, lane = tid % 32;
+    const int nb = p.nb_dim + p.nb_rot;
+    const uint32_t smem0 = (smem_u32(smem_raw) + 1023u) & ~1023u;
+    const uint32_t sQ = smem0, sK = smem0 + 2 * nb * WA_QBLK, sV = sK + p.stages * nb * WA_KBLK;
+
+    if (tid == 0) {
+        for (int u = 0; u < 2; ++u) {
+            mbar_init(smem_u32(&bar_q[u]), 1);
+            mbar_init(smem_u32(&bar_qfree[u]), 1);
+            mbar_init(smem_u32(&bar_s[u]), 1);
+            mbar_init(smem_u32(&bar_p[u]), 128);
+            mbar_init(smem_u32(&bar_o[u]), 1);
+        }
+        for (int s = 0; s < WA_MAXSTAGE; ++s) {
+            mbar_init(smem_u32(&bar_kfull[s]), 1);
+            mbar_init(smem_u32(&bar_kempty[s]), 1);
+            mbar_init(smem_u32(&bar_vfull[s]), 1);
+            mbar_init(smem_u32(&bar_vempty[s]), 1);
+        }
+        s_abort = 0;
+        fence_mbar_init();
+    }
+    if (warp == 8) {
+        tc::tmem_alloc(smem_u32(&s_tmem_base), WA_TMEM_COLS);
+        tc::tmem_relinquish();
+    }
+    tc::fence_before_sync();
+    __syncthreads();
+    tc::fence_after_sync();
+    const uint32_t tmem = s_tmem_base;
+
+    if (warp == 9) {
+        // ---------------------------------------------------------- TMA producer
+        if (lane == 0) {
+            prefetch_tensormap(&tmap_q);
+            prefetch_tensormap(&tmap_k);
+            prefetch_tensormap(&tmap_r);
+            prefetch_tensormap(&tmap_v);
+            bool ok = true;
+            int stage = 0;
+            uint32_t phase = 0, nq[2] = {0, 0};              // nq: query tiles loaded so far
+            for (int round = 0; ok; ++round) {
+                const int k = wa_unit_index(round, p.n_units);
+                if (k < 0) break;
+                const WaUnit w = wa_unit(p, k);
+#pragma unroll
+                for (int u = 0; u < 2; ++u) {
+                    if (!ok || w.last[u] < w.first[u]) continue;
+                    ok = mbar_wait(smem_u32(&bar_qfree[u]), (nq[u] & 1u) ^ 1u, &s_abort);
+                    if (!ok) continue;
+                    ++nq[u];
+                    mbar_arrive_expect_tx(smem_u32(&bar_q[u]), nb * WA_QBLK);
+                    for (int x = 0; x < nb; ++x) {
+                        const int col = x < p.nb_dim ? x * 64 : p.dim + (x - p.nb_dim) * 64;
+                        tma_load_4d(sQ + (u * nb + x) * WA_QBLK, &tmap_q, col, w.h, w.i0 + u * WA_BM, w.b, smem_u32(&bar_q[u]));
+                    }
+                }
+                for (int j = 0; ok && j < w.n; ++j) {
+                    const int key = w.key0 + j * WA_BN;
+                    ok = mbar_wait(smem_u32(&bar_kempty[stage]), phase ^ 1u, &s_abort);
+                    if (!ok) break;
+                    mbar_arrive_expect_tx(smem_u32(&bar_kfull[stage]), nb * WA_KBLK);
+                    for (int x = 0; x < p.nb_dim; ++x)
+                        tma_load_4d(sK + (stage * nb + x) * WA_KBLK, &tmap_k, x * 64, w.h, key, w.b, smem_u32(&bar_kfull[stage]));
+                    for (int x = 0; x < p.nb_rot; ++x)
+                        tma_load_4d(sK + (stage * nb + p.nb_dim + x) * WA_KBLK, &tmap_r, x * 64, 0, key, w.b, smem_u32(&bar_kfull[stage]));
+                    ok = mbar_wait(smem_u32(&bar_vempty[stage]), phase ^ 1u, &s_abort);
+                    if (!ok) break;
+                    mbar_arrive_expect_tx(smem_u32(&bar_vfull[stage]), p.nb_v * WA_KBLK);
+                    for (int x = 0; x < p.nb_v; ++x)
+                        tma_load_4d(sV + (stage * p.nb_v + x) * WA_KBLK, &tmap_v, x * 64, w.h, key, w.b, smem_u32(&bar_vfull[stage]));
+                    if (++stage == p.stages) { stage = 0; phase ^= 1u; }
+                }
+            }
+        }
+    } else if (warp == 8) {
+        // ------------------------------------------------------------ MMA issuer
+        constexpr uint32_t IDESC_QK = tc::idesc_bf16(WA_BM, WA_BN, 0), IDESC_PV = tc::idesc_bf16(WA_BM, 64, 1);
+        const uint64_t dZero = tc::smem_desc_sw128(0);               // descriptor = this + (address >> 4)
+        bool ok = true;
+        int kstage = 0, vstage = 0;
+        uint32_t kphase = 0, vphase = 0, nq[2] = {0, 0}, np[2] = {0, 0};
+        for (int round = 0; ok; ++round) {
+            const int k = wa_unit_index(round, p.n_units);
+            if (k < 0) break;
+            const WaUnit w = wa_unit(p, k);
+            for (int j = -1; ok && j < w.n; ++j) {
+                bool k_here = false, v_here = false;
+#pragma unroll
+                for (int u = 0; u < 2; ++u) {
+                    if (!ok) continue;
+                    const uint32_t tS = tmem + u * WA_BN, tO = tmem + WA_COL_O + u * WA_O_STRIDE;
+                    if (j >= w.first[u] && j <= w.last[u]) {          // O += P V of key tile j
+                        ok = mbar_wait(smem_u32(&bar_p[u]), np[u] & 1u, &s_abort);
+                        ++np[u];
+                        if (ok && !v_here) {
+                            ok = mbar_wait(smem_u32(&bar_vfull[vstage]), vphase, &s_abort);
+                            v_here = true;
+                        }
+                        if (!ok) continue;
+                        if (elect_one()) {
+                            tc::fence_after_sync();
+                            for (int x = 0; x < p.nb_v; ++x) {
+                                const uint32_t v = sV + (vstage * p.nb_v + x) * WA_KBLK;
+#pragma unroll
+                                for (int kk = 0; kk < WA_BN / 16; ++kk)
+                                    tc::mma_ts(tO + x * 64, tS + kk * 8, dZero + (uint64_t)((v >> 4) + kk * 128), IDESC_PV,
+                                               j > w.first[u] || kk > 0);
+                            }
+                            if (j == w.last[u]) tc::commit(smem_u32(&bar_o[u]));
+                        }
+                        __syncwarp();
+                    }
+                    if (j + 1 >= w.first[u] && j + 1 <= w.last[u]) {  // S = Q K^T of key tile j + 1
+                        if (j + 1 == w.first[u]) {
+                            ok = mbar_wait(smem_u32(&bar_q[u]), nq[u] & 1u, &s_abort);
+                            ++nq[u];
+                        }
+                        if (ok && !k_here) {
+                            ok = mbar_wait(smem_u32(&bar_kfull[kstage]), kphase, &s_abort);
+                            k_here = true;
+                        }
+                        if (!ok) continue;
+                        if (elect_one()) {
+                            tc::fence_after_sync();
+                            bool more = false;
+                            for (int x = 0; x < nb; ++x) {
+                                const int cols = x < p.nb_dim ? p.dim - x * 64 : p.rot - (x - p.nb_dim) * 64;
+                                const int steps = cols >= 64 ? 4 : (cols + 15) / 16;
+                                const uint32_t qa = sQ + (u * nb + x) * WA_QBLK, ka = sK + (kstage * nb + x) * WA_KBLK;
+                                for (int kk = 0; kk < steps; ++kk) {
+                                    tc::mma_ss(tS, dZero + (uint64_t)((qa >> 4) + kk * 2), dZero + (uint64_t)((ka >> 4) + kk * 2),
+                                               IDESC_QK, more);
+                                    more = true;
+                                }
+                            }
+                            tc::commit(smem_u32(&bar_s[u]));
+                            if (j + 1 == w.last[u]) tc::commit(smem_u32(&bar_qfree[u]));
+                        }
+                        __syncwarp();
+                    }
+                }
+                if (!ok) break;
+                if (elect_one()) {
+                    if (j >= 0) tc::commit(smem_u32(&bar_vempty[vstage]));
+                    if (j + 1 < w.n) tc::commit(smem_u32(&bar_kempty[kstage]));
+                }
+                __syncwarp();
+                if (j >= 0 && ++vstage == p.stages) { vstage = 0; vphase ^= 1u; }
+                if (j + 1 < w.n && ++kstage == p.stages) { kstage = 0; kphase ^= 1u; }
+            }
+        }
+    } else {
+        // ---------------------------------------------------------- softmax warps
+        const int u = warp / 4;
+        const uint32_t lane_base = ((uint32_t)((warp % 4) * 32)) << 16;
+        const uint32_t tS = tmem + lane_base + u * WA_BN, tO = tmem + lane_base + WA_COL_O + u * WA_O_STRIDE;
+        bool ok = true;
+        uint32_t ns = 0, no = 0;                                     // steps and tiles of this query tile so far
+        for (int round = 0; ok; ++round) {
+            const int k = wa_unit_index(round, p.n_units);
+            if (k < 0) break;
+            const WaUnit w = wa_unit(p, k);
+            if (w.last[u] < w.first[u]) continue;
+            const int row0 = w.i0 + u * WA_BM + (warp % 4) * 32;     // the warp's first row
+            const int gi = row0 + lane;
+            const int own = p.n_old + gi, oldest = own - p.window + 1;         // the keys this row sees
+            const int warp_own0 = p.n_old + row0, warp_oldest1 = warp_own0 + 31 - p.window + 1;
+            float m_ref = -INFINITY, l_run = 0.f;
+            for (int j = w.first[u]; j <= w.last[u]; ++j, ++ns) {
+                ok = mbar_wait(smem_u32(&bar_s[u]), ns & 1u, &s_abort);
+                if (!ok) break;
+                tc::fence_after_sync();
+                const int key = w.key0 + j * WA_BN;
+                const bool masked = key + WA_BN - 1 > warp_own0 || key < warp_oldest1;
+                uint32_t r[2][32];
+                tc::ld32(tS, r[0]);
+                tc::ld32(tS + 32, r[1]);
+                tc::wait_ld(r[0]);
+                tc::wait_ld(r[1]);
+                if (masked) {
+#pragma unroll
+                    for (int c = 0; c < 2; ++c)
+#pragma unroll
+                        for (int i = 0; i < 32; ++i) {
+                            const int kk = key + c * 32 + i;
+                            if (kk > own || kk < oldest) r[c][i] = 0xff800000u;          // -inf
+                        }
+                }
+                float t0 = -INFINITY, t1 = -INFINITY, t2 = -INFINITY, t3 = -INFINITY;
+#pragma unroll
+                for (int i = 0; i < 32; i += 2) {
+                    t0 = fmaxf(t0, __uint_as_float(r[0][i]));
+                    t1 = fmaxf(t1, __uint_as_float(r[0][i + 1]));
+                    t2 = fmaxf(t2, __uint_as_float(r[1][i]));
+                    t3 = fmaxf(t3, __uint_as_float(r[1][i + 1]));
+                }
+                const float m_new = fmaxf(m_ref, fmaxf(fmaxf(t0, t1), fmaxf(t2, t3)));
+                const bool grow = (m_new - m_ref) * p.scale_log2 > WA_RESCALE_THRESHOLD;   // NaN (both -inf) is false
+                if (__any_sync(0xffffffffu, grow)) {
+                    if (j > w.first[u]) {
+                        const float alpha = m_ref == -INFINITY ? 0.f : ex2((m_ref - m_new) * p.scale_log2);
+                        l_run *= alpha;
+                        for (int c = 0; c < 2 * p.nb_v; ++c) {
+                            uint32_t o[32];
+                            tc::ld32(tO + c * 32, o);
+                            tc::wait_ld(o);
+#pragma unroll
+                            for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * alpha);
+                            tc::st32(tO + c * 32, o);
+                        }
+                    }
+                    m_ref = m_new;
+                }
+                // a row that has seen no key yet has only -inf scores: any finite reference gives zero weights
+                const float mneg = m_ref == -INFINITY ? 0.f : -m_ref * p.scale_log2;
+                float l0 = 0.f, l1 = 0.f;
+#pragma unroll
+                for (int c = 0; c < 2; ++c) {
+                    uint32_t pk[16];
+#pragma unroll
+                    for (int i = 0; i < 32; i += 2) {
+                        const float p0 = ex2(fmaf(__uint_as_float(r[c][i]), p.scale_log2, mneg));
+                        const float p1 = ex2(fmaf(__uint_as_float(r[c][i + 1]), p.scale_log2, mneg));
+                        l0 += p0;
+                        l1 += p1;
+                        pk[i / 2] = pack_bf16(p0, p1);
+                    }
+                    tc::st16(tS + c * 16, pk);
+                }
+                l_run += l0 + l1;
+                tc::wait_st();
+                tc::fence_before_sync();
+                mbar_arrive(smem_u32(&bar_p[u]));
+            }
+            if (!ok) break;
+            // O / l -> bf16 -> global
+            ok = mbar_wait(smem_u32(&bar_o[u]), no & 1u, &s_abort);
+            ++no;
+            if (!ok) break;
+            tc::fence_after_sync();
+            const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+            __nv_bfloat16* dst = p.out + ((int64_t)w.b * p.S + gi) * p.out_ld + w.h * p.vdim;
+            for (int c = 0; c < 2 * p.nb_v; ++c) {
+                uint32_t o[32];
+                tc::ld32(tO + c * 32, o);
+                tc::wait_ld(o);
+                if (gi < p.S) {
+#pragma unroll
+                    for (int v = 0; v < 4; ++v)
+                        if (c * 32 + v * 8 < p.vdim) {                 // vdim is a multiple of 8
+                            uint4 o4;
+                            o4.x = pack_bf16(__uint_as_float(o[v * 8 + 0]) * inv, __uint_as_float(o[v * 8 + 1]) * inv);
+                            o4.y = pack_bf16(__uint_as_float(o[v * 8 + 2]) * inv, __uint_as_float(o[v * 8 + 3]) * inv);
+                            o4.z = pack_bf16(__uint_as_float(o[v * 8 + 4]) * inv, __uint_as_float(o[v * 8 + 5]) * inv);
+                            o4.w = pack_bf16(__uint_as_float(o[v * 8 + 6]) * inv, __uint_as_float(o[v * 8 + 7]) * inv);
+                            *reinterpret_cast<uint4*>(dst + c * 32 + v * 8) = o4;
+                        }
+                }
+            }
+            // the next unit's first PV overwrites O: it waits for this warp's next arrival on bar_p, which follows
+            tc::fence_before_sync();
+        }
+    }
+
+    // common exit: everybody arrives here (all waits are bounded), then TMEM is freed
+    tc::fence_before_sync();
+    __syncthreads();
+    if (tid == 0 && s_abort && p.error_word) atomicExch(p.error_word, BN_ERR_TIMEOUT);
+    if (warp == 8) {
+        tc::fence_after_sync();
+        tc::tmem_dealloc(tmem, WA_TMEM_COLS);
+    }
+}
+
+static int wa_stages(int nb, int nb_v) {
+    const int left = WA_SMEM_LIMIT - 1024 - 2 * nb * WA_QBLK;
+    const int per = (nb + nb_v) * WA_KBLK;
+    const int s = left > 0 ? left / per : 0;
+    return s > WA_MAXSTAGE ? WA_MAXSTAGE : s;
+}
+
+bool attn_window_sm100_ok(const AttnWindowParams& p) {
+    const int nb = (p.dim + 63) / 64 + (p.rot + 63) / 64, nb_v = (p.vdim + 63) / 64;
+    const uintptr_t bases = reinterpret_cast<uintptr_t>(p.q) | reinterpret_cast<uintptr_t>(p.k) | reinterpret_cast<uintptr_t>(p.v) |
+                            reinterpret_cast<uintptr_t>(p.krot) | reinterpret_cast<uintptr_t>(p.out);
+    return ((p.dim | p.rot | p.vdim | p.q_ld | p.kv_ld | p.krot_ld | p.out_ld) & 7) == 0 && p.rot > 0 && (bases & 15) == 0 &&
+           nb_v <= WA_MAXVB && wa_stages(nb, nb_v) >= 2 && p.scale > 0.f;
+}
+
+static int wa_map(CUtensorMap* m, const void* base, int inner, int heads, int64_t head_stride, int rows, int64_t ld, int B, int box_rows) {
+    const uint64_t dims[4] = {(uint64_t)inner, (uint64_t)heads, (uint64_t)rows, (uint64_t)B};
+    const uint64_t strides[3] = {(uint64_t)head_stride * 2, (uint64_t)ld * 2, (uint64_t)ld * 2 * rows};
+    const uint32_t box[4] = {64, 1, (uint32_t)box_rows, 1};
+    return make_tensor_map(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, base, dims, strides, box, CU_TENSOR_MAP_SWIZZLE_128B);
+}
+
+int attn_window_sm100(const AttnWindowParams& a, cudaStream_t st) {
+    const char* what = "bn_attn_window";
+    CUtensorMap mq, mk, mr, mv;
+    if (int rc = wa_map(&mq, a.q, a.dim + a.rot, a.H, a.dim + a.rot, a.S, a.q_ld, a.B, WA_BM)) return rc;
+    if (int rc = wa_map(&mk, a.k, a.dim, a.H, a.dim, a.rows_per_seq, a.kv_ld, a.B, WA_BN)) return rc;
+    if (int rc = wa_map(&mr, a.krot, a.rot, 1, a.krot_ld, a.rows_per_seq, a.krot_ld, a.B, WA_BN)) return rc;
+    if (int rc = wa_map(&mv, a.v, a.vdim, a.H, a.vdim, a.rows_per_seq, a.kv_ld, a.B, WA_BN)) return rc;
+    WaParams p;
+    p.out = static_cast<__nv_bfloat16*>(a.out);
+    p.out_ld = a.out_ld;
+    p.error_word = a.error_word;
+    p.B = a.B; p.S = a.S; p.n_old = a.n_old; p.H = a.H; p.dim = a.dim; p.rot = a.rot; p.vdim = a.vdim; p.window = a.window;
+    p.nb_dim = (a.dim + 63) / 64;
+    p.nb_rot = (a.rot + 63) / 64;
+    p.nb_v = (a.vdim + 63) / 64;
+    p.stages = wa_stages(p.nb_dim + p.nb_rot, p.nb_v);
+    p.n_pairs = (a.S + 2 * WA_BM - 1) / (2 * WA_BM);
+    const long long units = (long long)a.B * a.H * p.n_pairs;
+    if (units > (1 << 30)) return fail(BN_ERR_UNSUPPORTED, "%s: too many query tiles", what);
+    p.n_units = (int)units;
+    p.scale_log2 = a.scale * WA_LOG2E;
+    const int nb = p.nb_dim + p.nb_rot;
+    const size_t smem = 1024 + (size_t)2 * nb * WA_QBLK + (size_t)p.stages * (nb + p.nb_v) * WA_KBLK;
+    int dev = 0, sms = 0;
+    cudaGetDevice(&dev);
+    cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
+    static thread_local int configured_dev = -1;
+    if (configured_dev != dev) {
+        cudaError_t e = cudaFuncSetAttribute(attn_window_sm100_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, WA_SMEM_LIMIT);
+        if (e != cudaSuccess) return fail(BN_ERR_CUDA, "%s: %s", what, cudaGetErrorString(e));
+        configured_dev = dev;
+    }
+    const unsigned grid = (unsigned)(p.n_units < sms ? p.n_units : sms);
+    attn_window_sm100_kernel<<<grid, WA_THREADS, smem, st>>>(mq, mk, mr, mv, p);
+    return launch_status(what);
+}
+
+}  // namespace bn

@@ -107,7 +107,7 @@ class LatentAttention:
         splits = lib.bn_latent_decode_splits(B, c.heads, c.kv_rank, c.rot_dim, c.window, dt)
         partial = torch.empty((B, c.heads, splits, self.kv_ld), dtype=torch.float32, device=dev)
         lse = torch.empty((B, c.heads, splits), dtype=torch.float32, device=dev)
-        _lib.check(lib.bn_latent_decode(q_abs.data_ptr(), cache.ring.data_ptr(), cache.ring_tokens, seq_ids.data_ptr(),
+        _lib.check(lib.bn_latent_decode(q_abs.data_ptr(), cache.ring.data_ptr(), cache.num_seqs, cache.ring_tokens, seq_ids.data_ptr(),
                                         positions.data_ptr(), partial.data_ptr(), lse.data_ptr(), splits, B, c.heads, c.kv_rank,
                                         c.rot_dim, c.window, float(c.scale), dt, s))
         _lib.check(lib.bn_latent_expand_out(partial.data_ptr(), lse.data_ptr(), splits, self.uv.data_ptr(), out.data_ptr(),

@@ -443,7 +443,7 @@ BN_API int bn_latent_absorb_q(const void* q, int64_t q_ld, const void* wuk, cons
 /* how many parts bn_latent_decode cuts a window into (a size, 0 for a bad shape): partial holds
  * B * H * splits * round8(kv_rank) floats and lse B * H * splits */
 BN_API int bn_latent_decode_splits(int B, int H, int kv_rank, int rot, int window, int dtype);
-BN_API int bn_latent_decode(const void* q_abs, const void* ring, int ring_tokens, const int32_t* seq_ids,
+BN_API int bn_latent_decode(const void* q_abs, const void* ring, int num_slots, int ring_tokens, const int32_t* seq_ids,
                             const int32_t* positions, float* partial, float* lse, int splits, int B, int H, int kv_rank,
                             int rot, int window, float scale, int dtype, bn_stream_t stream);
 /* merges the parts and expands the latent sum: out (B, out_ld), column h * vdim + v; wuv (H * vdim, round8(kv_rank)) */
