@@ -1153,6 +1153,17 @@ def run_ours(args):
         dist.destroy_process_group()
 
 
+def run_soluzen(args):
+    import torch
+    import bench_soluzen
+    torch.cuda.set_device(0)
+    sampler = ClockSampler(0)
+    sampler.start()
+    res = bench_soluzen.run(peaks(), max(10, args.steps))
+    res["clocks"] = sampler.stop()
+    _emit(json.dumps(res))
+
+
 def main():
     # stdout carries exactly one JSON line: everything else that writes to file descriptor 1 (NCCL's version
     # banner, library chatter) is sent to stderr, and the line is written to the real stdout at the end
@@ -1179,7 +1190,13 @@ def main():
     ap.add_argument("--generate-steps", type=int, default=128, help="decode steps of the config-5 generation")
     ap.add_argument("--longctx-only", action="store_true",
                     help="run only the config-4 sequence-split decode (decode kernel + exchange); prints its object alone")
+    ap.add_argument("--soluzen", action="store_true",
+                    help="measure the Soluzen design (whole models beside LLaMA, and its kernels one by one) instead of the "
+                         "default workload; prints its object alone")
     args = ap.parse_args()
+    if args.soluzen:
+        run_soluzen(args)
+        return
     if args.warmup < 3 and args.impl == "ours":
         args.warmup = 3
     if args.impl == "reference":

@@ -79,7 +79,9 @@ def weights(cfg, seed=0, peak=2.5):
     for name, shape in shapes(cfg).items():
         x = rng.standard_normal(shape)
         leaf = name.rsplit(".", 1)[-1]
-        if name.endswith("norm") or leaf in ("norm1", "norm2"):
+        if name.endswith("side.norm"):
+            x = 0.3 + 0.1 * x                      # what is added is normalised: a full-size one would drown the rest
+        elif name.endswith("norm") or leaf in ("norm1", "norm2"):
             x = 1.0 + 0.3 * x
         elif leaf == "b":
             x = 0.2 * x
@@ -93,6 +95,8 @@ def weights(cfg, seed=0, peak=2.5):
             x = x * 0.7
         elif leaf == "uq":
             x = peak * x / np.sqrt(shape[1])
+        elif name == "loop.in":                    # mostly keeps the stream, mixes some of the embedding in
+            x = 0.3 * x / np.sqrt(shape[1]) + np.eye(*shape)
         elif leaf in ("embed", "step"):
             x = x * (1.0 if leaf == "embed" else 0.3)
         else:
@@ -105,10 +109,15 @@ def as_f64(w):
     return {k: v.double().numpy() for k, v in w.items()}
 
 
-def error(got, want):
-    """Root mean square of the difference of each row, mean taken off, over that of `want`; the largest row."""
+def row_errors(got, want):
+    """Root mean square of the difference of each row, mean taken off, over that of `want`."""
     got, want = np.asarray(got, dtype=np.float64), np.asarray(want, dtype=np.float64)
     d = got - want
     d = d - d.mean(axis=-1, keepdims=True)
     s = want - want.mean(axis=-1, keepdims=True)
-    return float((np.sqrt((d * d).mean(-1)) / np.sqrt((s * s).mean())).max())
+    return np.sqrt((d * d).mean(-1)) / np.sqrt((s * s).mean())
+
+
+def error(got, want):
+    """The largest of them."""
+    return float(row_errors(got, want).max())
