@@ -39,7 +39,8 @@ struct LatentPrepParams {
 
 constexpr int LP_THREADS = 128;
 
-template <typename T>
+// VEC = 4: ranks and row strides are multiples of 4 and every row starts on a 16-byte (bf16: 8-byte) boundary
+template <typename T, int VEC>
 __global__ void __launch_bounds__(LP_THREADS)
 latent_prep_kernel(const LatentPrepParams p) {
     __shared__ float sh[2][LP_THREADS / 32];
@@ -49,8 +50,23 @@ latent_prep_kernel(const LatentPrepParams p) {
         const int b = r / p.S, s = r - b * p.S;
         const T* in = static_cast<const T*>(p.proj) + (int64_t)r * p.proj_ld;
         float sq = 0.f, sk = 0.f;
-        for (int i = threadIdx.x; i < p.q_rank; i += LP_THREADS) { const float v = to_f(in[i]); sq = fmaf(v, v, sq); }
-        for (int i = threadIdx.x; i < p.kv_rank; i += LP_THREADS) { const float v = to_f(in[p.q_rank + i]); sk = fmaf(v, v, sk); }
+        auto sum_squares = [&](const T* x, int n) {
+            float s = 0.f;
+            if (VEC == 4) {
+#pragma unroll 4
+                for (int i = threadIdx.x * 4; i < n; i += LP_THREADS * 4) {
+                    float v[4];
+                    load4(x + i, v);
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) s = fmaf(v[e], v[e], s);
+                }
+            } else {
+                for (int i = threadIdx.x; i < n; i += LP_THREADS) { const float v = to_f(x[i]); s = fmaf(v, v, s); }
+            }
+            return s;
+        };
+        sq = sum_squares(in, p.q_rank);
+        sk = sum_squares(in + p.q_rank, p.kv_rank);
 #pragma unroll
         for (int o = 16; o > 0; o >>= 1) {
             sq += __shfl_xor_sync(0xffffffffu, sq, o);
@@ -64,9 +80,32 @@ latent_prep_kernel(const LatentPrepParams p) {
         for (int w = 0; w < LP_THREADS / 32; ++w) { sq += sh[0][w]; sk += sh[1][w]; }
         const float inv_q = rsqrtf(sq / (float)p.q_rank + p.eps), inv_k = rsqrtf(sk / (float)p.kv_rank + p.eps);
 
+        // n of ld columns normalised, the rest zero, to one or two places
+        auto emit = [&](const T* x, float inv, const float* w, int n, int ld, T* d0, T* d1) {
+            if (VEC == 4) {
+#pragma unroll 4
+                for (int i = threadIdx.x * 4; i < ld; i += LP_THREADS * 4) {
+                    float v[4] = {0.f, 0.f, 0.f, 0.f};
+                    if (i < n) {
+                        float w4[4];
+                        load4(x + i, v);
+                        load4(w + i, w4);
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) v[e] = v[e] * inv * w4[e];
+                    }
+                    if (d0) store4(d0 + i, v);
+                    if (d1) store4(d1 + i, v);
+                }
+            } else {
+                for (int i = threadIdx.x; i < ld; i += LP_THREADS) {
+                    const T v = from_f<T>(i < n ? to_f(x[i]) * inv * w[i] : 0.f);
+                    if (d0) d0[i] = v;
+                    if (d1) d1[i] = v;
+                }
+            }
+        };
         T* cq = static_cast<T*>(p.cq) + (int64_t)r * p.cq_ld;
-        for (int i = threadIdx.x; i < p.cq_ld; i += LP_THREADS)
-            cq[i] = from_f<T>(i < p.q_rank ? to_f(in[i]) * inv_q * p.q_norm[i] : 0.f);
+        emit(in, inv_q, p.q_norm, p.q_rank, (int)p.cq_ld, cq, nullptr);
 
         const int pos = p.positions[b] + s;
         const int64_t out_row = (int64_t)b * p.rows_per_seq + p.row_offset + s;
@@ -78,11 +117,7 @@ latent_prep_kernel(const LatentPrepParams p) {
             const int slot = p.seq_ids ? p.seq_ids[b] : b;
             ring = static_cast<T*>(p.ring) + ((int64_t)slot * p.ring_tokens + pos % p.ring_tokens) * (p.kv_ld + p.rot_ld);
         }
-        for (int i = threadIdx.x; i < p.kv_ld; i += LP_THREADS) {
-            const T v = from_f<T>(i < p.kv_rank ? to_f(in[p.q_rank + i]) * inv_k * p.kv_norm[i] : 0.f);
-            if (c) c[i] = v;
-            if (ring) ring[i] = v;
-        }
+        emit(in + p.q_rank, inv_k, p.kv_norm, p.kv_rank, p.kv_ld, c, ring);
         const T* rin = in + p.q_rank + p.kv_rank;
         for (int i = threadIdx.x; i < p.rot_ld / 2; i += LP_THREADS) {
             T lo = from_f<T>(0.f), hi = lo;
@@ -445,8 +480,13 @@ extern "C" int bn_latent_prep(const void* proj, int64_t proj_ld, const float* q_
                        kv_rank, rot, round8(kv_rank), round8(rot), rows_per_seq, row_offset, ring_tokens, eps};
     const int cap = sm_count() * 16;
     const unsigned grid = (unsigned)(B * S < cap ? B * S : cap);
-    if (dtype == 0) launch_dependent(latent_prep_kernel<float>, grid, LP_THREADS, 0, as_stream(stream), p);
-    else launch_dependent(latent_prep_kernel<__nv_bfloat16>, grid, LP_THREADS, 0, as_stream(stream), p);
+    const uintptr_t all = reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(q_norm) | reinterpret_cast<uintptr_t>(kv_norm) |
+                          reinterpret_cast<uintptr_t>(cq) | reinterpret_cast<uintptr_t>(c) | reinterpret_cast<uintptr_t>(ring);
+    const bool vec = q_rank % 4 == 0 && kv_rank % 4 == 0 && proj_ld % 4 == 0 && cq_ld % 4 == 0 && (all & 15) == 0;
+    if (dtype == 0 && vec) launch_dependent(latent_prep_kernel<float, 4>, grid, LP_THREADS, 0, as_stream(stream), p);
+    else if (dtype == 0) launch_dependent(latent_prep_kernel<float, 1>, grid, LP_THREADS, 0, as_stream(stream), p);
+    else if (vec) launch_dependent(latent_prep_kernel<__nv_bfloat16, 4>, grid, LP_THREADS, 0, as_stream(stream), p);
+    else launch_dependent(latent_prep_kernel<__nv_bfloat16, 1>, grid, LP_THREADS, 0, as_stream(stream), p);
     return launch_status(what);
 }
 
@@ -527,6 +567,8 @@ extern "C" int bn_latent_absorb_q(const void* q, int64_t q_ld, const void* wuk, 
     if (int rc = require_sm100()) return rc;
     if (B == 0) return BN_OK;
     const int kl = round8(kv_rank), rl = round8(rot);
+    if (dtype == 1 && latent_absorb_mma(q, q_ld, wuk, freq, positions, q_abs, B, H, dim, rot, kl, rl, as_stream(stream)))
+        return launch_status(what);
     const unsigned grid = (unsigned)(H * ((kl + LA_N - 1) / LA_N + 1) * ((B + LA_B - 1) / LA_B));
     const size_t smem = (size_t)LA_B * dim * sizeof(float);
     if (dtype == 0) {
@@ -583,6 +625,8 @@ extern "C" int bn_latent_expand_out(const float* partial, const float* lse, int 
     if (int rc = require_sm100()) return rc;
     if (B == 0) return BN_OK;
     const int kl = round8(kv_rank);
+    if (dtype == 1 && latent_expand_mma(partial, lse, splits, wuv, out, out_ld, B, H, vdim, kl, as_stream(stream)))
+        return launch_status(what);
     const unsigned grid = (unsigned)(((vdim + LO_V - 1) / LO_V) * H * ((B + LO_B - 1) / LO_B));
     const size_t smem = (size_t)LO_B * kl * sizeof(float);
     if (dtype == 0) {

@@ -15,6 +15,7 @@
 // A split's result is its normalised sum and log-sum-exp; bn_latent_expand_out merges the splits.
 // Waits are bounded: on expiry the CTA stops and leaves a NaN log-sum-exp, which surfaces as NaN logits.
 #include "common.cuh"
+#include "hybrid.cuh"
 #include "latent.cuh"
 #include "ptx.cuh"
 #include "tma.cuh"
@@ -283,6 +284,222 @@ int latent_decode_mma(const LatentDecodeParams& a, cudaStream_t st) {
     }
     launch_dependent(latent_decode_mma_kernel, (unsigned)((long long)a.B * p.groups * a.splits), LM_THREADS, L.total, st, tmap, p);
     return launch_status(what);
+}
+
+// ---------------------------------------------------------------------------------------------------------------
+// The two per-head products around it.  Both stream a head's weight once per 16 rows and request it before they wait for
+// the launch ahead of them: weights depend on nothing.
+// ---------------------------------------------------------------------------------------------------------------
+struct AbsorbParams {
+    const __nv_bfloat16 *q, *wuk;
+    const double* freq;
+    const int32_t* positions;
+    __nv_bfloat16* q_abs;
+    int64_t q_ld;
+    int B, H, dim, rot, kv_ld, rot_ld, kp, n_tiles;      // kp: dim rounded up to 16
+    int vec;                                             // query rows and heads start on 16-byte boundaries
+};
+
+constexpr int AB_N = 64;
+
+// q_abs = q W_uk for 16 rows, one head, 64 latent columns; the last tile of a head is its rotated part
+__global__ void __launch_bounds__(128)
+latent_absorb_mma_kernel(const AbsorbParams p) {
+    extern __shared__ __align__(16) uint8_t smem[];
+    const int lda = p.kp + 8;
+    __nv_bfloat16* sw = reinterpret_cast<__nv_bfloat16*>(smem);          // [kp][AB_N + 8]
+    __nv_bfloat16* sa = sw + p.kp * (AB_N + 8);                          // [16][kp + 8]
+    const int tile = blockIdx.x % (p.n_tiles + 1), h = blockIdx.x / (p.n_tiles + 1) % p.H;
+    const int b0 = blockIdx.x / ((p.n_tiles + 1) * p.H) * 16, nb = min(16, p.B - b0);
+    const int width = p.kv_ld + p.rot_ld, E = p.dim + p.rot, n0 = tile * AB_N;
+    const int warp = threadIdx.x / 32, lane = threadIdx.x % 32;
+    if (tile < p.n_tiles) {
+        const __nv_bfloat16* w = p.wuk + (int64_t)h * p.dim * p.kv_ld + n0;
+        for (int i = threadIdx.x; i < p.kp * (AB_N / 8); i += 128) {
+            const int k = i / (AB_N / 8), c = i % (AB_N / 8) * 8;
+            uint4 v = make_uint4(0, 0, 0, 0);
+            if (k < p.dim && n0 + c < p.kv_ld) v = __ldg(reinterpret_cast<const uint4*>(w + (int64_t)k * p.kv_ld + c));
+            *reinterpret_cast<uint4*>(sw + k * (AB_N + 8) + c) = v;
+        }
+    }
+    grid_dependency_wait();
+    grid_launch_dependents();
+    const __nv_bfloat16* q = p.q + (int64_t)b0 * p.q_ld + h * E;
+    if (tile == p.n_tiles) {
+        for (int i = threadIdx.x; i < nb * (p.rot_ld / 2); i += 128) {
+            const int b = i / (p.rot_ld / 2), j = i % (p.rot_ld / 2);
+            uint32_t o = 0;
+            if (2 * j < p.rot) {
+                const __nv_bfloat16* x = q + b * p.q_ld + p.dim + 2 * j;
+                const float u = to_f(x[0]), v = to_f(x[1]);
+                float cs, sn;
+                rotation(p.positions[b0 + b], p.freq[j], &cs, &sn);
+                o = pack_bf16(u * cs - v * sn, v * cs + u * sn);
+            }
+            *reinterpret_cast<uint32_t*>(p.q_abs + ((int64_t)(b0 + b) * p.H + h) * width + p.kv_ld + 2 * j) = o;
+        }
+        return;
+    }
+    if (p.vec) {
+        for (int i = threadIdx.x; i < 16 * (p.kp / 8); i += 128) {
+            const int b = i / (p.kp / 8), c = i % (p.kp / 8) * 8;
+            uint4 v = make_uint4(0, 0, 0, 0);
+            if (b < nb && c < p.dim) v = *reinterpret_cast<const uint4*>(q + b * p.q_ld + c);
+            *reinterpret_cast<uint4*>(sa + b * lda + c) = v;
+        }
+    } else {
+        for (int i = threadIdx.x; i < 16 * p.kp; i += 128) {
+            const int b = i / p.kp, c = i % p.kp;
+            sa[b * lda + c] = b < nb && c < p.dim ? q[b * p.q_ld + c] : __float2bfloat16(0.f);
+        }
+    }
+    __syncthreads();
+    float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};
+    const uint32_t ua = smem_u32(sa) + ((lane % 16) * lda + (lane / 16) * 8) * 2;
+    const uint32_t uw = smem_u32(sw) + ((lane % 16) * (AB_N + 8) + warp * 16 + (lane / 16) * 8) * 2;
+#pragma unroll 4
+    for (int ks = 0; ks < p.kp / 16; ++ks) {
+        uint32_t a0, a1, a2, a3, w0, w1, w2, w3;
+        ldmatrix_x4(ua + ks * 32, a0, a1, a2, a3);
+        ldmatrix_x4_trans(uw + ks * 16 * (AB_N + 8) * 2, w0, w1, w2, w3);
+        mma_bf16_16816(c0, a0, a1, a2, a3, w0, w1);
+        mma_bf16_16816(c1, a0, a1, a2, a3, w2, w3);
+    }
+    const int g = lane / 4, j = lane % 4;
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+        const int b = g + 8 * r;
+        if (b >= nb) continue;
+        __nv_bfloat16* o = p.q_abs + ((int64_t)(b0 + b) * p.H + h) * width + n0 + warp * 16 + 2 * j;
+        if (n0 + warp * 16 + 2 * j < p.kv_ld) *reinterpret_cast<uint32_t*>(o) = pack_bf16(c0[2 * r], c0[2 * r + 1]);
+        if (n0 + warp * 16 + 8 + 2 * j < p.kv_ld) *reinterpret_cast<uint32_t*>(o + 8) = pack_bf16(c1[2 * r], c1[2 * r + 1]);
+    }
+}
+
+bool latent_absorb_mma(const void* q, int64_t q_ld, const void* wuk, const double* freq, const int32_t* positions, void* q_abs, int B,
+                       int H, int dim, int rot, int kv_ld, int rot_ld, cudaStream_t st) {
+    const int kp = (dim + 15) / 16 * 16;
+    const size_t smem = ((size_t)kp * (AB_N + 8) + 16 * (kp + 8)) * 2;
+    if (smem > 48 * 1024 || (reinterpret_cast<uintptr_t>(wuk) & 15) || (reinterpret_cast<uintptr_t>(q_abs) & 3)) return false;
+    AbsorbParams p{static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(wuk), freq, positions,
+                   static_cast<__nv_bfloat16*>(q_abs), q_ld, B, H, dim, rot, kv_ld, rot_ld, kp, (kv_ld + AB_N - 1) / AB_N, 0};
+    p.vec = dim % 8 == 0 && rot % 8 == 0 && q_ld % 8 == 0 && (reinterpret_cast<uintptr_t>(q) & 15) == 0;
+    launch_dependent(latent_absorb_mma_kernel, (unsigned)((p.n_tiles + 1) * H * ((B + 15) / 16)), 128, smem, st, p);
+    return true;
+}
+
+struct ExpandParams {
+    const float *partial, *lse;
+    const __nv_bfloat16* wuv;
+    __nv_bfloat16* out;
+    int64_t out_ld;
+    int splits, B, H, vdim, kv_ld, v_tiles, steps;       // steps: 32-wide pieces of the latent, rounded up
+};
+
+constexpr int EX_V = 32, EX_BATCH = 8, EX_MAXSPLITS = 64;
+
+// Merge of the splits and out = o W_uv^T for 16 rows, one head, 32 value columns.  Eight warps = 4 pieces of 8 columns x 2
+// halves of the latent.  A lane holds 16 contiguous bytes of a weight row per 32-wide step and takes the same columns of
+// two rows of the merged sums from shared memory: any order of the inner index serves, as long as both sides use it.
+__global__ void __launch_bounds__(256)
+latent_expand_mma_kernel(const ExpandParams p) {
+    extern __shared__ __align__(16) uint8_t smem[];
+    __shared__ float s_w[16][EX_MAXSPLITS], s_part[8][16][9];
+    __nv_bfloat16* so = reinterpret_cast<__nv_bfloat16*>(smem);          // [16][steps * 32 + 8]
+    const int ldo = p.steps * 32 + 8;
+    const int vt = blockIdx.x % p.v_tiles, h = blockIdx.x / p.v_tiles % p.H;
+    const int b0 = blockIdx.x / (p.v_tiles * p.H) * 16, nb = min(16, p.B - b0);
+    const int warp = threadIdx.x / 32, lane = threadIdx.x % 32, g = lane / 4, j = lane % 4;
+    const int half = (p.steps + 1) / 2, s0 = warp / 4 * half, s1 = min(p.steps, s0 + half);
+    const int v = vt * EX_V + warp % 4 * 8 + g;
+    const __nv_bfloat16* w = p.wuv + ((int64_t)h * p.vdim + v) * p.kv_ld + j * 8;
+    uint4 wv[EX_BATCH];
+    auto load_w = [&](int s) {
+#pragma unroll
+        for (int i = 0; i < EX_BATCH; ++i) {
+            wv[i] = make_uint4(0, 0, 0, 0);
+            if (s + i < s1 && v < p.vdim && (s + i) * 32 + j * 8 < p.kv_ld) wv[i] = __ldg(reinterpret_cast<const uint4*>(w + (s + i) * 32));
+        }
+    };
+    load_w(s0);
+    grid_dependency_wait();
+    grid_launch_dependents();
+    // a row's weights of its splits
+    for (int b = warp; b < 16; b += 8) {
+        const float* l = p.lse + ((int64_t)(b0 + b) * p.H + h) * p.splits;
+        float x0 = -INFINITY, x1 = -INFINITY;
+        if (b < nb) {
+            if (lane < p.splits) x0 = l[lane];
+            if (lane + 32 < p.splits) x1 = l[lane + 32];
+        }
+        // fmaxf drops a NaN (a split that gave up): the sum below keeps it
+        float m = fmaxf(x0, x1);
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+        const float e0 = m == -INFINITY ? 0.f : expf(x0 - m), e1 = m == -INFINITY ? 0.f : expf(x1 - m);
+        float s = e0 + e1;
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+        const float inv = s == 0.f ? 0.f : 1.f / s;
+        if (lane < p.splits) s_w[b][lane] = e0 * inv;
+        if (lane + 32 < p.splits) s_w[b][lane + 32] = e1 * inv;
+    }
+    __syncthreads();
+    const int pieces = p.steps * 8;                                       // of 4 columns
+    for (int i = threadIdx.x; i < 16 * pieces; i += 256) {
+        const int b = i / pieces, c = i % pieces * 4;
+        float acc[4] = {0.f, 0.f, 0.f, 0.f};
+        if (b < nb && c < p.kv_ld) {
+            const float* src = p.partial + ((int64_t)(b0 + b) * p.H + h) * p.splits * p.kv_ld + c;
+#pragma unroll 8
+            for (int s = 0; s < p.splits; ++s) {
+                const float4 f = *reinterpret_cast<const float4*>(src + (int64_t)s * p.kv_ld);
+                const float x = s_w[b][s];
+                acc[0] = fmaf(f.x, x, acc[0]);
+                acc[1] = fmaf(f.y, x, acc[1]);
+                acc[2] = fmaf(f.z, x, acc[2]);
+                acc[3] = fmaf(f.w, x, acc[3]);
+            }
+        }
+        store4(so + b * ldo + c, acc);
+    }
+    __syncthreads();
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+    for (int s = s0; s < s1; s += EX_BATCH) {
+        if (s > s0) load_w(s);
+#pragma unroll
+        for (int i = 0; i < EX_BATCH; ++i) {
+            if (s + i >= s1) break;
+            const uint4 lo = *reinterpret_cast<const uint4*>(so + g * ldo + (s + i) * 32 + j * 8);
+            const uint4 hi = *reinterpret_cast<const uint4*>(so + (g + 8) * ldo + (s + i) * 32 + j * 8);
+            mma_bf16_16816(acc, lo.x, hi.x, lo.y, hi.y, wv[i].x, wv[i].y);
+            mma_bf16_16816(acc, lo.z, hi.z, lo.w, hi.w, wv[i].z, wv[i].w);
+        }
+    }
+    s_part[warp][g][2 * j] = acc[0];
+    s_part[warp][g][2 * j + 1] = acc[1];
+    s_part[warp][g + 8][2 * j] = acc[2];
+    s_part[warp][g + 8][2 * j + 1] = acc[3];
+    __syncthreads();
+    for (int i = threadIdx.x; i < 16 * EX_V; i += 256) {
+        const int b = i / EX_V, c = i % EX_V, col = vt * EX_V + c;
+        if (b < nb && col < p.vdim)
+            p.out[(b0 + b) * p.out_ld + h * p.vdim + col] = __float2bfloat16(s_part[c / 8][b][c % 8] + s_part[4 + c / 8][b][c % 8]);
+    }
+    if (h == p.H - 1 && vt == 0)                                          // the padding columns behind the last head
+        for (int b = 0; b < nb; ++b)
+            for (int i = p.H * p.vdim + threadIdx.x; i < p.out_ld; i += 256) p.out[(b0 + b) * p.out_ld + i] = __float2bfloat16(0.f);
+}
+
+bool latent_expand_mma(const float* partial, const float* lse, int splits, const void* wuv, void* out, int64_t out_ld, int B, int H,
+                       int vdim, int kv_ld, cudaStream_t st) {
+    const int steps = (kv_ld + 31) / 32;
+    const size_t smem = (size_t)16 * (steps * 32 + 8) * 2;
+    if (splits > EX_MAXSPLITS || smem > 32 * 1024 || ((reinterpret_cast<uintptr_t>(wuv) | reinterpret_cast<uintptr_t>(partial)) & 15)) return false;
+    ExpandParams p{partial, lse, static_cast<const __nv_bfloat16*>(wuv), static_cast<__nv_bfloat16*>(out), out_ld, splits, B, H, vdim,
+                   kv_ld, (vdim + EX_V - 1) / EX_V, steps};
+    launch_dependent(latent_expand_mma_kernel, (unsigned)(p.v_tiles * H * ((B + 15) / 16)), 256, smem, st, p);
+    return true;
 }
 
 }  // namespace bn

@@ -57,6 +57,11 @@ template <> struct ConvVec<__nv_bfloat16, 2> {
     }
 };
 
+template <> struct ConvVec<__nv_bfloat16, 4> {
+    static __device__ __forceinline__ void load(const __nv_bfloat16* p, float (&v)[4]) { load4(p, v); }
+    static __device__ __forceinline__ void store(__nv_bfloat16* p, const float (&v)[4]) { store4(p, v); }
+};
+
 // silu for the bf16 path: its result is rounded to bf16, so the fast exponential is far more exact than needed
 template <typename T> __device__ __forceinline__ float conv_silu_f(float z) { return silu_exact(z); }
 template <> __device__ __forceinline__ float conv_silu_f<__nv_bfloat16>(float z) { return activation_fast(BN_ACT_SILU, z); }
@@ -109,9 +114,8 @@ conv_step_kernel(const ConvParams p) {
             else if (pos0 + t >= 0) V::load(ring + (int64_t)((pos0 + t) % taps) * p.C, hist[k]);
         }
     T* out = static_cast<T*>(p.xbc) + (int64_t)b * p.S * p.xbc_ld + c;
-    for (int t = t0; t < t1; ++t) {
-        float v[VEC], y[VEC];
-        V::load(in + (int64_t)t * p.proj_ld + c, v);
+    auto token = [&](int t, const float (&v)[VEC]) {
+        float y[VEC];
 #pragma unroll
         for (int e = 0; e < VEC; ++e) {
             float s = fmaf(v[e], w[0][e], bias[e]);
@@ -127,6 +131,20 @@ conv_step_kernel(const ConvParams p) {
             for (int e = 0; e < VEC; ++e) hist[k][e] = hist[k - 1][e];
 #pragma unroll
         for (int e = 0; e < VEC; ++e) hist[0][e] = v[e];
+    };
+    constexpr int AHEAD = 8;                           // tokens whose loads are in flight together
+    int t = t0;
+    for (; t + AHEAD <= t1; t += AHEAD) {
+        float v[AHEAD][VEC];
+#pragma unroll
+        for (int a = 0; a < AHEAD; ++a) V::load(in + (int64_t)(t + a) * p.proj_ld + c, v[a]);
+#pragma unroll
+        for (int a = 0; a < AHEAD; ++a) token(t + a, v[a]);
+    }
+    for (; t < t1; ++t) {
+        float v[VEC];
+        V::load(in + (int64_t)t * p.proj_ld + c, v);
+        token(t, v);
     }
 }
 
@@ -234,7 +252,7 @@ mamba2_step_kernel(const StepParams p) {
     const int v0 = pt * p.p_per_block, nv = min(p.p_per_block, p.P - v0);
     float* state = p.state + (((int64_t)slot * p.H + h) * p.P + v0) * p.N;
     // the state of this warp's first values is requested before the convolution
-    constexpr int U = 4;                               // values in flight per warp
+    constexpr int U = VEC == 4 ? 64 / R : 4;           // values in flight per warp
     float s[U][R];
     auto load_state = [&](int v, float (&d)[R]) {
         const float* sv = state + (int64_t)v * p.N;
@@ -341,7 +359,7 @@ gated_norm_kernel(const GatedNormParams p) {
                         float z4[4];
                         load4(z + i, z4);
 #pragma unroll
-                        for (int e = 0; e < 4; ++e) v[k][e] *= silu_exact(z4[e]);
+                        for (int e = 0; e < 4; ++e) v[k][e] *= conv_silu_f<T>(z4[e]);
                     }
 #pragma unroll
                     for (int e = 0; e < 4; ++e) s = fmaf(v[k][e], v[k][e], s);
@@ -349,7 +367,7 @@ gated_norm_kernel(const GatedNormParams p) {
             }
         } else {
             for (int i = threadIdx.x; i < n; i += GN_THREADS) {
-                const float q = to_f(y[i]) * (z ? silu_exact(to_f(z[i])) : 1.f);
+                const float q = to_f(y[i]) * (z ? conv_silu_f<T>(to_f(z[i])) : 1.f);
                 part_buf[i] = q;
                 s = fmaf(q, q, s);
             }
@@ -458,10 +476,13 @@ extern "C" int bn_mamba2_conv(const void* proj, int64_t proj_ld, const float* co
     ConvParams p{proj, conv_w, conv_b, dt_bias, a_log, ring, seq_ids, positions, xbc, dt, a, proj_ld, xbc_ld, B, S, C, H, taps, inner};
     if ((long long)B * ((S + CV_TOK - 1) / CV_TOK) > 65535) return fail(BN_ERR_UNSUPPORTED, "%s: B=%d x S=%d too large", what, B, S);
     cudaStream_t st = as_stream(stream);
+    const bool fours = C % 4 == 0 && inner % 4 == 0 && proj_ld % 4 == 0 && xbc_ld % 4 == 0 && taps == 4 &&
+                       ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(ring) | reinterpret_cast<uintptr_t>(xbc)) & 7) == 0;
     const bool pairs = C % 2 == 0 && inner % 2 == 0 && proj_ld % 2 == 0 && xbc_ld % 2 == 0 &&
                        ((reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(ring) | reinterpret_cast<uintptr_t>(xbc)) & 3) == 0;
     int rc;
     if (dtype == 0) rc = conv_launch<float, 1>(p, st);
+    else if (fours) rc = conv_launch<__nv_bfloat16, 4>(p, st);
     else if (pairs) rc = conv_launch<__nv_bfloat16, 2>(p, st);
     else rc = conv_launch<__nv_bfloat16, 1>(p, st);
     if (rc) return rc;

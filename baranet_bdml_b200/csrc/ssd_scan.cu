@@ -12,7 +12,8 @@
 // CTA = (sequence, head, slice of 16 W values), W warps; warp w owns 16 values: their state as MMA accumulators
 // (16 x N fp32), the outputs of all 64 tokens for them.  An accumulator fragment of (value, state) is, register for
 // register, the B fragment of (state, value), so S enters S^T C without leaving the registers.  The 64 x 64 matrix of the
-// first sum is shared: the warps take its row blocks in turn and leave its two bf16 parts in shared memory.
+// first sum is shared: the warps take its row blocks in turn and leave its two bf16 parts in shared memory, only the blocks
+// on and below the diagonal (55 KB and 128 registers a thread: four CTAs per SM).
 #include "common.cuh"
 #include "hybrid.cuh"
 #include "mamba2.cuh"
@@ -22,7 +23,13 @@ namespace bn {
 using namespace ptx;
 
 constexpr int SD_Q = 64;                       // tokens per chunk
-constexpr int SD_LDM = SD_Q + 8;               // row stride of the 64 x 64 matrix, elements
+constexpr int SD_MBLOCKS = 10;                 // 16 x 16 blocks on and below the diagonal of the 64 x 64 matrix
+
+// Element offset of row r, columns 8 c .. 8 c + 7 (c = 0, 1) of block (mb, kb): blocks are packed, a row is 32 bytes, and
+// rows 4-7 of eight swap their halves, so that eight rows of one half lie in different banks.
+__device__ __forceinline__ int sd_m_offset(int mb, int kb, int r, int c) {
+    return (mb * (mb + 1) / 2 + kb) * 256 + r * 16 + ((c ^ (r >> 2 & 1)) << 3);
+}
 
 __device__ __forceinline__ void split_bf16(float a, float b, uint32_t& hi, uint32_t& lo) {
     hi = pack_bf16(a, b);
@@ -31,7 +38,7 @@ __device__ __forceinline__ void split_bf16(float a, float b, uint32_t& hi, uint3
 
 // NP: N rounded up to a multiple of 16 that the kernel is built for; columns N .. NP - 1 are zeros
 template <int NP>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(128, 4)
 ssd_scan_kernel(const SsmScanParams p, int slices) {
     constexpr int LDN = NP + 8;                // row stride of the B and C tiles, elements
     extern __shared__ __align__(16) uint8_t smem[];
@@ -39,9 +46,9 @@ ssd_scan_kernel(const SsmScanParams p, int slices) {
     const int PW = W * 16, LDX = PW + 8;
     __nv_bfloat16* sB = reinterpret_cast<__nv_bfloat16*>(smem);          // [64][LDN]
     __nv_bfloat16* sC = sB + SD_Q * LDN;                                 // [64][LDN]
-    __nv_bfloat16* sMh = sC + SD_Q * LDN;                                // [64][SD_LDM], high and low parts
-    __nv_bfloat16* sMl = sMh + SD_Q * SD_LDM;
-    __nv_bfloat16* sX = sMl + SD_Q * SD_LDM;                             // [64][LDX]
+    __nv_bfloat16* sMh = sC + SD_Q * LDN;                                // packed blocks, high and low parts
+    __nv_bfloat16* sMl = sMh + SD_MBLOCKS * 256;
+    __nv_bfloat16* sX = sMl + SD_MBLOCKS * 256;                          // [64][LDX]
     float* s_cum = reinterpret_cast<float*>(sX + SD_Q * LDX);            // [64] c_i
     float* s_dt = s_cum + SD_Q;                                          // [64]
     float* s_w = s_dt + SD_Q;                                            // [64] e^{c_last - c_j} dt_j
@@ -141,64 +148,78 @@ ssd_scan_kernel(const SsmScanParams p, int slices) {
                 const float m10 = q0 <= i1 ? acc[t][2] * __expf(c1 - e0) * d0 : 0.f, m11 = q1 <= i1 ? acc[t][3] * __expf(c1 - e1) * d1 : 0.f;
                 uint32_t hi, lo;
                 split_bf16(m00, m01, hi, lo);
-                *reinterpret_cast<uint32_t*>(sMh + i0 * SD_LDM + q0) = hi;
-                *reinterpret_cast<uint32_t*>(sMl + i0 * SD_LDM + q0) = lo;
+                const int o0 = sd_m_offset(mb, t / 2, g, t % 2) + 2 * j, o1 = sd_m_offset(mb, t / 2, g + 8, t % 2) + 2 * j;
+                *reinterpret_cast<uint32_t*>(sMh + o0) = hi;
+                *reinterpret_cast<uint32_t*>(sMl + o0) = lo;
                 split_bf16(m10, m11, hi, lo);
-                *reinterpret_cast<uint32_t*>(sMh + i1 * SD_LDM + q0) = hi;
-                *reinterpret_cast<uint32_t*>(sMl + i1 * SD_LDM + q0) = lo;
+                *reinterpret_cast<uint32_t*>(sMh + o1) = hi;
+                *reinterpret_cast<uint32_t*>(sMl + o1) = lo;
             }
         }
         __syncthreads();
-        // ---- outputs of this warp's 16 values, 16 tokens at a time
+        // ---- outputs of this warp's 16 values
         __nv_bfloat16* gy = static_cast<__nv_bfloat16*>(p.y) + ((int64_t)b * p.S + t0) * p.y_ld + h * p.P + v0;
-#pragma unroll 1
-        for (int mb = 0; mb < SD_Q / 16; ++mb) {
-            float y0[4] = {0.f, 0.f, 0.f, 0.f}, y1[4] = {0.f, 0.f, 0.f, 0.f};     // values 0-7 and 8-15 of the warp
-            const uint32_t ca = uC + ((mb * 16 + lane % 16) * LDN + (lane / 16) * 8) * 2;
+        float y[SD_Q / 16][2][4];                         // [16 tokens][values 0-7 | 8-15 of the warp]
 #pragma unroll
-            for (int ks = 0; ks < NP / 16; ++ks) {        // C S: the state's two parts, straight from its accumulators
-                uint32_t a0, a1, a2, a3, h0, h1, h2, h3, l0, l1, l2, l3;
-                ldmatrix_x4(ca + ks * 32, a0, a1, a2, a3);
-                split_bf16(st[2 * ks][0], st[2 * ks][1], h0, l0);
-                split_bf16(st[2 * ks + 1][0], st[2 * ks + 1][1], h1, l1);
-                split_bf16(st[2 * ks][2], st[2 * ks][3], h2, l2);
-                split_bf16(st[2 * ks + 1][2], st[2 * ks + 1][3], h3, l3);
-                mma_bf16_16816(y0, a0, a1, a2, a3, h0, h1);
-                mma_bf16_16816(y0, a0, a1, a2, a3, l0, l1);
-                mma_bf16_16816(y1, a0, a1, a2, a3, h2, h3);
-                mma_bf16_16816(y1, a0, a1, a2, a3, l2, l3);
+        for (int mb = 0; mb < SD_Q / 16; ++mb)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) y[mb][0][e] = y[mb][1][e] = 0.f;
+        const uint32_t ca = uC + ((lane % 16) * LDN + (lane / 16) * 8) * 2;
+#pragma unroll
+        for (int ks = 0; ks < NP / 16; ++ks) {            // C S: the state's two parts, straight from its accumulators
+            uint32_t h0, h1, h2, h3, l0, l1, l2, l3;
+            split_bf16(st[2 * ks][0], st[2 * ks][1], h0, l0);
+            split_bf16(st[2 * ks + 1][0], st[2 * ks + 1][1], h1, l1);
+            split_bf16(st[2 * ks][2], st[2 * ks][3], h2, l2);
+            split_bf16(st[2 * ks + 1][2], st[2 * ks + 1][3], h3, l3);
+#pragma unroll
+            for (int mb = 0; mb < SD_Q / 16; ++mb) {
+                uint32_t a0, a1, a2, a3;
+                ldmatrix_x4(ca + (mb * 16 * LDN + ks * 16) * 2, a0, a1, a2, a3);
+                mma_bf16_16816(y[mb][0], a0, a1, a2, a3, h0, h1);
+                mma_bf16_16816(y[mb][1], a0, a1, a2, a3, h2, h3);
+                mma_bf16_16816(y[mb][0], a0, a1, a2, a3, l0, l1);
+                mma_bf16_16816(y[mb][1], a0, a1, a2, a3, l2, l3);
             }
-            const int i0 = mb * 16 + g, i1 = i0 + 8;
-            const float e0 = expf(s_cum[i0]), e1 = expf(s_cum[i1]);
-            y0[0] *= e0; y0[1] *= e0; y0[2] *= e1; y0[3] *= e1;
-            y1[0] *= e0; y1[1] *= e0; y1[2] *= e1; y1[3] *= e1;
-            const uint32_t ma = ((mb * 16 + lane % 16) * SD_LDM + (lane / 16) * 8) * 2;
-            for (int ks = 0; ks <= mb; ++ks) {            // M x
-                uint32_t b0, b1, b2, b3, a0, a1, a2, a3;
-                ldmatrix_x4_trans(uX + ((ks * 16 + lane % 16) * LDX + warp * 16 + (lane / 16) * 8) * 2, b0, b1, b2, b3);
-                ldmatrix_x4(uMh + ma + ks * 32, a0, a1, a2, a3);
-                mma_bf16_16816(y0, a0, a1, a2, a3, b0, b1);
-                mma_bf16_16816(y1, a0, a1, a2, a3, b2, b3);
-                ldmatrix_x4(uMl + ma + ks * 32, a0, a1, a2, a3);
-                mma_bf16_16816(y0, a0, a1, a2, a3, b0, b1);
-                mma_bf16_16816(y1, a0, a1, a2, a3, b2, b3);
+        }
+#pragma unroll
+        for (int mb = 0; mb < SD_Q / 16; ++mb) {
+            const float e0 = expf(s_cum[mb * 16 + g]), e1 = expf(s_cum[mb * 16 + g + 8]);
+#pragma unroll
+            for (int q = 0; q < 2; ++q) { y[mb][q][0] *= e0; y[mb][q][1] *= e0; y[mb][q][2] *= e1; y[mb][q][3] *= e1; }
+        }
+#pragma unroll
+        for (int ks = 0; ks < SD_Q / 16; ++ks) {          // M x
+            uint32_t b0, b1, b2, b3;
+            ldmatrix_x4_trans(uX + ((ks * 16 + lane % 16) * LDX + warp * 16 + (lane / 16) * 8) * 2, b0, b1, b2, b3);
+#pragma unroll
+            for (int mb = ks; mb < SD_Q / 16; ++mb) {
+                uint32_t a0, a1, a2, a3, d0, d1, d2, d3;
+                const uint32_t o = sd_m_offset(mb, ks, lane % 16, lane / 16) * 2;
+                ldmatrix_x4(uMh + o, a0, a1, a2, a3);
+                ldmatrix_x4(uMl + o, d0, d1, d2, d3);
+                mma_bf16_16816(y[mb][0], a0, a1, a2, a3, b0, b1);
+                mma_bf16_16816(y[mb][1], a0, a1, a2, a3, b2, b3);
+                mma_bf16_16816(y[mb][0], d0, d1, d2, d3, b0, b1);
+                mma_bf16_16816(y[mb][1], d0, d1, d2, d3, b2, b3);
             }
-            // + D x, rounded; y0[0..1]: token i0, values 2 j, 2 j + 1 of the warp
+        }
+        // + D x, rounded; a lane has tokens g and g + 8 of each 16 and values 2 j, 2 j + 1 of each 8
+#pragma unroll
+        for (int mb = 0; mb < SD_Q / 16; ++mb)
 #pragma unroll
             for (int half = 0; half < 2; ++half) {
-                const int i = half ? i1 : i0;
+                const int i = mb * 16 + g + half * 8;
 #pragma unroll
                 for (int q = 0; q < 2; ++q) {
                     const int v = warp * 16 + q * 8 + 2 * j;
                     if (i < nt && v < nv) {
                         const uint32_t x2 = *reinterpret_cast<const uint32_t*>(sX + i * LDX + v);
-                        const float ya = (q ? y1 : y0)[half * 2], yb = (q ? y1 : y0)[half * 2 + 1];
                         *reinterpret_cast<uint32_t*>(gy + (int64_t)i * p.y_ld + v) =
-                            pack_bf16(fmaf(D, bf16_lo(x2), ya), fmaf(D, bf16_hi(x2), yb));
+                            pack_bf16(fmaf(D, bf16_lo(x2), y[mb][q][half * 2]), fmaf(D, bf16_hi(x2), y[mb][q][half * 2 + 1]));
                     }
                 }
             }
-        }
         // ---- state: S^T (values x N) = e^{c_last} S^T + (w x)^T B
         const float decay = expf(s_cum[SD_Q - 1]);
 #pragma unroll
@@ -223,8 +244,8 @@ ssd_scan_kernel(const SsmScanParams p, int slices) {
                 uint32_t b0, b1, b2, b3;                  // rows = tokens, columns = state: transposing load
                 ldmatrix_x4_trans(uB + ((ks * 16 + lane % 16) * LDN + t2 * 16 + (lane / 16) * 8) * 2, b0, b1, b2, b3);
                 mma_bf16_16816(st[2 * t2], h0, h1, h2, h3, b0, b1);
-                mma_bf16_16816(st[2 * t2], l0, l1, l2, l3, b0, b1);
                 mma_bf16_16816(st[2 * t2 + 1], h0, h1, h2, h3, b2, b3);
+                mma_bf16_16816(st[2 * t2], l0, l1, l2, l3, b0, b1);
                 mma_bf16_16816(st[2 * t2 + 1], l0, l1, l2, l3, b2, b3);
             }
         }
@@ -246,7 +267,7 @@ bool ssd_scan_ok(const SsmScanParams& p) {
 template <int NP>
 static int ssd_launch(const SsmScanParams& p, int W, cudaStream_t st) {
     const int PW = W * 16, slices = (p.P + PW - 1) / PW;
-    const size_t smem = (size_t)(2 * SD_Q * (NP + 8) + 2 * SD_Q * SD_LDM + SD_Q * (PW + 8)) * 2 + 3 * SD_Q * 4;
+    const size_t smem = (size_t)(2 * SD_Q * (NP + 8) + 2 * SD_MBLOCKS * 256 + SD_Q * (PW + 8)) * 2 + 3 * SD_Q * 4;
     int dev = 0;
     cudaGetDevice(&dev);
     static thread_local int configured_dev = -1;

@@ -28,7 +28,7 @@ def config(layers, width, vocab, side, loop=None, eps=1e-5):
 
 CASES = {
     # nothing a multiple of 8, a loop from the first layer on, a feed-forward behind a recurrence and none behind attention
-    "odd": config([layer(mamba(), 52), layer(attention()), layer(mamba(heads=5, vdim=7, state=9, groups=1, conv=4, norm_groups=5)),
+    "odd": config([layer(mamba(), 52), layer(attention()), layer(mamba(heads=5, vdim=19, state=9, groups=1, conv=4, norm_groups=5)),
                    layer(attention(heads=2, dim=10, rot_dim=6, vdim=11, q_rank=13, kv_rank=17, window=19, base=500.0), 31)],
                   width=74, vocab=101, side=12, loop=(0, 3, 3)),
     # the sizes that the tensor-core kernels take, two kinds of attention

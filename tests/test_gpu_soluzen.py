@@ -1,7 +1,7 @@
 """Soluzen on the GPU against the plain fp64 restatement (oracle/ref_soluzen.py): every mechanism alone, whole prompts,
 portions, one-token steps, slots used again, and generation through the framework's entry point.
 
-fp32 gate 1e-4, bf16 gate 4e-2, both of the root mean square of the expected rows.  A random model amplifies rounding at a
+fp32 gate 1e-4, bf16 gate 5e-2, both of the root mean square of the expected rows.  A random model amplifies rounding at a
 few positions (rounding the restatement's own activations to bf16 moves single rows by up to 0.2), so whole models in bf16
 are held to the gate at nine rows in ten and to ten times the gate at every row; a single mechanism, and everything in
 fp32, is held to its gate at every row.  `test_the_gates_see_planted_mistakes` plants mistakes in the restatement and
@@ -20,7 +20,7 @@ from oracle import ref_soluzen as R
 
 pytestmark = pytest.mark.gpu
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
-GATE = {torch.float32: 1e-4, torch.bfloat16: 4e-2}
+GATE = {torch.float32: 1e-4, torch.bfloat16: 5e-2}
 DTYPES = pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16], ids=["f32", "bf16"])
 
 
