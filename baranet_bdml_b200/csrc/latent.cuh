@@ -34,7 +34,7 @@ int latent_decode_mma(const LatentDecodeParams& p, cudaStream_t stream);
 // bf16 forms of bn_latent_absorb_q and bn_latent_expand_out; false when the sizes or alignments are not theirs
 bool latent_absorb_mma(const void* q, int64_t q_ld, const void* wuk, const double* freq, const int32_t* positions, void* q_abs, int B,
                        int H, int dim, int rot, int kv_ld, int rot_ld, cudaStream_t stream);
-bool latent_expand_mma(const float* partial, const float* lse, int splits, const void* wuv, void* out, int64_t out_ld, int B, int H,
+bool latent_expand_mma(float* partial, const float* lse, int splits, const void* wuv, void* out, int64_t out_ld, int B, int H,
                        int vdim, int kv_ld, cudaStream_t stream);
 
 }  // namespace bn

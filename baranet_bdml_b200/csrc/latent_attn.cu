@@ -134,6 +134,105 @@ latent_prep_kernel(const LatentPrepParams p) {
     }
 }
 
+// The same with a row held in registers: cq_ld <= 512 NQ, kv_ld <= 512 NK, ranks and strides multiples of 4, rows aligned,
+// rot <= 2 LP_THREADS.
+// Everything a row needs is requested before the sums.
+template <typename T, int NQ, int NK>
+__global__ void __launch_bounds__(LP_THREADS)
+latent_prep_regs_kernel(const LatentPrepParams p) {
+    __shared__ float sh[2][LP_THREADS / 32];
+    const int tid = threadIdx.x;
+    float wq[NQ][4], wk[NK][4];                          // the norms' weights stay for all rows of the block
+#pragma unroll
+    for (int k = 0; k < NQ; ++k)
+        if ((tid + k * LP_THREADS) * 4 < p.q_rank) load4(p.q_norm + (tid + k * LP_THREADS) * 4, wq[k]);
+#pragma unroll
+    for (int k = 0; k < NK; ++k)
+        if ((tid + k * LP_THREADS) * 4 < p.kv_rank) load4(p.kv_norm + (tid + k * LP_THREADS) * 4, wk[k]);
+    ptx::grid_dependency_wait();
+    ptx::grid_launch_dependents();
+    for (int r = blockIdx.x; r < p.rows; r += gridDim.x) {
+        const int b = r / p.S, s = r - b * p.S;
+        const T* in = static_cast<const T*>(p.proj) + (int64_t)r * p.proj_ld;
+        const T* rin = in + p.q_rank + p.kv_rank;
+        float vq[NQ][4], vk[NK][4], u = 0.f, v = 0.f;
+#pragma unroll
+        for (int k = 0; k < NQ; ++k) {
+            vq[k][0] = vq[k][1] = vq[k][2] = vq[k][3] = 0.f;
+            if ((tid + k * LP_THREADS) * 4 < p.q_rank) load4(in + (tid + k * LP_THREADS) * 4, vq[k]);
+        }
+#pragma unroll
+        for (int k = 0; k < NK; ++k) {
+            vk[k][0] = vk[k][1] = vk[k][2] = vk[k][3] = 0.f;
+            if ((tid + k * LP_THREADS) * 4 < p.kv_rank) load4(in + p.q_rank + (tid + k * LP_THREADS) * 4, vk[k]);
+        }
+        if (2 * tid < p.rot) { u = to_f(rin[2 * tid]); v = to_f(rin[2 * tid + 1]); }
+        const int pos = p.positions[b] + s, slot = p.seq_ids ? p.seq_ids[b] : b;
+        float sq = 0.f, sk = 0.f;
+#pragma unroll
+        for (int k = 0; k < NQ; ++k)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) sq = fmaf(vq[k][e], vq[k][e], sq);
+#pragma unroll
+        for (int k = 0; k < NK; ++k)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) sk = fmaf(vk[k][e], vk[k][e], sk);
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            sq += __shfl_xor_sync(0xffffffffu, sq, o);
+            sk += __shfl_xor_sync(0xffffffffu, sk, o);
+        }
+        __syncthreads();
+        if (tid % 32 == 0) { sh[0][tid / 32] = sq; sh[1][tid / 32] = sk; }
+        __syncthreads();
+        sq = sk = 0.f;
+#pragma unroll
+        for (int w = 0; w < LP_THREADS / 32; ++w) { sq += sh[0][w]; sk += sh[1][w]; }
+        const float inv_q = rsqrtf(sq / (float)p.q_rank + p.eps), inv_k = rsqrtf(sk / (float)p.kv_rank + p.eps);
+        T* cq = static_cast<T*>(p.cq) + (int64_t)r * p.cq_ld;
+        const int64_t out_row = (int64_t)b * p.rows_per_seq + p.row_offset + s;
+        T* c = p.c ? static_cast<T*>(p.c) + out_row * p.kv_ld : nullptr;
+        T* kr = p.krot ? static_cast<T*>(p.krot) + out_row * p.rot_ld : nullptr;
+        T* ring = nullptr;
+        if (p.ring && s >= p.S - p.ring_tokens)
+            ring = static_cast<T*>(p.ring) + ((int64_t)slot * p.ring_tokens + pos % p.ring_tokens) * (p.kv_ld + p.rot_ld);
+        const float zero[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int k = 0; k < NQ; ++k) {
+            const int i = (tid + k * LP_THREADS) * 4;
+            if (i < p.q_rank) {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) vq[k][e] = vq[k][e] * inv_q * wq[k][e];
+                store4(cq + i, vq[k]);
+            } else if (i < p.cq_ld) store4(cq + i, zero);
+        }
+#pragma unroll
+        for (int k = 0; k < NK; ++k) {
+            const int i = (tid + k * LP_THREADS) * 4;
+            if (i < p.kv_rank) {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) vk[k][e] = vk[k][e] * inv_k * wk[k][e];
+                if (c) store4(c + i, vk[k]);
+                if (ring) store4(ring + i, vk[k]);
+            } else if (i < p.kv_ld) {
+                if (c) store4(c + i, zero);
+                if (ring) store4(ring + i, zero);
+            }
+        }
+        if (2 * tid < p.rot_ld) {
+            T lo = from_f<T>(0.f), hi = lo;
+            if (2 * tid < p.rot) {
+                float cs, sn;
+                rotation(pos, p.freq[tid], &cs, &sn);
+                lo = from_f<T>(u * cs - v * sn);
+                hi = from_f<T>(v * cs + u * sn);
+            }
+            if (kr) { kr[2 * tid] = lo; kr[2 * tid + 1] = hi; }
+            if (ring) { ring[p.kv_ld + 2 * tid] = lo; ring[p.kv_ld + 2 * tid + 1] = hi; }
+        }
+    }
+}
+
 // the `n_old` tokens before the portion, out of the ring, to rows 0 .. n_old - 1 of each sequence's block of rows
 template <typename T>
 __global__ void __launch_bounds__(128)
@@ -482,9 +581,14 @@ extern "C" int bn_latent_prep(const void* proj, int64_t proj_ld, const float* q_
     const unsigned grid = (unsigned)(B * S < cap ? B * S : cap);
     const uintptr_t all = reinterpret_cast<uintptr_t>(proj) | reinterpret_cast<uintptr_t>(q_norm) | reinterpret_cast<uintptr_t>(kv_norm) |
                           reinterpret_cast<uintptr_t>(cq) | reinterpret_cast<uintptr_t>(c) | reinterpret_cast<uintptr_t>(ring);
+    const int kl = p.kv_ld;
     const bool vec = q_rank % 4 == 0 && kv_rank % 4 == 0 && proj_ld % 4 == 0 && cq_ld % 4 == 0 && (all & 15) == 0;
     if (dtype == 0 && vec) launch_dependent(latent_prep_kernel<float, 4>, grid, LP_THREADS, 0, as_stream(stream), p);
     else if (dtype == 0) launch_dependent(latent_prep_kernel<float, 1>, grid, LP_THREADS, 0, as_stream(stream), p);
+    else if (vec && cq_ld <= 1024 && kl <= 512 && rot <= 2 * LP_THREADS)
+        launch_dependent(latent_prep_regs_kernel<__nv_bfloat16, 2, 1>, grid, LP_THREADS, 0, as_stream(stream), p);
+    else if (vec && cq_ld <= 2048 && kl <= 1024 && rot <= 2 * LP_THREADS)
+        launch_dependent(latent_prep_regs_kernel<__nv_bfloat16, 4, 2>, grid, LP_THREADS, 0, as_stream(stream), p);
     else if (vec) launch_dependent(latent_prep_kernel<__nv_bfloat16, 4>, grid, LP_THREADS, 0, as_stream(stream), p);
     else launch_dependent(latent_prep_kernel<__nv_bfloat16, 1>, grid, LP_THREADS, 0, as_stream(stream), p);
     return launch_status(what);
@@ -617,7 +721,7 @@ extern "C" int bn_latent_decode(const void* q_abs, const void* ring, int num_slo
     return launch_status(what);
 }
 
-extern "C" int bn_latent_expand_out(const float* partial, const float* lse, int splits, const void* wuv, void* out, int64_t out_ld,
+extern "C" int bn_latent_expand_out(float* partial, const float* lse, int splits, const void* wuv, void* out, int64_t out_ld,
                                     int B, int H, int vdim, int kv_rank, int dtype, bn_stream_t stream) {
     const char* what = "bn_latent_expand_out";
     if (!partial || !lse || !wuv || !out) return fail(BN_ERR_INVALID_ARG, "%s: null pointer", what);

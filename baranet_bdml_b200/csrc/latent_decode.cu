@@ -12,7 +12,7 @@
 //   sum      warp w: an eighth of the latent's columns, all 64 rows
 // Softmax does not care about order, so the ring is walked in ROW order: row r holds position pos - (pos - r mod ring),
 // and a row whose position is outside the window (or was never written) gets weight zero.
-// A split's result is its normalised sum and log-sum-exp; bn_latent_expand_out merges the splits.
+// A split's result is its normalised sum and log-sum-exp; bn_latent_expand_out merges the splits (in place).
 // Waits are bounded: on expiry the CTA stops and leaves a NaN log-sum-exp, which surfaces as NaN logits.
 #include "common.cuh"
 #include "hybrid.cuh"
@@ -388,23 +388,78 @@ bool latent_absorb_mma(const void* q, int64_t q_ld, const void* wuk, const doubl
     return true;
 }
 
+// Merges a (row, head)'s splits into its split 0: a thread owns four columns of all splits, which it reads before it writes.
+constexpr int MG_MAXSPLITS = 64, MG_BATCH = 8;
+
+__global__ void __launch_bounds__(128)
+latent_merge_kernel(float* partial, const float* lse, int splits, int kv_ld) {
+    __shared__ float s_w[MG_MAXSPLITS];
+    grid_dependency_wait();
+    grid_launch_dependents();
+    float* base = partial + (int64_t)blockIdx.x * splits * kv_ld;
+    float4 f[MG_BATCH];
+    const int c0 = threadIdx.x * 4;
+    if (c0 < kv_ld) {
+#pragma unroll
+        for (int s = 0; s < MG_BATCH; ++s)
+            if (s < splits) f[s] = *reinterpret_cast<const float4*>(base + (int64_t)s * kv_ld + c0);
+    }
+    if (threadIdx.x < 32) {
+        const int lane = threadIdx.x;
+        const float* l = lse + (int64_t)blockIdx.x * splits;
+        const float x0 = lane < splits ? l[lane] : -INFINITY, x1 = lane + 32 < splits ? l[lane + 32] : -INFINITY;
+        float m = fmaxf(x0, x1);                 // drops a NaN (a split that gave up); the sum below keeps it
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+        const float e0 = m == -INFINITY ? 0.f : expf(x0 - m), e1 = m == -INFINITY ? 0.f : expf(x1 - m);
+        float t = e0 + e1;
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) t += __shfl_xor_sync(0xffffffffu, t, o);
+        const float inv = t == 0.f ? 0.f : 1.f / t;
+        if (lane < splits) s_w[lane] = e0 * inv;
+        if (lane + 32 < splits) s_w[lane + 32] = e1 * inv;
+    }
+    __syncthreads();
+    for (int c = c0; c < kv_ld; c += 512) {
+        float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+        for (int s0 = 0; s0 < splits; s0 += MG_BATCH) {
+            if (c > c0 || s0 > 0) {
+#pragma unroll
+                for (int s = 0; s < MG_BATCH; ++s)
+                    if (s0 + s < splits) f[s] = *reinterpret_cast<const float4*>(base + (int64_t)(s0 + s) * kv_ld + c);
+            }
+#pragma unroll
+            for (int s = 0; s < MG_BATCH; ++s)
+                if (s0 + s < splits) {
+                    const float x = s_w[s0 + s];
+                    o.x = fmaf(f[s].x, x, o.x);
+                    o.y = fmaf(f[s].y, x, o.y);
+                    o.z = fmaf(f[s].z, x, o.z);
+                    o.w = fmaf(f[s].w, x, o.w);
+                }
+        }
+        *reinterpret_cast<float4*>(base + c) = o;
+    }
+}
+
 struct ExpandParams {
-    const float *partial, *lse;
+    const float *sums, *lse;                             // sums: [B][H], `stride` floats apart
     const __nv_bfloat16* wuv;
     __nv_bfloat16* out;
-    int64_t out_ld;
-    int splits, B, H, vdim, kv_ld, v_tiles, steps;       // steps: 32-wide pieces of the latent, rounded up
+    int64_t out_ld, stride;
+    int B, H, vdim, kv_ld, v_tiles, steps;               // steps: 32-wide pieces of the latent, rounded up
 };
 
-constexpr int EX_V = 32, EX_BATCH = 8, EX_MAXSPLITS = 64;
+constexpr int EX_V = 32, EX_BATCH = 8;
 
-// Merge of the splits and out = o W_uv^T for 16 rows, one head, 32 value columns.  Eight warps = 4 pieces of 8 columns x 2
-// halves of the latent.  A lane holds 16 contiguous bytes of a weight row per 32-wide step and takes the same columns of
-// two rows of the merged sums from shared memory: any order of the inner index serves, as long as both sides use it.
+// out = o W_uv^T for 16 rows, one head, 32 value columns.  Eight warps = 4 pieces of 8 columns x 2 halves of the latent.  A
+// lane holds 16 contiguous bytes of a weight row per 32-wide step and takes the same columns of two rows of the sums from
+// shared memory: any order of the inner index serves, as long as both sides use it.  `lse` (an unmerged single split) is
+// looked at only for the mark of a split that gave up.
 __global__ void __launch_bounds__(256)
 latent_expand_mma_kernel(const ExpandParams p) {
     extern __shared__ __align__(16) uint8_t smem[];
-    __shared__ float s_w[16][EX_MAXSPLITS], s_part[8][16][9];
+    __shared__ float s_part[8][16][9];
     __nv_bfloat16* so = reinterpret_cast<__nv_bfloat16*>(smem);          // [16][steps * 32 + 8]
     const int ldo = p.steps * 32 + 8;
     const int vt = blockIdx.x % p.v_tiles, h = blockIdx.x / p.v_tiles % p.H;
@@ -424,44 +479,13 @@ latent_expand_mma_kernel(const ExpandParams p) {
     load_w(s0);
     grid_dependency_wait();
     grid_launch_dependents();
-    // a row's weights of its splits
-    for (int b = warp; b < 16; b += 8) {
-        const float* l = p.lse + ((int64_t)(b0 + b) * p.H + h) * p.splits;
-        float x0 = -INFINITY, x1 = -INFINITY;
-        if (b < nb) {
-            if (lane < p.splits) x0 = l[lane];
-            if (lane + 32 < p.splits) x1 = l[lane + 32];
-        }
-        // fmaxf drops a NaN (a split that gave up): the sum below keeps it
-        float m = fmaxf(x0, x1);
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
-        const float e0 = m == -INFINITY ? 0.f : expf(x0 - m), e1 = m == -INFINITY ? 0.f : expf(x1 - m);
-        float s = e0 + e1;
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
-        const float inv = s == 0.f ? 0.f : 1.f / s;
-        if (lane < p.splits) s_w[b][lane] = e0 * inv;
-        if (lane + 32 < p.splits) s_w[b][lane + 32] = e1 * inv;
-    }
-    __syncthreads();
     const int pieces = p.steps * 8;                                       // of 4 columns
+#pragma unroll 8
     for (int i = threadIdx.x; i < 16 * pieces; i += 256) {
         const int b = i / pieces, c = i % pieces * 4;
-        float acc[4] = {0.f, 0.f, 0.f, 0.f};
-        if (b < nb && c < p.kv_ld) {
-            const float* src = p.partial + ((int64_t)(b0 + b) * p.H + h) * p.splits * p.kv_ld + c;
-#pragma unroll 8
-            for (int s = 0; s < p.splits; ++s) {
-                const float4 f = *reinterpret_cast<const float4*>(src + (int64_t)s * p.kv_ld);
-                const float x = s_w[b][s];
-                acc[0] = fmaf(f.x, x, acc[0]);
-                acc[1] = fmaf(f.y, x, acc[1]);
-                acc[2] = fmaf(f.z, x, acc[2]);
-                acc[3] = fmaf(f.w, x, acc[3]);
-            }
-        }
-        store4(so + b * ldo + c, acc);
+        float x[4] = {0.f, 0.f, 0.f, 0.f};
+        if (b < nb && c < p.kv_ld) load4(p.sums + ((int64_t)(b0 + b) * p.H + h) * p.stride + c, x);
+        store4(so + b * ldo + c, x);
     }
     __syncthreads();
     float acc[4] = {0.f, 0.f, 0.f, 0.f};
@@ -483,21 +507,28 @@ latent_expand_mma_kernel(const ExpandParams p) {
     __syncthreads();
     for (int i = threadIdx.x; i < 16 * EX_V; i += 256) {
         const int b = i / EX_V, c = i % EX_V, col = vt * EX_V + c;
-        if (b < nb && col < p.vdim)
-            p.out[(b0 + b) * p.out_ld + h * p.vdim + col] = __float2bfloat16(s_part[c / 8][b][c % 8] + s_part[4 + c / 8][b][c % 8]);
+        if (b < nb && col < p.vdim) {
+            float y = s_part[c / 8][b][c % 8] + s_part[4 + c / 8][b][c % 8];
+            if (p.lse) {
+                const float l = p.lse[(int64_t)(b0 + b) * p.H + h];
+                if (l != l) y = l;
+            }
+            p.out[(b0 + b) * p.out_ld + h * p.vdim + col] = __float2bfloat16(y);
+        }
     }
     if (h == p.H - 1 && vt == 0)                                          // the padding columns behind the last head
         for (int b = 0; b < nb; ++b)
             for (int i = p.H * p.vdim + threadIdx.x; i < p.out_ld; i += 256) p.out[(b0 + b) * p.out_ld + i] = __float2bfloat16(0.f);
 }
 
-bool latent_expand_mma(const float* partial, const float* lse, int splits, const void* wuv, void* out, int64_t out_ld, int B, int H,
+bool latent_expand_mma(float* partial, const float* lse, int splits, const void* wuv, void* out, int64_t out_ld, int B, int H,
                        int vdim, int kv_ld, cudaStream_t st) {
     const int steps = (kv_ld + 31) / 32;
     const size_t smem = (size_t)16 * (steps * 32 + 8) * 2;
-    if (splits > EX_MAXSPLITS || smem > 32 * 1024 || ((reinterpret_cast<uintptr_t>(wuv) | reinterpret_cast<uintptr_t>(partial)) & 15)) return false;
-    ExpandParams p{partial, lse, static_cast<const __nv_bfloat16*>(wuv), static_cast<__nv_bfloat16*>(out), out_ld, splits, B, H, vdim,
-                   kv_ld, (vdim + EX_V - 1) / EX_V, steps};
+    if (splits > MG_MAXSPLITS || smem > 32 * 1024 || ((reinterpret_cast<uintptr_t>(wuv) | reinterpret_cast<uintptr_t>(partial)) & 15)) return false;
+    if (splits > 1) launch_dependent(latent_merge_kernel, (unsigned)(B * H), 128, 0, st, partial, lse, splits, kv_ld);
+    ExpandParams p{partial, splits > 1 ? nullptr : lse, static_cast<const __nv_bfloat16*>(wuv), static_cast<__nv_bfloat16*>(out), out_ld,
+                   (int64_t)splits * kv_ld, B, H, vdim, kv_ld, (vdim + EX_V - 1) / EX_V, steps};
     launch_dependent(latent_expand_mma_kernel, (unsigned)(p.v_tiles * H * ((B + 15) / 16)), 256, smem, st, p);
     return true;
 }

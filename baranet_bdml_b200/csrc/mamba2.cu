@@ -222,23 +222,43 @@ struct StepParams {
     int B, H, P, G, N, taps, p_per_block;
 };
 
-constexpr int ST_WARPS = 4;
+constexpr int ST_WARPS = 8;
 
-template <typename T>
-__device__ __forceinline__ float conv_one(const StepParams& p, const T* in, T* ring, int c, int C, int pos, bool write) {
-    const T cur = in[c];
-    float s = fmaf(to_f(cur), p.conv_w[(int64_t)c * p.taps + p.taps - 1], p.conv_b[c]);
-    for (int k = 1; k < p.taps; ++k)
-        if (pos - k >= 0) s = fmaf(to_f(ring[(int64_t)((pos - k) % p.taps) * C + c]), p.conv_w[(int64_t)c * p.taps + p.taps - 1 - k], s);
-    if (write) ring[(int64_t)(pos % p.taps) * C + c] = cur;
-    return round_to<T>(conv_silu_f<T>(s));
-}
+// What the convolution of one channel needs, loaded before any of it is used
+template <typename T, int TAPS>
+struct ConvLoads {
+    static constexpr int W = TAPS ? TAPS : CV_MAXTAPS;
+    T cur, back[W];
+    float w[W], bias;
+
+    __device__ __forceinline__ void load(const StepParams& p, const T* in, const T* ring, int c, int C, int pos) {
+        const int taps = TAPS ? TAPS : p.taps;
+        cur = in[c];
+        bias = __ldg(p.conv_b + c);
+        if (TAPS == 4) {
+            const float4 f = __ldg(reinterpret_cast<const float4*>(p.conv_w) + c);
+            w[0] = f.w; w[1] = f.z; w[2] = f.y; w[3] = f.x;
+        } else {
+#pragma unroll
+            for (int k = 0; k < W; ++k) w[k] = k < taps ? __ldg(p.conv_w + (int64_t)c * taps + taps - 1 - k) : 0.f;
+        }
+#pragma unroll
+        for (int k = 1; k < W; ++k)
+            back[k] = k < taps && pos >= k ? ring[(int64_t)((pos - k) % taps) * C + c] : from_f<T>(0.f);
+    }
+    __device__ __forceinline__ float result() const {
+        float s = fmaf(to_f(cur), w[0], bias);
+#pragma unroll
+        for (int k = 1; k < W; ++k) s = fmaf(to_f(back[k]), w[k], s);
+        return round_to<T>(conv_silu_f<T>(s));
+    }
+};
 
 // R = state elements per lane and value (N <= 32 R), VEC = 4: in pieces of 16 bytes (N a multiple of 128)
-template <typename T, int R, int VEC>
+template <typename T, int R, int VEC, int TAPS>
 __global__ void __launch_bounds__(ST_WARPS * 32)
 mamba2_step_kernel(const StepParams p) {
-    extern __shared__ float sm[];                      // B [N], C [N], x [p_per_block]
+    extern __shared__ float sm[];                      // B [N], C [N], x [p_per_block], silu(z) [p_per_block]
     ptx::grid_dependency_wait();
     ptx::grid_launch_dependents();
     const int warp = threadIdx.x / 32, lane = threadIdx.x % 32;
@@ -252,7 +272,7 @@ mamba2_step_kernel(const StepParams p) {
     const int v0 = pt * p.p_per_block, nv = min(p.p_per_block, p.P - v0);
     float* state = p.state + (((int64_t)slot * p.H + h) * p.P + v0) * p.N;
     // the state of this warp's first values is requested before the convolution
-    constexpr int U = VEC == 4 ? 64 / R : 4;           // values in flight per warp
+    constexpr int U = 4;                               // values in flight per warp
     float s[U][R];
     auto load_state = [&](int v, float (&d)[R]) {
         const float* sv = state + (int64_t)v * p.N;
@@ -269,16 +289,34 @@ mamba2_step_kernel(const StepParams p) {
 #pragma unroll
     for (int u = 0; u < U; ++u)
         if (warp + u * ST_WARPS < nv) load_state(warp + u * ST_WARPS, s[u]);
-    float *sB = sm, *sC = sm + p.N, *sx = sm + 2 * p.N;
-    // every block of a group computes the group's B and C; one of them writes their ring row
+    float *sB = sm, *sC = sm + p.N, *sx = sm + 2 * p.N, *sz = sx + p.p_per_block;
+    const float raw_dt = to_f(in[C + h]), dt_bias = p.dt_bias[h], a_log = p.a_log[h], D = p.D[h];
+    // Every block of a group computes the group's B and C; one of them writes their ring row.  Two channels per thread at
+    // a time, all loads of both before the arithmetic of either.
     const bool owner = pt == 0 && h % (p.H / p.G) == 0;
-    for (int i = threadIdx.x; i < 2 * p.N + nv; i += blockDim.x) {
-        if (i < p.N) sB[i] = conv_one(p, in, ring, inner + g * p.N + i, C, pos, owner);
-        else if (i < 2 * p.N) sC[i - p.N] = conv_one(p, in, ring, inner + GN + g * p.N + (i - p.N), C, pos, owner);
-        else sx[i - 2 * p.N] = conv_one(p, in, ring, h * p.P + v0 + (i - 2 * p.N), C, pos, true);
+    const int n_conv = 2 * p.N + nv, taps = TAPS ? TAPS : p.taps;
+    auto channel = [&](int i) {
+        return i < p.N ? inner + g * p.N + i : i < 2 * p.N ? inner + GN + g * p.N + (i - p.N) : h * p.P + v0 + (i - 2 * p.N);
+    };
+    constexpr int IT = TAPS ? 2 : 1;
+    for (int i0 = threadIdx.x; i0 < n_conv; i0 += IT * ST_WARPS * 32) {
+        ConvLoads<T, TAPS> ld[IT];
+#pragma unroll
+        for (int it = 0; it < IT; ++it) {
+            const int i = i0 + it * ST_WARPS * 32;
+            if (i < n_conv) ld[it].load(p, in, ring, channel(i), C, pos);
+        }
+#pragma unroll
+        for (int it = 0; it < IT; ++it) {
+            const int i = i0 + it * ST_WARPS * 32;
+            if (i < n_conv) {
+                sm[i] = ld[it].result();               // B, C and x lie one behind the other
+                if (owner || i >= 2 * p.N) ring[(int64_t)(pos % taps) * C + channel(i)] = ld[it].cur;
+            }
+        }
     }
-    const float dt = softplus_exact(to_f(in[C + h]) + p.dt_bias[h]);
-    const float decay = expf(-expf(p.a_log[h]) * dt), D = p.D[h];
+    for (int i = threadIdx.x; i < nv; i += ST_WARPS * 32) sz[i] = conv_silu_f<T>(to_f(row[h * p.P + v0 + i]));
+    const float dt = softplus_exact(raw_dt + dt_bias), decay = expf(-expf(a_log) * dt);
     __syncthreads();
     float Bv[R], Cv[R];
 #pragma unroll
@@ -311,10 +349,7 @@ mamba2_step_kernel(const StepParams p) {
             if (next < nv) load_state(next, s[u]);
 #pragma unroll
             for (int o = 16; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-            if (lane == 0) {
-                const int col = h * p.P + v0 + vu;
-                p.gated[(int64_t)b * inner + col] = fmaf(D, x, y) * silu_exact(to_f(row[col]));
-            }
+            if (lane == 0) p.gated[(int64_t)b * inner + h * p.P + v0 + vu] = fmaf(D, x, y) * sz[vu];
         }
     }
 }
@@ -439,16 +474,24 @@ static int conv_launch(const ConvParams& p, cudaStream_t st) {
     return launch_status("bn_mamba2_conv");
 }
 
+template <typename T, int R, int VEC>
+static int step_launch_taps(const StepParams& p, cudaStream_t st) {
+    const unsigned grid = (unsigned)((long long)p.B * p.H * ((p.P + p.p_per_block - 1) / p.p_per_block));
+    const size_t smem = (size_t)(2 * p.N + 2 * p.p_per_block) * sizeof(float);
+    if (smem > 48 * 1024) return fail(BN_ERR_UNSUPPORTED, "bn_mamba2_step: vdim=%d", p.P);
+    if (p.taps == 4 && (reinterpret_cast<uintptr_t>(p.conv_w) & 15) == 0)
+        launch_dependent(mamba2_step_kernel<T, R, VEC, 4>, grid, ST_WARPS * 32, smem, st, p);
+    else launch_dependent(mamba2_step_kernel<T, R, VEC, 0>, grid, ST_WARPS * 32, smem, st, p);
+    return launch_status("bn_mamba2_step");
+}
+
 template <typename T>
 static int step_launch(const StepParams& p, cudaStream_t st) {
-    const unsigned grid = (unsigned)((long long)p.B * p.H * ((p.P + p.p_per_block - 1) / p.p_per_block));
-    const size_t smem = (size_t)(2 * p.N + p.p_per_block) * sizeof(float);
-    if (p.N == 128) launch_dependent(mamba2_step_kernel<T, 4, 4>, grid, ST_WARPS * 32, smem, st, p);
-    else if (p.N == 256) launch_dependent(mamba2_step_kernel<T, 8, 4>, grid, ST_WARPS * 32, smem, st, p);
-    else if (p.N <= 64) launch_dependent(mamba2_step_kernel<T, 2, 1>, grid, ST_WARPS * 32, smem, st, p);
-    else if (p.N <= 256) launch_dependent(mamba2_step_kernel<T, 8, 1>, grid, ST_WARPS * 32, smem, st, p);
-    else launch_dependent(mamba2_step_kernel<T, 16, 1>, grid, ST_WARPS * 32, smem, st, p);
-    return launch_status("bn_mamba2_step");
+    if (p.N == 128) return step_launch_taps<T, 4, 4>(p, st);
+    if (p.N == 256) return step_launch_taps<T, 8, 4>(p, st);
+    if (p.N <= 64) return step_launch_taps<T, 2, 1>(p, st);
+    if (p.N <= 256) return step_launch_taps<T, 8, 1>(p, st);
+    return step_launch_taps<T, 16, 1>(p, st);
 }
 
 }  // namespace bn

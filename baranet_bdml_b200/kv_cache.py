@@ -146,21 +146,25 @@ class RecurrentState:
 
 
 class SequenceSlots:
-    """Which slot of the per-layer caches and states a live sequence has, and how many tokens it has seen.  A slot is reset
-    in every layer when it is taken, so what an earlier sequence left never reaches the next one."""
+    """Which slot of the per-layer caches and states a live sequence has, and how many tokens it has seen.  A slot that has
+    been used is reset in every layer when it is taken again, so what an earlier sequence left never reaches the next one
+    (states are made zeroed)."""
 
     def __init__(self, num_seqs: int, states, device="cuda"):
         self.num_seqs, self.states = num_seqs, list(states)
         self.lens = torch.zeros((num_seqs,), dtype=torch.int32, device=device)
         self.free = list(range(num_seqs - 1, -1, -1))
+        self.used = set()
 
     def acquire(self) -> int:
         if not self.free:
             raise RuntimeError(f"all {self.num_seqs} sequence slots are in use")
         slot = self.free.pop()
-        self.lens[slot] = 0
-        for s in self.states:
-            s.reset(slot)
+        if slot in self.used:
+            self.lens[slot] = 0
+            for s in self.states:
+                s.reset(slot)
+        self.used.add(slot)
         return slot
 
     def release(self, slot: int) -> None:

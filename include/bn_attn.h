@@ -446,8 +446,8 @@ BN_API int bn_latent_decode_splits(int B, int H, int kv_rank, int rot, int windo
 BN_API int bn_latent_decode(const void* q_abs, const void* ring, int num_slots, int ring_tokens, const int32_t* seq_ids,
                             const int32_t* positions, float* partial, float* lse, int splits, int B, int H, int kv_rank,
                             int rot, int window, float scale, int dtype, bn_stream_t stream);
-/* merges the parts and expands the latent sum: out (B, out_ld), column h * vdim + v; wuv (H * vdim, round8(kv_rank)) */
-BN_API int bn_latent_expand_out(const float* partial, const float* lse, int splits, const void* wuv, void* out,
+/* merges the parts (in place: partial is changed) and expands the latent sum: out (B, out_ld), column h * vdim + v; wuv (H * vdim, round8(kv_rank)) */
+BN_API int bn_latent_expand_out(float* partial, const float* lse, int splits, const void* wuv, void* out,
                                 int64_t out_ld, int B, int H, int vdim, int kv_rank, int dtype, bn_stream_t stream);
 
 /* ------------------------------------------------------------------------
