@@ -138,17 +138,11 @@ latent_prep_kernel(const LatentPrepParams p) {
 // rot <= 2 LP_THREADS.
 // Everything a row needs is requested before the sums.
 template <typename T, int NQ, int NK>
-__global__ void __launch_bounds__(LP_THREADS)
+__global__ void __launch_bounds__(LP_THREADS, 8)
 latent_prep_regs_kernel(const LatentPrepParams p) {
     __shared__ float sh[2][LP_THREADS / 32];
     const int tid = threadIdx.x;
-    float wq[NQ][4], wk[NK][4];                          // the norms' weights stay for all rows of the block
-#pragma unroll
-    for (int k = 0; k < NQ; ++k)
-        if ((tid + k * LP_THREADS) * 4 < p.q_rank) load4(p.q_norm + (tid + k * LP_THREADS) * 4, wq[k]);
-#pragma unroll
-    for (int k = 0; k < NK; ++k)
-        if ((tid + k * LP_THREADS) * 4 < p.kv_rank) load4(p.kv_norm + (tid + k * LP_THREADS) * 4, wk[k]);
+    const double freq = 2 * tid < p.rot ? p.freq[tid] : 0.0;
     ptx::grid_dependency_wait();
     ptx::grid_launch_dependents();
     for (int r = blockIdx.x; r < p.rows; r += gridDim.x) {
@@ -168,6 +162,8 @@ latent_prep_regs_kernel(const LatentPrepParams p) {
         }
         if (2 * tid < p.rot) { u = to_f(rin[2 * tid]); v = to_f(rin[2 * tid + 1]); }
         const int pos = p.positions[b] + s, slot = p.seq_ids ? p.seq_ids[b] : b;
+        float cs = 1.f, sn = 0.f;
+        if (2 * tid < p.rot) rotation(pos, freq, &cs, &sn);      // while the row is on its way
         float sq = 0.f, sk = 0.f;
 #pragma unroll
         for (int k = 0; k < NQ; ++k)
@@ -201,8 +197,10 @@ latent_prep_regs_kernel(const LatentPrepParams p) {
         for (int k = 0; k < NQ; ++k) {
             const int i = (tid + k * LP_THREADS) * 4;
             if (i < p.q_rank) {
+                float w4[4];
+                load4(p.q_norm + i, w4);
 #pragma unroll
-                for (int e = 0; e < 4; ++e) vq[k][e] = vq[k][e] * inv_q * wq[k][e];
+                for (int e = 0; e < 4; ++e) vq[k][e] = vq[k][e] * inv_q * w4[e];
                 store4(cq + i, vq[k]);
             } else if (i < p.cq_ld) store4(cq + i, zero);
         }
@@ -210,8 +208,10 @@ latent_prep_regs_kernel(const LatentPrepParams p) {
         for (int k = 0; k < NK; ++k) {
             const int i = (tid + k * LP_THREADS) * 4;
             if (i < p.kv_rank) {
+                float w4[4];
+                load4(p.kv_norm + i, w4);
 #pragma unroll
-                for (int e = 0; e < 4; ++e) vk[k][e] = vk[k][e] * inv_k * wk[k][e];
+                for (int e = 0; e < 4; ++e) vk[k][e] = vk[k][e] * inv_k * w4[e];
                 if (c) store4(c + i, vk[k]);
                 if (ring) store4(ring + i, vk[k]);
             } else if (i < p.kv_ld) {
@@ -222,8 +222,6 @@ latent_prep_regs_kernel(const LatentPrepParams p) {
         if (2 * tid < p.rot_ld) {
             T lo = from_f<T>(0.f), hi = lo;
             if (2 * tid < p.rot) {
-                float cs, sn;
-                rotation(pos, p.freq[tid], &cs, &sn);
                 lo = from_f<T>(u * cs - v * sn);
                 hi = from_f<T>(v * cs + u * sn);
             }

@@ -20,8 +20,8 @@
 namespace bn {
 
 // ---------------------------------------------------------------------------------------------------------------
-// Convolution + silu of a portion, and the step sizes.  A thread owns VEC neighbouring channels (or dt columns) over
-// CV_TOK tokens, with the last taps - 1 inputs in registers.
+// Convolution + silu of a portion.  A thread owns VEC neighbouring channels over CV_TOK tokens, with the last taps - 1
+// inputs in registers.
 // ---------------------------------------------------------------------------------------------------------------
 struct ConvParams {
     const void* proj;                 // row stride proj_ld; the convolved channels start at column first_col
@@ -69,7 +69,7 @@ template <> __device__ __forceinline__ float conv_silu_f<__nv_bfloat16>(float z)
 // TAPS > 0: known at compile time; 0: p.taps (at most CV_MAXTAPS)
 template <typename T, int VEC, int TAPS>
 __global__ void __launch_bounds__(128)
-conv_step_kernel(const ConvParams p) {
+conv_silu_kernel(const ConvParams p) {
     using V = ConvVec<T, VEC>;
     ptx::grid_dependency_wait();
     ptx::grid_launch_dependents();
@@ -79,21 +79,7 @@ conv_step_kernel(const ConvParams p) {
     const int b = blockIdx.y / segs, t0 = (blockIdx.y % segs) * CV_TOK, t1 = min(p.S, t0 + CV_TOK);
     const int c = (blockIdx.x * 128 + threadIdx.x) * VEC;
     const T* in = static_cast<const T*>(p.proj) + (int64_t)b * p.S * p.proj_ld + p.first_col;
-    if (c >= p.C) {                                    // the dt columns follow the convolved ones
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) {
-            const int h = c + e - p.C;
-            if (h >= p.H) continue;
-            const float bias = p.dt_bias[h], neg_a = -expf(p.a_log[h]);
-            for (int t = t0; t < t1; ++t) {
-                const float d = softplus_exact(to_f(in[(int64_t)t * p.proj_ld + p.C + h]) + bias);
-                const int64_t o = ((int64_t)b * p.S + t) * p.H + h;
-                p.dt[o] = d;
-                p.a[o] = neg_a * d;
-            }
-        }
-        return;
-    }
+    if (c >= p.C) return;
     float w[W][VEC], bias[VEC], hist[W][VEC];          // hist[k]: the input k + 1 tokens back
 #pragma unroll
     for (int e = 0; e < VEC; ++e) bias[e] = p.bias[c + e];
@@ -148,18 +134,30 @@ conv_step_kernel(const ConvParams p) {
     }
 }
 
-// the portion's last inputs into the ring (after the convolution has read it)
+// What else a portion leaves: its last inputs in the ring (after the convolution has read it), and the step size and log
+// decay of every token and head.
 template <typename T>
-__global__ void __launch_bounds__(128)
-conv_ring_kernel(const T* proj, int64_t proj_ld, int first_col, T* ring, const int32_t* seq_ids, const int32_t* positions, int B,
-                 int S, int C, int taps) {
+__global__ void __launch_bounds__(256)
+conv_tail_kernel(const ConvParams p, T* ring) {
     ptx::grid_dependency_wait();
     ptx::grid_launch_dependents();
-    const int keep = min(S, taps), b = blockIdx.y / keep, t = S - keep + blockIdx.y % keep;
-    const int c = blockIdx.x * 128 + threadIdx.x;
-    if (c >= C) return;
-    const int slot = seq_ids ? seq_ids[b] : b;
-    ring[((int64_t)slot * taps + (positions[b] + t) % taps) * C + c] = proj[((int64_t)b * S + t) * proj_ld + first_col + c];
+    const int keep = min(p.S, p.taps);
+    const long long n_ring = (long long)p.B * keep * p.C, n = n_ring + (long long)p.B * p.S * p.H;
+    for (long long i = (long long)blockIdx.x * 256 + threadIdx.x; i < n; i += (long long)gridDim.x * 256) {
+        if (i < n_ring) {
+            const int c = (int)(i % p.C), k = (int)(i / p.C % keep), b = (int)(i / p.C / keep), t = p.S - keep + k;
+            const int slot = p.seq_ids ? p.seq_ids[b] : b;
+            ring[((int64_t)slot * p.taps + (p.positions[b] + t) % p.taps) * p.C + c] =
+                static_cast<const T*>(p.proj)[((int64_t)b * p.S + t) * p.proj_ld + p.first_col + c];
+        } else {
+            const long long q = i - n_ring;
+            const int64_t row = q / p.H;
+            const int h = (int)(q - row * p.H);
+            const float d = softplus_exact(to_f(static_cast<const T*>(p.proj)[row * p.proj_ld + p.first_col + p.C + h]) + p.dt_bias[h]);
+            p.dt[q] = d;
+            p.a[q] = -expf(p.a_log[h]) * d;
+        }
+    }
 }
 
 // ---------------------------------------------------------------------------------------------------------------
@@ -467,10 +465,10 @@ static int gated_norm_launch(const GatedNormParams& p, bn_stream_t stream) {
 
 template <typename T, int VEC>
 static int conv_launch(const ConvParams& p, cudaStream_t st) {
-    const int cols = p.C + p.H, segs = (p.S + CV_TOK - 1) / CV_TOK;
-    const dim3 grid((cols + 128 * VEC - 1) / (128 * VEC), (unsigned)(p.B * segs));
-    if (p.taps == 4) conv_step_kernel<T, VEC, 4><<<grid, 128, 0, st>>>(p);
-    else conv_step_kernel<T, VEC, 0><<<grid, 128, 0, st>>>(p);
+    const int segs = (p.S + CV_TOK - 1) / CV_TOK;
+    const dim3 grid((p.C + 128 * VEC - 1) / (128 * VEC), (unsigned)(p.B * segs));
+    if (p.taps == 4) conv_silu_kernel<T, VEC, 4><<<grid, 128, 0, st>>>(p);
+    else conv_silu_kernel<T, VEC, 0><<<grid, 128, 0, st>>>(p);
     return launch_status("bn_mamba2_conv");
 }
 
@@ -529,13 +527,10 @@ extern "C" int bn_mamba2_conv(const void* proj, int64_t proj_ld, const float* co
     else if (pairs) rc = conv_launch<__nv_bfloat16, 2>(p, st);
     else rc = conv_launch<__nv_bfloat16, 1>(p, st);
     if (rc) return rc;
-    const dim3 grid((C + 127) / 128, (unsigned)(B * (S < taps ? S : taps)));
-    if (dtype == 0)
-        conv_ring_kernel<float><<<grid, 128, 0, st>>>(static_cast<const float*>(proj), proj_ld, inner, static_cast<float*>(ring), seq_ids,
-                                                 positions, B, S, C, taps);
-    else
-        conv_ring_kernel<__nv_bfloat16><<<grid, 128, 0, st>>>(static_cast<const __nv_bfloat16*>(proj), proj_ld, inner,
-                                                         static_cast<__nv_bfloat16*>(ring), seq_ids, positions, B, S, C, taps);
+    const long long n = (long long)B * (S < taps ? S : taps) * C + (long long)B * S * H, blocks = (n + 255) / 256;
+    const unsigned grid = (unsigned)(blocks < 8192 ? blocks : 8192);
+    if (dtype == 0) launch_dependent(conv_tail_kernel<float>, grid, 256, 0, st, p, static_cast<float*>(ring));
+    else launch_dependent(conv_tail_kernel<__nv_bfloat16>, grid, 256, 0, st, p, static_cast<__nv_bfloat16*>(ring));
     return launch_status(what);
 }
 

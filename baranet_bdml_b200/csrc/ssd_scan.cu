@@ -82,20 +82,19 @@ ssd_scan_kernel(const SsmScanParams p, int slices) {
         // ---- tiles of the chunk (pieces of 8; beyond the sequence or the matrix: zeros)
         for (int i = threadIdx.x; i < SD_Q * (NP / 8); i += blockDim.x) {
             const int r = i / (NP / 8), c = i % (NP / 8) * 8;
-            uint4 vb = make_uint4(0, 0, 0, 0), vc = vb;
-            if (r < nt && c < p.N) {           // N is a multiple of 8
-                vb = *reinterpret_cast<const uint4*>(gB + (int64_t)(t0 + r) * p.xbc_ld + c);
-                vc = *reinterpret_cast<const uint4*>(gC + (int64_t)(t0 + r) * p.xbc_ld + c);
-            }
-            *reinterpret_cast<uint4*>(sB + r * LDN + c) = vb;
-            *reinterpret_cast<uint4*>(sC + r * LDN + c) = vc;
+            const bool in = r < nt && c < p.N;                           // N is a multiple of 8
+            const int64_t o = in ? (int64_t)(t0 + r) * p.xbc_ld + c : 0;
+            cp_async_16(uB + (r * LDN + c) * 2, gB + o, in ? 16 : 0);
+            cp_async_16(uC + (r * LDN + c) * 2, gC + o, in ? 16 : 0);
         }
         for (int i = threadIdx.x; i < SD_Q * (PW / 8); i += blockDim.x) {
             const int r = i / (PW / 8), c = i % (PW / 8) * 8;
-            uint4 vx = make_uint4(0, 0, 0, 0);
-            if (r < nt && c < nv) vx = *reinterpret_cast<const uint4*>(gx + (int64_t)(t0 + r) * p.xbc_ld + c);   // P a multiple of 8
-            *reinterpret_cast<uint4*>(sX + r * LDX + c) = vx;
+            const bool in = r < nt && c < nv;                            // P is a multiple of 8
+            cp_async_16(uX + (r * LDX + c) * 2, gx + (in ? (int64_t)(t0 + r) * p.xbc_ld + c : 0), in ? 16 : 0);
         }
+        // the next chunk's values on their way to L2 (its B and C serve all heads of a group and are there already)
+        if (threadIdx.x < SD_Q && t0 + SD_Q + (int)threadIdx.x < p.S)
+            asm volatile("prefetch.global.L2 [%0];" ::"l"(gx + (int64_t)(t0 + SD_Q + threadIdx.x) * p.xbc_ld));
         if (warp == 0) {                       // running sum of the log decays, two tokens per lane
             const int i0 = 2 * lane;
             const int64_t row = (int64_t)b * p.S + t0;
@@ -117,6 +116,7 @@ ssd_scan_kernel(const SsmScanParams p, int slices) {
             s_w[i0] = expf(last - (before + a0)) * d0;
             s_w[i0 + 1] = expf(last - s) * d1;
         }
+        cp_async_wait_all();
         __syncthreads();
         // ---- M = (C B^T) e^{c_i - c_j} dt_j for j <= i, 16 rows at a time
         for (int mb = warp; mb < SD_Q / 16; mb += W) {
