@@ -5,6 +5,7 @@ This module holds what is particular to the design: how its config.json is read 
 The sublayers are in mixers.py, caches and states in kv_cache.py, generation in model.py."""
 from __future__ import annotations
 
+import warnings
 from dataclasses import dataclass
 from typing import List, Optional, Sequence
 
@@ -131,7 +132,7 @@ class SoluzenModel(CausalLM):
         self.final_norm = ops.NormWeight(w("final.norm", width), w("final.norm.b", width), c.eps)
         self.head = ops.Linear(w("head", c.vocab_size, width), dtype)
         if w.leftover():
-            raise RuntimeError(f"tensors that this design does not have: {w.leftover()[:5]}")
+            warnings.warn(f"checkpoint tensors that this design does not have: {w.leftover()[:5]}")
         self.slots: Optional[SequenceSlots] = None
         self._id_error = torch.zeros(1, dtype=torch.int32, device="cuda")
 
