@@ -17,7 +17,7 @@ LIB_PATH = os.environ.get("BN_ATTN_LIB") or os.path.join(_HERE, "libbn_attn.so")
 BN_OK, BN_ERR_INVALID_ARG, BN_ERR_UNSUPPORTED, BN_ERR_CUDA, BN_ERR_ARCH, BN_ERR_TIMEOUT, BN_ERR_WORKSPACE = range(7)
 BN_HEADS_COLLAPSED, BN_HEADS_PER_HEAD = 0, 1
 BN_PAGE_TOKENS = 16
-BN_ACT_NONE, BN_ACT_SILU, BN_ACT_GELU_TANH = range(3)
+BN_ACT_NONE, BN_ACT_SILU, BN_ACT_GELU_TANH, BN_ACT_RELU2 = range(4)
 
 _i, _i64, _f, _p, _sz = C.c_int, C.c_int64, C.c_float, C.c_void_p, C.c_size_t
 
@@ -88,6 +88,18 @@ SIGNATURES = {
                             _p]),
     "bn_ssm_scan": (_i, [_p, _i64, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _p, _i64, _i, _p]),
     "bn_mamba2_step": (_i, [_p, _i64, _p, _p, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _p, _i, _p]),
+    "bn_gemm_bias_act_bf16_nt": (_i, [_p, _p, _p, _p, _i, _i, _i, _i, _p, _p]),
+    "bn_gemm_bias_act_bf16_nt_small_m": (_i, [_p, _p, _p, _p, _i, _i, _i, _i, _p, _sz, _p, _p]),
+    "bn_gemm_bias_act_bf16_nt_skinny": (_i, [_p, _p, _p, _p, _i, _i, _i, _i, _p]),
+    "bn_bias_act_f32": (_i, [_p, _i64, _p, _i, _i, _i, _p]),
+    "bn_hyper_norm": (_i, [_p, _i, _i, _p, _p, _p, _p, _i64, _p, _p, _p, _p, _i64, _i, _i, _i, _f, _p]),
+    "bn_kv_prep": (_i, [_p, _p, _i64, _p, _i64, _f, _p, _p, _i, _i, _i, _i, _i, _i, _f, _p, _p, _i, _i, _p, _p, _i, _i, _i, _p]),
+    "bn_kv_gather": (_i, [_p, _p, _i, _i, _i, _i, _i, _p, _p, _i, _i, _p, _p, _i, _i, _p]),
+    "bn_attn_chunked": (_i, [_p, _i64, _p, _i64, _p, _i64, _p, _i64, _p, _i64, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _f,
+                             _p, _i, _p]),
+    "bn_gqa_step_splits": (_i, [_i, _i, _i, _i, _i, _i, _i]),
+    "bn_gqa_step": (_i, [_p, _p, _p, _p, _i64, _p, _i64, _f, _p, _p, _i, _i, _i, _p, _p, _p, _p, _i, _p, _i64, _i, _i, _i, _i, _i,
+                         _i, _f, _f, _p, _i, _p]),
     "bn_gated_group_norm": (_i, [_p, _i64, _i, _p, _i64, _p, _p, _i64, _i, _i, _i, _f, _i, _p]),
 }
 

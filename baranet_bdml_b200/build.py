@@ -19,11 +19,14 @@ LIB = os.path.join(HERE, "libbn_attn.so")
 OBJ = os.path.join(HERE, "build")
 SOURCES = ["api.cu", "tma.cu", "attn_f32.cu", "rmsnorm.cu", "embed_argmax.cu", "kv_cache.cu", "attn_decode.cu",
            "attn_prefill_sm100.cu", "gemm_bf16_sm100.cu", "gemm_skinny.cu", "exchange.cu", "residual_norm.cu",
-           "latent_attn.cu", "latent_prefill_sm100.cu", "latent_decode.cu", "mamba2.cu", "ssd_scan.cu", "mm_f32.cu"]
+           "attn_portion.cu", "attn_portion_sm100.cu", "latent_attn.cu", "latent_decode.cu", "mamba2.cu", "ssd_scan.cu", "mm_f32.cu",
+           "hyper_norm.cu", "gqa_chunk.cu"]
 # what a model family launches
 FAMILIES = {
     "soluzen": ["api.cu", "tma.cu", "mm_f32.cu", "embed_argmax.cu", "gemm_bf16_sm100.cu", "gemm_skinny.cu", "residual_norm.cu",
-                "latent_attn.cu", "latent_prefill_sm100.cu", "latent_decode.cu", "mamba2.cu", "ssd_scan.cu"],
+                "attn_portion.cu", "attn_portion_sm100.cu", "latent_attn.cu", "latent_decode.cu", "mamba2.cu", "ssd_scan.cu"],
+    "duponex": ["api.cu", "tma.cu", "mm_f32.cu", "embed_argmax.cu", "gemm_bf16_sm100.cu", "gemm_skinny.cu", "residual_norm.cu",
+                "hyper_norm.cu", "attn_portion.cu", "attn_portion_sm100.cu", "gqa_chunk.cu"],
 }
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "--expt-relaxed-constexpr", "-Xcompiler", "-fPIC,-fvisibility=hidden",

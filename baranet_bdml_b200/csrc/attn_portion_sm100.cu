@@ -1,6 +1,6 @@
-// Windowed attention of a prompt portion on the 5th-generation tensor cores: per-head keys of dim unrotated columns plus
-// one rotated part shared by all heads, values of another width, a sliding window, and keys that start before the
-// portion's first query (bn_attn_window's fast path, bf16).
+// Attention of a prompt portion on the 5th-generation tensor cores: keys of dim columns per key head, plus optionally one
+// rotated part shared by all heads, values of another width, a sliding window or chunks, and keys that start before the
+// portion's first query (the fast path of bn_attn_window and bn_attn_chunked, bf16).
 //
 // Persistent, one CTA per SM, ten warps.  Work unit = (sequence, head, PAIR of 128-row query tiles); a unit walks the
 // 64-key tiles from the first key that the pair's first row sees to the last row's own key:
@@ -17,11 +17,14 @@
 // scores never overtake the read of the weights they replace, and while one tile's softmax runs the other tile's products
 // do.  A commit covers everything issued before it, so the scores' barrier of step j also says that PV of step j - 1 has
 // landed and O may be rescaled.
+// Optional: queries divided by their root mean square - a softmax thread sums its row's squares out of the Q tile and folds
+// the reciprocal into the row's score scale - and outputs multiplied by the sigmoid of a gate on their way out.
 // A key tile that a query tile does not see at all is skipped for that tile.  Masks are applied only by warps that have an
 // edge (a row's own key, or the window's far end) inside the key tile.
 // Every wait is bounded; on expiry the kernel raises the caller's error word, frees TMEM and returns.
+#include "attn_portion.cuh"
 #include "common.cuh"
-#include "latent.cuh"
+#include "hybrid.cuh"
 #include "ptx.cuh"
 #include "tcgen05.cuh"
 #include "tma.cuh"
@@ -42,12 +45,13 @@ constexpr float WA_RESCALE_THRESHOLD = 8.0f;                     // log2 units
 
 struct WaParams {
     __nv_bfloat16* out;
-    int64_t out_ld;
+    const __nv_bfloat16* gate;
+    int64_t out_ld, gate_ld;
     int* error_word;
-    int B, S, n_old, H, dim, rot, vdim, window;
+    int B, S, n_old, H, rep, dim, rot, vdim, mask, span, rms_dim;
     int nb_dim, nb_rot, nb_v, stages;        // 64-column blocks of the unrotated / rotated key parts and of the values
     int n_pairs, n_units;
-    float scale_log2;
+    float scale_log2, rms_eps;
 };
 
 struct WaUnit {
@@ -62,13 +66,13 @@ __device__ __forceinline__ WaUnit wa_unit(const WaParams& p, int k) {
     w.i0 = (p.n_pairs - 1 - k / (p.B * p.H)) * 2 * WA_BM;          // late rows see the most keys: they come first
     w.b = bh / p.H;
     w.h = bh - w.b * p.H;
-    w.key0 = max(0, p.n_old + w.i0 - p.window + 1);
+    w.key0 = max(0, mask_oldest(p.mask, p.span, p.n_old + w.i0));
     w.n = 0;
 #pragma unroll
     for (int u = 0; u < 2; ++u) {
         const int r0 = w.i0 + u * WA_BM;
         if (r0 >= p.S) { w.first[u] = 0; w.last[u] = -1; continue; }
-        const int lo = max(0, p.n_old + r0 - p.window + 1), hi = p.n_old + min(r0 + WA_BM, p.S) - 1;
+        const int lo = max(0, mask_oldest(p.mask, p.span, p.n_old + r0)), hi = p.n_old + min(r0 + WA_BM, p.S) - 1;
         w.first[u] = (lo - w.key0) / WA_BN;
         w.last[u] = (hi - w.key0) / WA_BN;
         w.n = w.last[u] + 1;                                       // tile 1's last key is never before tile 0's
@@ -101,7 +105,7 @@ attn_window_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
     if (tid == 0) {
         for (int u = 0; u < 2; ++u) {
             mbar_init(smem_u32(&bar_q[u]), 1);
-            mbar_init(smem_u32(&bar_qfree[u]), 1);
+            mbar_init(smem_u32(&bar_qfree[u]), p.rms_dim ? 5 : 1);      // the last Q K^T, and the softmax warps that read Q
             mbar_init(smem_u32(&bar_s[u]), 1);
             mbar_init(smem_u32(&bar_p[u]), 128);
             mbar_init(smem_u32(&bar_o[u]), 1);
@@ -156,14 +160,14 @@ attn_window_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
                     if (!ok) break;
                     mbar_arrive_expect_tx(smem_u32(&bar_kfull[stage]), nb * WA_KBLK);
                     for (int x = 0; x < p.nb_dim; ++x)
-                        tma_load_4d(sK + (stage * nb + x) * WA_KBLK, &tmap_k, x * 64, w.h, key, w.b, smem_u32(&bar_kfull[stage]));
+                        tma_load_4d(sK + (stage * nb + x) * WA_KBLK, &tmap_k, x * 64, w.h / p.rep, key, w.b, smem_u32(&bar_kfull[stage]));
                     for (int x = 0; x < p.nb_rot; ++x)
                         tma_load_4d(sK + (stage * nb + p.nb_dim + x) * WA_KBLK, &tmap_r, x * 64, 0, key, w.b, smem_u32(&bar_kfull[stage]));
                     ok = mbar_wait(smem_u32(&bar_vempty[stage]), phase ^ 1u, &s_abort);
                     if (!ok) break;
                     mbar_arrive_expect_tx(smem_u32(&bar_vfull[stage]), p.nb_v * WA_KBLK);
                     for (int x = 0; x < p.nb_v; ++x)
-                        tma_load_4d(sV + (stage * p.nb_v + x) * WA_KBLK, &tmap_v, x * 64, w.h, key, w.b, smem_u32(&bar_vfull[stage]));
+                        tma_load_4d(sV + (stage * p.nb_v + x) * WA_KBLK, &tmap_v, x * 64, w.h / p.rep, key, w.b, smem_u32(&bar_vfull[stage]));
                     if (++stage == p.stages) { stage = 0; phase ^= 1u; }
                 }
             }
@@ -251,7 +255,7 @@ attn_window_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
         const uint32_t lane_base = ((uint32_t)((warp % 4) * 32)) << 16;
         const uint32_t tS = tmem + lane_base + u * WA_BN, tO = tmem + lane_base + WA_COL_O + u * WA_O_STRIDE;
         bool ok = true;
-        uint32_t ns = 0, no = 0;                                     // steps and tiles of this query tile so far
+        uint32_t ns = 0, no = 0, nq = 0;                             // steps and tiles of this query tile so far
         for (int round = 0; ok; ++round) {
             const int k = wa_unit_index(round, p.n_units);
             if (k < 0) break;
@@ -259,8 +263,29 @@ attn_window_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
             if (w.last[u] < w.first[u]) continue;
             const int row0 = w.i0 + u * WA_BM + (warp % 4) * 32;     // the warp's first row
             const int gi = row0 + lane;
-            const int own = p.n_old + gi, oldest = own - p.window + 1;         // the keys this row sees
-            const int warp_own0 = p.n_old + row0, warp_oldest1 = warp_own0 + 31 - p.window + 1;
+            const int own = p.n_old + gi, oldest = mask_oldest(p.mask, p.span, own);         // the keys this row sees
+            const int warp_own0 = p.n_old + row0, warp_oldest1 = mask_oldest(p.mask, p.span, warp_own0 + 31);
+            float scale_log2 = p.scale_log2;
+            if (p.rms_dim) {
+                ok = mbar_wait(smem_u32(&bar_q[u]), nq & 1u, &s_abort);
+                ++nq;
+                if (!ok) break;
+                const uint8_t* qrow = smem_raw + (sQ - smem_u32(smem_raw)) + u * nb * WA_QBLK + ((warp % 4) * 32 + lane) * 128;
+                float s0 = 0.f, s1 = 0.f;
+                for (int x = 0; x < p.nb_dim; ++x) {
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) {      // the row's 16-byte pieces in an order without bank conflicts
+                        const uint4 v = *reinterpret_cast<const uint4*>(qrow + x * WA_QBLK + ((i ^ (lane & 7)) << 4));
+                        s0 = fmaf(bf16_lo(v.x), bf16_lo(v.x), s0); s1 = fmaf(bf16_hi(v.x), bf16_hi(v.x), s1);
+                        s0 = fmaf(bf16_lo(v.y), bf16_lo(v.y), s0); s1 = fmaf(bf16_hi(v.y), bf16_hi(v.y), s1);
+                        s0 = fmaf(bf16_lo(v.z), bf16_lo(v.z), s0); s1 = fmaf(bf16_hi(v.z), bf16_hi(v.z), s1);
+                        s0 = fmaf(bf16_lo(v.w), bf16_lo(v.w), s0); s1 = fmaf(bf16_hi(v.w), bf16_hi(v.w), s1);
+                    }
+                }
+                scale_log2 *= rsqrtf((s0 + s1) / (float)p.rms_dim + p.rms_eps);
+                __syncwarp();
+                if (lane == 0) mbar_arrive(smem_u32(&bar_qfree[u]));
+            }
             float m_ref = -INFINITY, l_run = 0.f;
             for (int j = w.first[u]; j <= w.last[u]; ++j, ++ns) {
                 ok = mbar_wait(smem_u32(&bar_s[u]), ns & 1u, &s_abort);
@@ -291,10 +316,10 @@ attn_window_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
                     t3 = fmaxf(t3, __uint_as_float(r[1][i + 1]));
                 }
                 const float m_new = fmaxf(m_ref, fmaxf(fmaxf(t0, t1), fmaxf(t2, t3)));
-                const bool grow = (m_new - m_ref) * p.scale_log2 > WA_RESCALE_THRESHOLD;   // NaN (both -inf) is false
+                const bool grow = (m_new - m_ref) * scale_log2 > WA_RESCALE_THRESHOLD;   // NaN (both -inf) is false
                 if (__any_sync(0xffffffffu, grow)) {
                     if (j > w.first[u]) {
-                        const float alpha = m_ref == -INFINITY ? 0.f : ex2((m_ref - m_new) * p.scale_log2);
+                        const float alpha = m_ref == -INFINITY ? 0.f : ex2((m_ref - m_new) * scale_log2);
                         l_run *= alpha;
                         for (int c = 0; c < 2 * p.nb_v; ++c) {
                             uint32_t o[32];
@@ -308,15 +333,15 @@ attn_window_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
                     m_ref = m_new;
                 }
                 // a row that has seen no key yet has only -inf scores: any finite reference gives zero weights
-                const float mneg = m_ref == -INFINITY ? 0.f : -m_ref * p.scale_log2;
+                const float mneg = m_ref == -INFINITY ? 0.f : -m_ref * scale_log2;
                 float l0 = 0.f, l1 = 0.f;
 #pragma unroll
                 for (int c = 0; c < 2; ++c) {
                     uint32_t pk[16];
 #pragma unroll
                     for (int i = 0; i < 32; i += 2) {
-                        const float p0 = ex2(fmaf(__uint_as_float(r[c][i]), p.scale_log2, mneg));
-                        const float p1 = ex2(fmaf(__uint_as_float(r[c][i + 1]), p.scale_log2, mneg));
+                        const float p0 = ex2(fmaf(__uint_as_float(r[c][i]), scale_log2, mneg));
+                        const float p1 = ex2(fmaf(__uint_as_float(r[c][i + 1]), scale_log2, mneg));
                         l0 += p0;
                         l1 += p1;
                         pk[i / 2] = pack_bf16(p0, p1);
@@ -336,11 +361,25 @@ attn_window_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
             tc::fence_after_sync();
             const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
             __nv_bfloat16* dst = p.out + ((int64_t)w.b * p.S + gi) * p.out_ld + w.h * p.vdim;
+            const __nv_bfloat16* gate = p.gate ? p.gate + ((int64_t)w.b * p.S + gi) * p.gate_ld + w.h * p.vdim : nullptr;
             for (int c = 0; c < 2 * p.nb_v; ++c) {
                 uint32_t o[32];
                 tc::ld32(tO + c * 32, o);
                 tc::wait_ld(o);
                 if (gi < p.S) {
+                    if (gate) {
+#pragma unroll
+                        for (int v = 0; v < 4; ++v)
+                            if (c * 32 + v * 8 < p.vdim) {
+                                const uint4 g4 = *reinterpret_cast<const uint4*>(gate + c * 32 + v * 8);
+                                const uint32_t* gw = reinterpret_cast<const uint32_t*>(&g4);
+#pragma unroll
+                                for (int e = 0; e < 4; ++e) {
+                                    o[v * 8 + 2 * e] = __float_as_uint(__uint_as_float(o[v * 8 + 2 * e]) * sigmoid_fast(bf16_lo(gw[e])));
+                                    o[v * 8 + 2 * e + 1] = __float_as_uint(__uint_as_float(o[v * 8 + 2 * e + 1]) * sigmoid_fast(bf16_hi(gw[e])));
+                                }
+                            }
+                    }
 #pragma unroll
                     for (int v = 0; v < 4; ++v)
                         if (c * 32 + v * 8 < p.vdim) {                 // vdim is a multiple of 8
@@ -375,11 +414,12 @@ static int wa_stages(int nb, int nb_v) {
     return s > WA_MAXSTAGE ? WA_MAXSTAGE : s;
 }
 
-bool attn_window_sm100_ok(const AttnWindowParams& p) {
+bool attn_window_sm100_ok(const AttnPortionParams& p) {
     const int nb = (p.dim + 63) / 64 + (p.rot + 63) / 64, nb_v = (p.vdim + 63) / 64;
     const uintptr_t bases = reinterpret_cast<uintptr_t>(p.q) | reinterpret_cast<uintptr_t>(p.k) | reinterpret_cast<uintptr_t>(p.v) |
-                            reinterpret_cast<uintptr_t>(p.krot) | reinterpret_cast<uintptr_t>(p.out);
-    return ((p.dim | p.rot | p.vdim | p.q_ld | p.kv_ld | p.krot_ld | p.out_ld) & 7) == 0 && p.rot > 0 && (bases & 15) == 0 &&
+                            reinterpret_cast<uintptr_t>(p.krot) | reinterpret_cast<uintptr_t>(p.gate) | reinterpret_cast<uintptr_t>(p.out);
+    const int64_t strides = p.q_ld | p.k_ld | p.v_ld | p.krot_ld | p.gate_ld | p.out_ld | p.k_head | p.v_head;
+    return ((p.dim | p.rot | p.vdim | strides) & 7) == 0 && (bases & 15) == 0 && !(p.rms_dim && p.rot) && !p.positions &&
            nb_v <= WA_MAXVB && wa_stages(nb, nb_v) >= 2 && p.scale > 0.f;
 }
 
@@ -390,18 +430,23 @@ static int wa_map(CUtensorMap* m, const void* base, int inner, int heads, int64_
     return make_tensor_map(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, base, dims, strides, box, CU_TENSOR_MAP_SWIZZLE_128B);
 }
 
-int attn_window_sm100(const AttnWindowParams& a, cudaStream_t st) {
-    const char* what = "bn_attn_window";
+int attn_window_sm100(const AttnPortionParams& a, cudaStream_t st) {
+    const char* what = "portion attention";
     CUtensorMap mq, mk, mr, mv;
     if (int rc = wa_map(&mq, a.q, a.dim + a.rot, a.H, a.dim + a.rot, a.S, a.q_ld, a.B, WA_BM)) return rc;
-    if (int rc = wa_map(&mk, a.k, a.dim, a.H, a.dim, a.rows_per_seq, a.kv_ld, a.B, WA_BN)) return rc;
-    if (int rc = wa_map(&mr, a.krot, a.rot, 1, a.krot_ld, a.rows_per_seq, a.krot_ld, a.B, WA_BN)) return rc;
-    if (int rc = wa_map(&mv, a.v, a.vdim, a.H, a.vdim, a.rows_per_seq, a.kv_ld, a.B, WA_BN)) return rc;
+    if (int rc = wa_map(&mk, a.k, a.dim, a.kv_heads, a.k_head, a.rows_per_seq, a.k_ld, a.B, WA_BN)) return rc;
+    mr = mk;                                                           // without a rotated part nothing reads it
+    if (a.rot)
+        if (int rc = wa_map(&mr, a.krot, a.rot, 1, a.krot_ld, a.rows_per_seq, a.krot_ld, a.B, WA_BN)) return rc;
+    if (int rc = wa_map(&mv, a.v, a.vdim, a.kv_heads, a.v_head, a.rows_per_seq, a.v_ld, a.B, WA_BN)) return rc;
     WaParams p;
     p.out = static_cast<__nv_bfloat16*>(a.out);
     p.out_ld = a.out_ld;
     p.error_word = a.error_word;
-    p.B = a.B; p.S = a.S; p.n_old = a.n_old; p.H = a.H; p.dim = a.dim; p.rot = a.rot; p.vdim = a.vdim; p.window = a.window;
+    p.gate = static_cast<const __nv_bfloat16*>(a.gate);
+    p.gate_ld = a.gate_ld;
+    p.B = a.B; p.S = a.S; p.n_old = a.n_old; p.H = a.H; p.rep = a.H / a.kv_heads; p.dim = a.dim; p.rot = a.rot; p.vdim = a.vdim;
+    p.mask = a.mask; p.span = a.span; p.rms_dim = a.rms_dim; p.rms_eps = a.rms_eps;
     p.nb_dim = (a.dim + 63) / 64;
     p.nb_rot = (a.rot + 63) / 64;
     p.nb_v = (a.vdim + 63) / 64;

@@ -47,6 +47,23 @@ inline void launch_dependent(void (*kernel)(P...), unsigned grid, unsigned block
     }
 }
 
+// SMs of the current device
+inline int sm_count() {
+    int dev = 0, sms = 148;
+    cudaGetDevice(&dev);
+    cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
+    return sms;
+}
+
+// Lets `kernel` be launched with this much dynamic shared memory
+template <typename K>
+inline int allow_smem(K kernel, size_t bytes, const char* what) {
+    if (bytes <= 48 * 1024) return BN_OK;
+    if (bytes > 200 * 1024) return fail(BN_ERR_UNSUPPORTED, "%s: %zu bytes of shared memory", what, bytes);
+    cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
+    return e == cudaSuccess ? BN_OK : fail(BN_ERR_CUDA, "%s: %s", what, cudaGetErrorString(e));
+}
+
 // Byte offsets inside the scratch buffer of bn_attn_prefill_bf16 (cos/sin table, per-tile key norms, rotated K) and
 // its size: the fused q/k/v projection writes the last two itself.
 inline void prefill_bf16_workspace_layout(int B, int S, int Hkv, size_t* table, size_t* kmax2, size_t* krot, size_t* total) {

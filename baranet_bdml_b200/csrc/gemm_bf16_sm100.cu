@@ -13,7 +13,7 @@
 // runs under the main loop of the next.  Tiles are walked N-panel by N-panel with M fastest, so the CTAs that run
 // together share their Bt panel in L2.  Edges: TMA zero-fills loads beyond M, N, K; stores are bounds-checked.
 // Epilogue variants: plain (C = the accumulator as bf16), fp32 (the accumulator itself), the accumulator's activation
-// times a matrix given by the caller, and the gated linear unit (SwiGLU in `MLP.__call__`,
+// times a matrix given by the caller, the activation of the accumulator plus a bias, and the gated linear unit (SwiGLU in `MLP.__call__`,
 // mygrad/llama/llama_layers.py:217-232, SiLU as op_silu.cuh:7-15; GELU for other models): Bt holds, per 256-row tile, 128
 // rows of the gate weight followed by the 128 rows of the up weight for the same intermediate indices, so one thread finds
 // gate and up of an output element in the same accumulator row and writes act(gate) * up -- the two GEMMs, the activation
@@ -57,7 +57,7 @@ struct QkvEpilogue {
 };
 
 // EPI_GLU + activation: one instantiation per activation keeps the choice out of the epilogue's loop
-constexpr int EPI_PLAIN = 0, EPI_PARTIAL = 2, EPI_QKV = 3, EPI_F32 = 4, EPI_ACTMUL = 5, EPI_GLU = 16;
+constexpr int EPI_PLAIN = 0, EPI_PARTIAL = 2, EPI_QKV = 3, EPI_F32 = 4, EPI_ACTMUL = 5, EPI_BIAS = 6, EPI_GLU = 16;
 constexpr int EPI_GLU_SILU = EPI_GLU + BN_ACT_SILU, EPI_GLU_GELU = EPI_GLU + BN_ACT_GELU_TANH;
 
 struct GemmParams {
@@ -71,8 +71,8 @@ struct GemmParams {
     const __nv_bfloat16* mul;  // EPI_ACTMUL: (M, mul_ld), C = act(accumulator) * mul
     long long mul_ld;
     int act;
+    const float* bias;         // EPI_BIAS: C = act(accumulator + bias), bias (n_out) or null
 };
-
 
 
 template <int EPI, int GM_BN>
@@ -208,6 +208,31 @@ gemm_bf16_nt_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
                                 o4.z = pack_bf16(__uint_as_float(r[v * 8 + 4]), __uint_as_float(r[v * 8 + 5]));
                                 o4.w = pack_bf16(__uint_as_float(r[v * 8 + 6]), __uint_as_float(r[v * 8 + 7]));
                                 *reinterpret_cast<uint4*>(crow + c * 32 + v * 8) = o4;
+                            }
+                        }
+                    }
+                }
+            } else if (EPI == EPI_BIAS) {
+                __nv_bfloat16* crow = p.c + (size_t)gm * p.n_out + n0;
+#pragma unroll 1
+                for (int c = 0; c < GM_BN / 32; ++c) {
+                    uint32_t r[32];
+                    tc::ld32(tmem + lane_base + acc * GM_BN + c * 32, r);
+                    tc::wait_ld(r);
+                    if (gm < p.M) {
+#pragma unroll
+                        for (int v = 0; v < 4; ++v) {
+                            const int col = n0 + c * 32 + v * 8;
+                            if (col < p.n_out) {
+                                float h[8], b4[4] = {0.f, 0.f, 0.f, 0.f}, b8[4] = {0.f, 0.f, 0.f, 0.f};
+                                if (p.bias) { load4(p.bias + col, b4); load4(p.bias + col + 4, b8); }
+#pragma unroll
+                                for (int e = 0; e < 4; ++e) {
+                                    h[e] = activation_fast(p.act, __uint_as_float(r[v * 8 + e]) + b4[e]);
+                                    h[4 + e] = activation_fast(p.act, __uint_as_float(r[v * 8 + 4 + e]) + b8[e]);
+                                }
+                                *reinterpret_cast<uint4*>(crow + c * 32 + v * 8) =
+                                    make_uint4(pack_bf16(h[0], h[1]), pack_bf16(h[2], h[3]), pack_bf16(h[4], h[5]), pack_bf16(h[6], h[7]));
                             }
                         }
                     }
@@ -412,7 +437,8 @@ using namespace bn;
 // activation times `mul`
 __global__ void __launch_bounds__(256)
 gemm_splitk_reduce_kernel(const float* __restrict__ partial, __nv_bfloat16* __restrict__ c, long long mn4, int splits,
-                          float* __restrict__ c32, const __nv_bfloat16* __restrict__ mul, long long mul_ld, int N, int act) {
+                          float* __restrict__ c32, const __nv_bfloat16* __restrict__ mul, long long mul_ld, int N, int act,
+                          const float* __restrict__ bias) {
     const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;     // one group of 4 outputs
     if (i >= mn4) return;
     const float4* p4 = reinterpret_cast<const float4*>(partial);
@@ -432,6 +458,15 @@ gemm_splitk_reduce_kernel(const float* __restrict__ partial, __nv_bfloat16* __re
         acc.y = activation_fast(act, acc.y) * bf16_hi(m.x);
         acc.z = activation_fast(act, acc.z) * bf16_lo(m.y);
         acc.w = activation_fast(act, acc.w) * bf16_hi(m.y);
+    } else {
+        if (bias) {
+            const float4 b = *reinterpret_cast<const float4*>(bias + i * 4 % N);
+            acc.x += b.x; acc.y += b.y; acc.z += b.z; acc.w += b.w;
+        }
+        acc.x = activation_fast(act, acc.x);
+        acc.y = activation_fast(act, acc.y);
+        acc.z = activation_fast(act, acc.z);
+        acc.w = activation_fast(act, acc.w);
     }
     reinterpret_cast<uint2*>(c)[i] = make_uint2(pack_bf16(acc.x, acc.y), pack_bf16(acc.z, acc.w));
 }
@@ -463,13 +498,13 @@ static int gemm_configure(int dev) {
 static int gemm_launch(const void* a, const void* bt, void* c, int M, int N, int K, int n_out, int epi, int* error_word,
                        bn_stream_t stream, const char* what, float* partial = nullptr, int splits = 1,
                        int k_per_split = 0, const QkvEpilogue* qkv = nullptr, float* c32 = nullptr,
-                       const void* mul = nullptr, long long mul_ld = 0, int act = BN_ACT_NONE) {
+                       const void* mul = nullptr, long long mul_ld = 0, int act = BN_ACT_NONE, const float* bias = nullptr) {
     if (!a || !bt || (!c && !c32)) return fail(BN_ERR_INVALID_ARG, "%s: null pointer", what);
     if (M < 0 || N < 0 || K < 0 || n_out < 0) return fail(BN_ERR_INVALID_ARG, "%s: bad shape M=%d N=%d K=%d", what, M, N, K);
     if (n_out % 8 || K % 8)
         return fail(BN_ERR_UNSUPPORTED, "%s: N=%d and K=%d must be multiples of 8 (16-byte rows)", what, n_out, K);
     if ((reinterpret_cast<uintptr_t>(a) | reinterpret_cast<uintptr_t>(bt) | reinterpret_cast<uintptr_t>(c) |
-         reinterpret_cast<uintptr_t>(c32) | reinterpret_cast<uintptr_t>(mul)) & 15)
+         reinterpret_cast<uintptr_t>(c32) | reinterpret_cast<uintptr_t>(mul) | reinterpret_cast<uintptr_t>(bias)) & 15)
         return fail(BN_ERR_INVALID_ARG, "%s: a/bt/c must be 16-byte aligned", what);
     if (mul && (mul_ld < n_out || mul_ld % 8))
         return fail(BN_ERR_INVALID_ARG, "%s: row stride %lld of the factor (a multiple of 8, at least %d)", what, mul_ld, n_out);
@@ -502,7 +537,7 @@ static int gemm_launch(const void* a, const void* bt, void* c, int M, int N, int
     cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
     const long long n_items = (long long)((M + GM_BM - 1) / GM_BM) * ((N + bn - 1) / bn) * splits;
     GemmParams p{static_cast<__nv_bfloat16*>(c), error_word, M, N, K, n_out, partial, splits, k_per_split, QkvEpilogue{},
-                 static_cast<const __nv_bfloat16*>(mul), mul_ld, act};
+                 static_cast<const __nv_bfloat16*>(mul), mul_ld, act, bias};
     if (epi == EPI_F32) p.partial = c32;
     if (qkv) p.qkv = *qkv;
     const unsigned grid = (unsigned)(n_items < sms ? n_items : sms);
@@ -522,6 +557,9 @@ static int gemm_launch(const void* a, const void* bt, void* c, int M, int N, int
     } else if (epi == EPI_ACTMUL) {
         if (int rc = gemm_configure<EPI_ACTMUL, 256>(dev)) return rc;
         gemm_bf16_nt_kernel<EPI_ACTMUL, 256><<<grid, GM_THREADS, GemmShape<256>::SMEM_BYTES, st>>>(tmap_a, tmap_b, p);
+    } else if (epi == EPI_BIAS) {
+        if (int rc = gemm_configure<EPI_BIAS, 256>(dev)) return rc;
+        gemm_bf16_nt_kernel<EPI_BIAS, 256><<<grid, GM_THREADS, GemmShape<256>::SMEM_BYTES, st>>>(tmap_a, tmap_b, p);
     } else if (epi == EPI_QKV) {
         if (int rc = gemm_configure<EPI_QKV, 256>(dev)) return rc;
         gemm_bf16_nt_kernel<EPI_QKV, 256><<<grid, GM_THREADS, GemmShape<256>::SMEM_BYTES, st>>>(tmap_a, tmap_b, p);
@@ -531,7 +569,7 @@ static int gemm_launch(const void* a, const void* bt, void* c, int M, int N, int
         if (int rc = launch_status(what)) return rc;
         const long long mn4 = (long long)M * N / 4;
         gemm_splitk_reduce_kernel<<<(unsigned)((mn4 + 255) / 256), 256, 0, st>>>(partial, static_cast<__nv_bfloat16*>(c),
-                                                                             mn4, splits, c32, p.mul, mul_ld, N, act);
+                                                                             mn4, splits, c32, p.mul, mul_ld, N, act, bias);
     }
     return launch_status(what);
 }
@@ -568,6 +606,12 @@ extern "C" int bn_gemm_act_mul_bf16_nt(const void* a, const void* bt, const void
                        nullptr, mul, mul_ld, act);
 }
 
+extern "C" int bn_gemm_bias_act_bf16_nt(const void* a, const void* bt, const float* bias, void* c, int M, int N, int K, int act,
+                                        int* error_word, bn_stream_t stream) {
+    return gemm_launch(a, bt, c, M, N, K, N, EPI_BIAS, error_word, stream, "bn_gemm_bias_act_bf16_nt", nullptr, 1, 0, nullptr, nullptr,
+                       nullptr, 0, act, bias);
+}
+
 extern "C" size_t bn_gemm_bf16_nt_small_m_workspace_bytes(int M, int N, int K) {
     if (M <= 0 || N <= 0 || K <= 0) return 0;
     int dev = 0, sms = 0, splits = 1, per = 0;
@@ -580,7 +624,7 @@ extern "C" size_t bn_gemm_bf16_nt_small_m_workspace_bytes(int M, int N, int K) {
 
 static int small_m_launch(const void* a, const void* bt, void* c, float* c32, const void* mul, int64_t mul_ld, int act, int M,
                           int N, int K, void* workspace, size_t workspace_bytes, int* error_word, bn_stream_t stream,
-                          const char* what) {
+                          const char* what, const float* bias = nullptr) {
     int splits = 1, per = 0;
     if (M > 0 && N > 0 && K > 0) {
         if (!workspace || (reinterpret_cast<uintptr_t>(workspace) & 15))
@@ -593,7 +637,7 @@ static int small_m_launch(const void* a, const void* bt, void* c, float* c32, co
             return fail(BN_ERR_WORKSPACE, "%s: workspace of %zu bytes is too small", what, workspace_bytes);
     }
     return gemm_launch(a, bt, c, M, N, K, N, EPI_PARTIAL, error_word, stream, what, static_cast<float*>(workspace), splits, per,
-                       nullptr, c32, mul, mul_ld, act);
+                       nullptr, c32, mul, mul_ld, act, bias);
 }
 
 extern "C" int bn_gemm_bf16_nt_small_m(const void* a, const void* bt, void* c, int M, int N, int K, void* workspace,
@@ -614,6 +658,13 @@ extern "C" int bn_gemm_act_mul_bf16_nt_small_m(const void* a, const void* bt, co
     if (!mul) return fail(BN_ERR_INVALID_ARG, "bn_gemm_act_mul_bf16_nt_small_m: null pointer");
     return small_m_launch(a, bt, c, nullptr, mul, mul_ld, act, M, N, K, workspace, workspace_bytes, error_word, stream,
                           "bn_gemm_act_mul_bf16_nt_small_m");
+}
+
+extern "C" int bn_gemm_bias_act_bf16_nt_small_m(const void* a, const void* bt, const float* bias, void* c, int M, int N, int K,
+                                                int act, void* workspace, size_t workspace_bytes, int* error_word,
+                                                bn_stream_t stream) {
+    return small_m_launch(a, bt, c, nullptr, nullptr, 0, act, M, N, K, workspace, workspace_bytes, error_word, stream,
+                          "bn_gemm_bias_act_bf16_nt_small_m", bias);
 }
 
 extern "C" int bn_gemm_qkv_rope_bf16(const void* x, const void* wqkv_t, void* q_out, void* v_out, int B, int S, int hidden,

@@ -16,7 +16,7 @@
 // Variants: up to three column ranges of one concatenated weight written to separate outputs (q, k, v of the layer in one
 // launch); the same with the K and V ranges rotated / appended to the paged cache by the epilogue instead (what
 // bn_kv_append would do with them, mygrad/llama/llama_layers.py:161-171 for the new token); and the gated pair (two weights, h = act(x Wg) * (x Wu); SwiGLU: op_silu.cuh:7-15);
-// an fp32 output; and the result's activation times a matrix given by the caller.
+// an fp32 output; the result's activation times a matrix given by the caller; and the activation of the result plus a bias.
 // K is a multiple of 8 and at most 8192, N a multiple of 8.  When K is a multiple of 256 a warp's eighth is a whole number
 // of 32-wide steps; otherwise (RAGGED) the eighths are rounded up and pieces beyond K read as zero.  Anything else belongs to bn_gemm_bf16_nt_small_m.
 #include "common.cuh"
@@ -41,7 +41,8 @@ struct SkinnyParams {
     float* out32;                       // when set, the (single) output range in fp32 instead of out[0]
     const __nv_bfloat16* mul;           // when set, out[0] = act(x W) * mul, mul (M, mul_ld)
     long long mul_ld;
-    int act;                            // of the gated pair, or of `mul`
+    int act;                            // of the gated pair, of `mul`, or of the result plus bias
+    const float* bias;                  // optional, (N)
     // APPEND: columns from n_end[0] on are the K and V projections of one new token per row and go to the paged cache
     // instead of out[1] / out[2] (arguments as bn_kv_append)
     __nv_bfloat16* pool;
@@ -173,7 +174,9 @@ gemm_skinny_kernel(const SkinnyParams p) {
         } else if (row < p.M && p.out32) {
             p.out32[(size_t)row * p.N + n] = v;
         } else if (row < p.M) {
-            if (p.mul) v = activation_fast(p.act, v) * __bfloat162float(p.mul[row * p.mul_ld + n]);
+            if (p.bias) v += __ldg(p.bias + n);
+            if (!SWIGLU) v = activation_fast(p.act, v);
+            if (p.mul) v *= __bfloat162float(p.mul[row * p.mul_ld + n]);
             // selects, not indexed parameter arrays (an index known only at run time would copy them to local memory)
             __nv_bfloat16* o = p.out[0];
             int ld = p.ld[0], first = 0;
@@ -242,6 +245,22 @@ extern "C" int bn_gemm_bf16_nt_skinny_f32(const void* a, const void* bt, int M, 
     p.bt = static_cast<const __nv_bfloat16*>(bt);
     p.out32 = out;
     p.n_end[0] = p.n_end[1] = p.n_end[2] = N;
+    p.M = M; p.N = N; p.K = K; p.steps = (K + SK_WARPS * 32 - 1) / (SK_WARPS * 32);
+    return skinny_launch<false, false>(p, as_stream(stream), what);
+}
+
+extern "C" int bn_gemm_bias_act_bf16_nt_skinny(const void* a, const void* bt, const float* bias, void* out, int M, int N, int K,
+                                               int act, bn_stream_t stream) {
+    const char* what = "bn_gemm_bias_act_bf16_nt_skinny";
+    if (int rc = skinny_check(what, a, bt, M, N, K)) return rc;
+    if (!out || act < 0 || act > BN_ACT_LAST) return fail(BN_ERR_INVALID_ARG, "%s: bad argument", what);
+    SkinnyParams p{};
+    p.a = static_cast<const __nv_bfloat16*>(a);
+    p.bt = static_cast<const __nv_bfloat16*>(bt);
+    p.out[0] = static_cast<__nv_bfloat16*>(out);
+    p.n_end[0] = p.n_end[1] = p.n_end[2] = N;
+    p.ld[0] = N;
+    p.bias = bias; p.act = act;
     p.M = M; p.N = N; p.K = K; p.steps = (K + SK_WARPS * 32 - 1) / (SK_WARPS * 32);
     return skinny_launch<false, false>(p, as_stream(stream), what);
 }

@@ -35,16 +35,35 @@ __device__ __forceinline__ float gelu_tanh_exact(float z) {
 // softplus(z) = log(1 + e^z) without overflow
 __device__ __forceinline__ float softplus_exact(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
-// act: BN_ACT_NONE, BN_ACT_SILU, BN_ACT_GELU_TANH
+__device__ __forceinline__ float relu2(float z) { const float t = fmaxf(z, 0.f); return t * t; }
+__device__ __forceinline__ float sigmoid_exact(float z) { return 1.f / (1.f + expf(-z)); }
+__device__ __forceinline__ float sigmoid_fast(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
+
+// act: BN_ACT_NONE, BN_ACT_SILU, BN_ACT_GELU_TANH, BN_ACT_RELU2
 __device__ __forceinline__ float activation_exact(int act, float z) {
-    return act == BN_ACT_SILU ? silu_exact(z) : act == BN_ACT_GELU_TANH ? gelu_tanh_exact(z) : z;
+    return act == BN_ACT_SILU ? silu_exact(z) : act == BN_ACT_GELU_TANH ? gelu_tanh_exact(z) : act == BN_ACT_RELU2 ? relu2(z) : z;
 }
 // The epilogues of the bf16 products: the result is rounded to bf16, so the fast exponential suffices.
 // gelu_tanh(z) = z * sigmoid(2 u) with u = sqrt(2/pi) (z + 0.044715 z^3), because (1 + tanh u) / 2 = 1 / (1 + e^(-2u)).
 __device__ __forceinline__ float activation_fast(int act, float z) {
     if (act == BN_ACT_NONE) return z;
+    if (act == BN_ACT_RELU2) return relu2(z);
     const float t = act == BN_ACT_GELU_TANH ? 1.5957691216057308f * fmaf(0.044715f * z * z, z, z) : z;
     return __fdividef(z, 1.f + __expf(-t));
+}
+
+// sum over a block of THREADS threads, the same bits in every thread; sh holds THREADS / 32 floats
+template <int THREADS>
+__device__ __forceinline__ float block_sum(float v, float* sh) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    __syncthreads();                      // sh may still be read from the sum before
+    if (threadIdx.x % 32 == 0) sh[threadIdx.x / 32] = v;
+    __syncthreads();
+    float t = 0.f;
+#pragma unroll
+    for (int w = 0; w < THREADS / 32; ++w) t += sh[w];
+    return t;
 }
 
 // cos and sin of position * frequency.  The product and its reduction to one turn are taken in fp64, so that the angle

@@ -14,7 +14,7 @@
 // dot products may run over them.
 //
 // The kernels of this file take any sizes, in fp32 and in bf16; the tensor-core forms for the common sizes are in
-// latent_prefill_sm100.cu and latent_decode.cu.
+// latent_decode.cu, attention over expanded keys is in attn_portion.cu.
 #include "common.cuh"
 #include "hybrid.cuh"
 #include "latent.cuh"
@@ -274,78 +274,6 @@ rope_heads_kernel(T* q, int64_t q_ld, long long n, int S, int H, int dim, int ro
 }
 
 // ---------------------------------------------------------------------------------------------------------------
-// Windowed attention over expanded keys, any sizes: a warp per (query row, head); 32 keys at a time, a lane per key for
-// the scores, then a lane per value column.  Scores, weights and sums in fp32.
-// ---------------------------------------------------------------------------------------------------------------
-constexpr int AW_WARPS = 4, AW_MAXV = 16;      // vdim <= 512
-
-template <typename T>
-__global__ void __launch_bounds__(AW_WARPS * 32)
-attn_window_kernel(const AttnWindowParams p) {
-    extern __shared__ float q_smem[];
-    ptx::grid_dependency_wait();
-    ptx::grid_launch_dependents();
-    const int warp = threadIdx.x / 32, lane = threadIdx.x % 32;
-    const int E = p.dim + p.rot;
-    float* qs = q_smem + warp * E;
-    const long long n = (long long)p.B * p.S * p.H;
-    for (long long item = (long long)blockIdx.x * AW_WARPS + warp; item < n; item += (long long)gridDim.x * AW_WARPS) {
-        const int h = (int)(item % p.H);
-        const long long row = item / p.H;
-        const int b = (int)(row / p.S), s = (int)(row - (long long)b * p.S);
-        const T* q = static_cast<const T*>(p.q) + row * p.q_ld + h * E;
-        __syncwarp();
-        for (int e = lane; e < E; e += 32) qs[e] = to_f(q[e]);
-        __syncwarp();
-        const int last = p.n_old + s, first = max(0, last - p.window + 1);
-        const int64_t seq_row = (int64_t)b * p.rows_per_seq;
-        float m = -INFINITY, l = 0.f, acc[AW_MAXV];
-#pragma unroll
-        for (int v = 0; v < AW_MAXV; ++v) acc[v] = 0.f;
-        for (int k0 = first; k0 <= last; k0 += 32) {
-            const int k = k0 + lane;
-            float sc = -INFINITY;
-            if (k <= last) {
-                const T* kn = static_cast<const T*>(p.k) + (seq_row + k) * p.kv_ld + h * p.dim;
-                const T* kr = static_cast<const T*>(p.krot) + (seq_row + k) * p.krot_ld;
-                float d = 0.f;
-                for (int e = 0; e < p.dim; ++e) d = fmaf(qs[e], to_f(kn[e]), d);
-                for (int e = 0; e < p.rot; ++e) d = fmaf(qs[p.dim + e], to_f(kr[e]), d);
-                sc = d * p.scale;
-            }
-            float mx = sc;
-#pragma unroll
-            for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-            const float m_new = fmaxf(m, mx);
-            const float shrink = expf(m - m_new);      // 0 at the first keys (m = -inf)
-            const float w = expf(sc - m_new);
-            float sum = w;
-#pragma unroll
-            for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-            l = l * shrink + sum;
-            m = m_new;
-#pragma unroll
-            for (int v = 0; v < AW_MAXV; ++v) acc[v] *= shrink;
-            const int nk = min(32, last - k0 + 1);
-            for (int j = 0; j < nk; ++j) {
-                const float wj = __shfl_sync(0xffffffffu, w, j);
-                const T* vr = static_cast<const T*>(p.v) + (seq_row + k0 + j) * p.kv_ld + h * p.vdim;
-#pragma unroll
-                for (int v = 0; v < AW_MAXV; ++v)
-                    if (v * 32 + lane < p.vdim) acc[v] = fmaf(wj, to_f(vr[v * 32 + lane]), acc[v]);
-            }
-        }
-        T* out = static_cast<T*>(p.out) + row * p.out_ld + h * p.vdim;
-#pragma unroll
-        for (int v = 0; v < AW_MAXV; ++v)
-            if (v * 32 + lane < p.vdim) out[v * 32 + lane] = from_f<T>(acc[v] / l);
-        if (h == p.H - 1)                                   // the padding columns behind the last head
-            for (int i = p.H * p.vdim + lane; i < p.out_ld; i += 32)
-                static_cast<T*>(p.out)[row * p.out_ld + i] = from_f<T>(0.f);
-    }
-}
-
-// ---------------------------------------------------------------------------------------------------------------
 // One new token per row: the query moved into latent space.  Block (row group, n tile, head); the last n tile is the
 // rotation.
 //   q_abs[b][h][0..kv_ld) = sum_i q[b][h][i] W_uk[h * dim + i][:]      q_abs[b][h][kv_ld..) = rotated part
@@ -544,21 +472,6 @@ latent_expand_out_kernel(const float* partial, const float* lse, int splits, con
             for (int i = H * vdim + threadIdx.x; i < out_ld; i += blockDim.x) out[(b0 + b) * out_ld + i] = from_f<T>(0.f);
 }
 
-static int sm_count() {
-    int dev = 0, sms = 148;
-    cudaGetDevice(&dev);
-    cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
-    return sms;
-}
-
-template <typename K>
-static int allow_smem(K kernel, size_t bytes, const char* what) {
-    if (bytes <= 48 * 1024) return BN_OK;
-    if (bytes > 200 * 1024) return fail(BN_ERR_UNSUPPORTED, "%s: %zu bytes of shared memory", what, bytes);
-    cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
-    return e == cudaSuccess ? BN_OK : fail(BN_ERR_CUDA, "%s: %s", what, cudaGetErrorString(e));
-}
-
 }  // namespace bn
 
 using namespace bn;
@@ -630,34 +543,6 @@ extern "C" int bn_rope_heads(void* q, int64_t q_ld, int B, int S, int H, int dim
     else
         launch_dependent(rope_heads_kernel<__nv_bfloat16>, grid, 256, 0, as_stream(stream), static_cast<__nv_bfloat16*>(q), q_ld, n,
                          S, H, dim, rot, freq, positions);
-    return launch_status(what);
-}
-
-extern "C" int bn_attn_window(const void* q, int64_t q_ld, const void* k, const void* v, int64_t kv_ld, const void* krot,
-                              int64_t krot_ld, void* out, int64_t out_ld, int B, int S, int n_old, int rows_per_seq, int H,
-                              int dim, int rot, int vdim, int window, float scale, int* error_word, int dtype,
-                              bn_stream_t stream) {
-    const char* what = "bn_attn_window";
-    if (!q || !k || !v || !krot || !out) return fail(BN_ERR_INVALID_ARG, "%s: null pointer", what);
-    if (B < 0 || S < 0 || n_old < 0 || n_old + S > rows_per_seq || H <= 0 || dim <= 0 || rot < 0 || vdim <= 0 || window <= 0 || (dtype & ~1))
-        return fail(BN_ERR_INVALID_ARG, "%s: bad shape B=%d S=%d n_old=%d H=%d dim=%d rot=%d vdim=%d window=%d", what, B, S, n_old,
-                    H, dim, rot, vdim, window);
-    if (int rc = require_sm100()) return rc;
-    if (B == 0 || S == 0) return BN_OK;
-    AttnWindowParams p{q, k, v, krot, out, q_ld, kv_ld, krot_ld, out_ld, B, S, n_old, rows_per_seq, H, dim, rot, vdim, window, scale,
-                       error_word};
-    if (dtype == 1 && attn_window_sm100_ok(p)) return attn_window_sm100(p, as_stream(stream));
-    if (vdim > AW_MAXV * 32) return fail(BN_ERR_UNSUPPORTED, "%s: vdim=%d (at most %d)", what, vdim, AW_MAXV * 32);
-    const size_t smem = (size_t)AW_WARPS * (dim + rot) * sizeof(float);
-    const long long blocks = ((long long)B * S * H + AW_WARPS - 1) / AW_WARPS, cap = (long long)sm_count() * 64;
-    const unsigned grid = (unsigned)(blocks < cap ? blocks : cap);
-    if (dtype == 0) {
-        if (int rc = allow_smem(attn_window_kernel<float>, smem, what)) return rc;
-        launch_dependent(attn_window_kernel<float>, grid, AW_WARPS * 32, smem, as_stream(stream), p);
-    } else {
-        if (int rc = allow_smem(attn_window_kernel<__nv_bfloat16>, smem, what)) return rc;
-        launch_dependent(attn_window_kernel<__nv_bfloat16>, grid, AW_WARPS * 32, smem, as_stream(stream), p);
-    }
     return launch_status(what);
 }
 

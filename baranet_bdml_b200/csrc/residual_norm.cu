@@ -30,19 +30,6 @@ struct ResidualNormParams {
 
 constexpr int RS_THREADS = 256;
 
-// sum over the block, the same bits in every thread
-__device__ __forceinline__ float block_sum(float v, float* sh) {
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-    __syncthreads();                      // sh may still be read from the sum before
-    if (threadIdx.x % 32 == 0) sh[threadIdx.x / 32] = v;
-    __syncthreads();
-    float t = 0.f;
-#pragma unroll
-    for (int w = 0; w < RS_THREADS / 32; ++w) t += sh[w];
-    return t;
-}
-
 // NV = float4 pieces per thread: hidden <= 1024 * NV, hidden % 4 == 0, every row start 16-byte (T = bf16: 8-byte) aligned
 template <typename T, typename TD, int NV>
 __global__ void __launch_bounds__(RS_THREADS)
@@ -79,7 +66,7 @@ residual_norm_regs_kernel(const ResidualNormParams p) {
             for (int k = 0; k < NV; ++k)
 #pragma unroll
                 for (int e = 0; e < 4; ++e) s = fmaf(v[k][e], v[k][e], s);
-            const float inv = rsqrtf(block_sum(s, sh) * inv_n + p.delta_eps);
+            const float inv = rsqrtf(block_sum<RS_THREADS>(s, sh) * inv_n + p.delta_eps);
 #pragma unroll
             for (int k = 0; k < NV; ++k) {
                 const int c = threadIdx.x + k * RS_THREADS;
@@ -122,7 +109,7 @@ residual_norm_regs_kernel(const ResidualNormParams p) {
             }
         }
         if (!p.w) continue;
-        s = block_sum(s, sh) * inv_n;
+        s = block_sum<RS_THREADS>(s, sh) * inv_n;
         float mean = 0.f;
         if (p.center) {
             mean = s;
@@ -133,7 +120,7 @@ residual_norm_regs_kernel(const ResidualNormParams p) {
 #pragma unroll
                     for (int e = 0; e < 4; ++e) q = fmaf(v[k][e] - mean, v[k][e] - mean, q);
                 }
-            s = block_sum(q, sh) * inv_n;
+            s = block_sum<RS_THREADS>(q, sh) * inv_n;
         }
         const float inv = rsqrtf(s + p.eps);
         T* yr = static_cast<T*>(p.y) + (int64_t)r * p.y_ld;
@@ -167,7 +154,7 @@ residual_norm_any_kernel(const ResidualNormParams p) {
         if (dr && p.delta_w) {
             float s = 0.f;
             for (int i = threadIdx.x; i < p.hidden; i += RS_THREADS) { const float d = to_f(dr[i]); s = fmaf(d, d, s); }
-            inv_d = rsqrtf(block_sum(s, sh) / n + p.delta_eps);
+            inv_d = rsqrtf(block_sum<RS_THREADS>(s, sh) / n + p.delta_eps);
         }
         float s = 0.f;
         for (int i = threadIdx.x; i < p.hidden; i += RS_THREADS) {
@@ -185,13 +172,13 @@ residual_norm_any_kernel(const ResidualNormParams p) {
             s += p.center ? v : v * v;
         }
         if (!p.w) continue;
-        s = block_sum(s, sh) / n;
+        s = block_sum<RS_THREADS>(s, sh) / n;
         float mean = 0.f;
         if (p.center) {
             mean = s;
             float q = 0.f;
             for (int i = threadIdx.x; i < p.hidden; i += RS_THREADS) q = fmaf(row_buf[i] - mean, row_buf[i] - mean, q);
-            s = block_sum(q, sh) / n;
+            s = block_sum<RS_THREADS>(q, sh) / n;
         }
         const float inv = rsqrtf(s + p.eps);
         T* yr = static_cast<T*>(p.y) + (int64_t)r * p.y_ld;
@@ -242,6 +229,15 @@ act_mul_kernel(const float* a, int64_t a_ld, const float* b, int64_t b_ld, float
     }
 }
 
+// x = act(x + bias) in place, fp32 rows (the unfused form of the products with a bias or an activation)
+__global__ void __launch_bounds__(256)
+bias_act_kernel(float* x, int64_t ld, const float* bias, long long n, int cols, int act) {
+    for (long long i = (long long)blockIdx.x * 256 + threadIdx.x; i < n; i += (long long)gridDim.x * 256) {
+        const int64_t r = i / cols, c = i - r * cols;
+        x[r * ld + c] = activation_exact(act, x[r * ld + c] + (bias ? bias[c] : 0.f));
+    }
+}
+
 }  // namespace bn
 
 using namespace bn;
@@ -276,4 +272,15 @@ extern "C" int bn_act_mul_f32(const float* a, int64_t a_ld, const float* b, int6
     act_mul_kernel<<<(unsigned)(blocks < 4096 ? blocks : 4096), 256, 0, as_stream(stream)>>>(a, a_ld, b, b_ld, out, out_ld, n,
                                                                                        cols, act);
     return launch_status("bn_act_mul_f32");
+}
+
+extern "C" int bn_bias_act_f32(float* x, int64_t ld, const float* bias, int rows, int cols, int act, bn_stream_t stream) {
+    if (!x) return fail(BN_ERR_INVALID_ARG, "bn_bias_act_f32: null pointer");
+    if (rows < 0 || cols < 0 || act < 0 || act > BN_ACT_LAST) return fail(BN_ERR_INVALID_ARG, "bn_bias_act_f32: bad shape or activation");
+    if (int rc = require_sm100()) return rc;
+    const long long n = (long long)rows * cols;
+    if (n == 0) return BN_OK;
+    const long long blocks = (n + 255) / 256;
+    bias_act_kernel<<<(unsigned)(blocks < 4096 ? blocks : 4096), 256, 0, as_stream(stream)>>>(x, ld, bias, n, cols, act);
+    return launch_status("bn_bias_act_f32");
 }

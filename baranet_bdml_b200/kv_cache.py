@@ -127,6 +127,38 @@ class LatentRingCache:
             seq_ids.numel(), n_old, latents.data_ptr(), keys.data_ptr(), rows_per_seq, _dt(self.dtype), _stream()))
 
 
+class ChunkCache:
+    """Keys and values of a sequence's current chunk of positions, for attention that never looks behind a chunk's start: the
+    token of position p in row p % chunk, so the next chunk overwrites the one before it.  `max_tokens` (the most tokens a
+    sequence will have) bounds the rows where it is less than a chunk.
+
+    k[slot][kv_head][ring_tokens][round8(dim)], v likewise, zeros behind the values."""
+
+    def __init__(self, num_seqs: int, chunk: int, kv_heads: int, dim: int, vdim: int, dtype=torch.bfloat16,
+                 max_tokens: Optional[int] = None, groups: int = 1, device="cuda"):
+        from .ops import round8
+        self.num_seqs, self.chunk, self.kv_heads, self.dtype = num_seqs, chunk, kv_heads, dtype
+        self.dim_ld, self.vdim_ld = round8(dim), round8(vdim)
+        self.ring_tokens = chunk if max_tokens is None else max(1, min(chunk, max_tokens))
+        self.k = torch.zeros((num_seqs, kv_heads, self.ring_tokens, self.dim_ld), dtype=dtype, device=device)
+        self.v = torch.zeros((num_seqs, kv_heads, self.ring_tokens, self.vdim_ld), dtype=dtype, device=device)
+        self.tickets = torch.zeros(num_seqs * kv_heads * groups, dtype=torch.int32, device=device)   # of the one-token kernel, left zero by it
+
+    def reset(self, slot: int) -> None:
+        """Nothing to clear: a row is read only for positions that the sequence itself has written."""
+
+    def tensors(self):
+        return [self.k, self.v]
+
+    def gather(self, seq_ids, positions, n_old: int, k: torch.Tensor, v: torch.Tensor, rows_per_seq: int) -> None:
+        """The n_old = positions % chunk tokens before `positions` to the first rows of each sequence's block of k / v."""
+        from .ops import _dt
+        _lib.check(_lib.load().bn_kv_gather(
+            self.k.data_ptr(), self.v.data_ptr(), self.ring_tokens, self.chunk, self.kv_heads, self.dim_ld, self.vdim_ld,
+            seq_ids.data_ptr(), positions.data_ptr(), seq_ids.numel(), n_old, k.data_ptr(), v.data_ptr(), rows_per_seq,
+            _dt(self.dtype), _stream()))
+
+
 class RecurrentState:
     """What a Mamba-2 layer keeps of a sequence: its state matrices, fp32, and the convolution's last inputs in a ring
     (the input of position p in row p % taps)."""

@@ -1,6 +1,6 @@
-"""Sublayers of the models whose layers mix attention and recurrence, in fp32 and in bf16: latent attention with a sliding
-window, the Mamba-2 mixer, a gated MLP with a choice of activation, and the per-layer token input.  Sizes and constants are
-parameters; weights come from a function name -> tensor.
+"""Sublayers of the models that are served from per-sequence slots, in fp32 and in bf16: latent attention with a sliding
+window, grouped-query attention in chunks, the Mamba-2 mixer, MLPs with a choice of activation, and the per-layer token
+input.  Sizes and constants are parameters; weights come from a function name -> tensor.
 
 A mixer is called with the rows of B sequences x S new tokens: `seq_ids` (B) are the sequences' slots in its cache or state
 (which `new_state` makes), `positions` (B) the position of each one's first new token, both int32 on the GPU.  `n_old` is how
@@ -14,7 +14,7 @@ from typing import Callable, Optional
 import torch
 
 from . import _lib, ops
-from .kv_cache import LatentRingCache, RecurrentState
+from .kv_cache import ChunkCache, LatentRingCache, RecurrentState
 from .ops import _dt, _ptr, _stream, round8
 
 
@@ -115,6 +115,107 @@ class LatentAttention:
 
 
 @dataclass(frozen=True)
+class ChunkedAttentionConfig:
+    heads: int
+    kv_heads: int
+    dim: int                # per-head query / key columns
+    vdim: int
+    chunk: int              # a position sees its own chunk up to itself; chunks start at the multiples of this
+    scale: float
+    mixes_values: bool      # whether the layer takes part in value mixing
+
+    def __post_init__(self):
+        if min(self.heads, self.kv_heads, self.dim, self.vdim, self.chunk) <= 0 or self.heads % self.kv_heads:
+            raise ValueError(f"chunked attention: bad sizes {self}")
+
+
+def pad_heads(rows: torch.Tensor, heads: int, dim: int) -> torch.Tensor:
+    """(heads * dim, ...) -> (heads * round8(dim), ...), zeros behind each head: every head starts on a 16-byte boundary."""
+    out = torch.zeros((heads, round8(dim)) + tuple(rows.shape[1:]), dtype=rows.dtype, device=rows.device)
+    out[:, :dim] = rows.reshape((heads, dim) + tuple(rows.shape[1:]))
+    return out.reshape((heads * round8(dim),) + tuple(rows.shape[1:]))
+
+
+class ChunkedAttention:
+    """Grouped-query attention in chunks of positions, unit-RMS queries and keys, no rotation, a sigmoid gate on the heads'
+    outputs, biases on the projections, and values mixed with those of an earlier layer.
+
+    `project` gives the rows [q | k | v | gate] that everything else reads; `values` is the v of them, which a later layer may
+    take as `v_first`."""
+
+    def __init__(self, cfg: ChunkedAttentionConfig, width: int, eps: float, weight: Callable, dtype):
+        c = cfg
+        self.cfg, self.dtype, self.eps = cfg, dtype, float(eps)
+        self.dim_ld, self.vdim_ld = round8(c.dim), round8(c.vdim)
+        self.head_groups = -(-(c.heads // c.kv_heads) // 16)                          # of 16 query heads per key head
+        sizes = [("q", c.heads, c.dim), ("k", c.kv_heads, c.dim), ("v", c.kv_heads, c.vdim), ("g", c.heads, c.vdim)]
+        w = [pad_heads(weight(n, h * d, width), h, d) for n, h, d in sizes]
+        b = [pad_heads(weight(n + ".b", h * d), h, d) for n, h, d in sizes[:3]]
+        b.append(torch.zeros(w[3].shape[0], dtype=b[0].dtype, device=b[0].device))                      # the gate has no bias
+        self.proj = ops.Linear(torch.cat(w), dtype, bias=torch.cat(b))
+        self.cols = [0]
+        for part in w:
+            self.cols.append(self.cols[-1] + part.shape[0])
+        o = weight("o", width, c.heads * c.vdim)
+        self.o = ops.Linear(pad_heads(o.t(), c.heads, c.vdim).t(), dtype, bias=weight("o.b", width))
+        self.mix = float(weight("vmix").reshape(-1)[0]) if c.mixes_values else 0.0
+
+    def new_state(self, num_seqs: int, max_tokens: Optional[int] = None) -> ChunkCache:
+        c = self.cfg
+        return ChunkCache(num_seqs, c.chunk, c.kv_heads, c.dim, c.vdim, self.dtype, max_tokens, self.head_groups)
+
+    def project(self, h: torch.Tensor) -> torch.Tensor:
+        return self.proj(h)
+
+    def values(self, proj: torch.Tensor) -> torch.Tensor:
+        return proj[:, self.cols[2]:self.cols[3]]
+
+    def __call__(self, proj: torch.Tensor, B: int, S: int, cache: ChunkCache, seq_ids, positions, n_old: Optional[int],
+                 v_first: Optional[torch.Tensor] = None):
+        c = self.cfg
+        if v_first is not None and (v_first.dtype != self.dtype or tuple(v_first.shape) != (B * S, c.kv_heads * self.vdim_ld)):
+            raise RuntimeError("chunked attention: the values to mix in must have this layer's heads and sizes")
+        out = torch.empty((B * S, self.o.k), dtype=self.dtype, device=proj.device)
+        (self._one_token if n_old is None else self._portion)(proj, B, S, cache, seq_ids, positions, n_old, v_first, out)
+        return self.o(out)
+
+    def _columns(self, proj):
+        """pointers to the q, k, v and gate columns"""
+        return [proj.data_ptr() + at * proj.element_size() for at in self.cols[:4]]
+
+    def _portion(self, proj, B, S, cache, seq_ids, positions, n_old, v_first, out):
+        c, dev, dt, lib, s = self.cfg, proj.device, _dt(self.dtype), _lib.load(), _stream()
+        q, k, v, g = self._columns(proj)
+        n_old %= c.chunk                                      # the tokens of the portion's first chunk that it still sees
+        n = n_old + S
+        keys = torch.empty((B * n, c.kv_heads * self.dim_ld), dtype=self.dtype, device=dev)
+        values = torch.empty((B * n, c.kv_heads * self.vdim_ld), dtype=self.dtype, device=dev)
+        if n_old:                                             # before the portion's own rows replace any in the cache
+            cache.gather(seq_ids, positions, n_old, keys, values, n)
+        _lib.check(lib.bn_kv_prep(
+            k, v, proj.stride(0), _ptr(v_first), 0 if v_first is None else v_first.stride(0), self.mix, seq_ids.data_ptr(),
+            positions.data_ptr(), B, S, c.kv_heads, self.dim_ld, self.vdim_ld, c.dim, self.eps, keys.data_ptr(), values.data_ptr(), n,
+            n_old, cache.k.data_ptr(), cache.v.data_ptr(), cache.ring_tokens, c.chunk, dt, s))
+        _lib.check(lib.bn_attn_chunked(
+            q, proj.stride(0), keys.data_ptr(), keys.stride(0), values.data_ptr(), values.stride(0), g, proj.stride(0), out.data_ptr(),
+            out.stride(0), B, S, n_old, n, c.heads, c.kv_heads, self.dim_ld, self.vdim_ld, c.chunk, c.dim, self.eps, float(c.scale),
+            ops.status_word(dev).data_ptr(), dt, s))
+
+    def _one_token(self, proj, B, S, cache, seq_ids, positions, n_old, v_first, out):
+        c, dev, dt, lib = self.cfg, proj.device, _dt(self.dtype), _lib.load()
+        q, k, v, g = self._columns(proj)
+        splits = lib.bn_gqa_step_splits(B, c.heads, c.kv_heads, self.dim_ld, self.vdim_ld, cache.ring_tokens, dt)
+        partial = None
+        if splits > 1:
+            partial = torch.empty(B * c.kv_heads * self.head_groups * splits * 16 * (self.vdim_ld + 2), dtype=torch.float32, device=dev)
+        _lib.check(lib.bn_gqa_step(
+            q, k, v, g, proj.stride(0), _ptr(v_first), 0 if v_first is None else v_first.stride(0), self.mix, cache.k.data_ptr(),
+            cache.v.data_ptr(), cache.num_seqs, cache.ring_tokens, c.chunk, seq_ids.data_ptr(), positions.data_ptr(), _ptr(partial),
+            cache.tickets.data_ptr(), splits, out.data_ptr(), out.stride(0), B, c.heads, c.kv_heads, self.dim_ld, self.vdim_ld, c.dim,
+            self.eps, float(c.scale), ops.status_word(dev).data_ptr(), dt, _stream()))
+
+
+@dataclass(frozen=True)
 class Mamba2Config:
     heads: int
     vdim: int
@@ -193,6 +294,17 @@ class GatedMLP:
 
     def __call__(self, h: torch.Tensor) -> torch.Tensor:
         return self.down(self.gate_up(h))
+
+
+class MLP:
+    """down(act(up x))"""
+
+    def __init__(self, inter: int, width: int, act: str, weight: Callable, dtype):
+        self.up = ops.Linear(weight("up", inter, width), dtype, act=act)
+        self.down = ops.Linear(weight("down", width, inter), dtype)
+
+    def __call__(self, h: torch.Tensor) -> torch.Tensor:
+        return self.down(self.up(h))
 
 
 class TokenSide:

@@ -10,13 +10,13 @@ Greedy decoding only (temperature / top-k sampling of the reference is host code
 """
 from __future__ import annotations
 
-from typing import List, Optional
+from typing import List, Optional, Sequence
 
 import numpy as np
 import torch
 
 from . import _lib, ops
-from .kv_cache import PAGE_TOKENS, PagedKVCache
+from .kv_cache import PAGE_TOKENS, PagedKVCache, SequenceSlots
 from .layers import LLaMAConfig, LLaMADecoderLayerBF16
 
 
@@ -93,6 +93,96 @@ class CausalLM:
                 break
             logits = self.decode_step(nxt)
         return out
+
+
+class SequenceLM(CausalLM):
+    """A model whose layers keep caches and states per sequence slot: prompts in portions of any size, sequences of unequal
+    lengths in one step, slots that are given back and used again.
+
+    A family supplies
+      new_states(num_seqs, max_tokens)   one state per layer run (reset(slot), tensors()); max_tokens: the most tokens a
+                                         sequence will have, or None
+      _forward(ids, B, S, seq_ids, positions, n_old)   all layers over B x S new tokens -> whatever _logits takes.  `n_old`:
+                                         how many earlier tokens each of the B sequences has; None with S = 1 selects the
+                                         one-token kernels, for which the sequences' lengths may differ
+      _select(state, rows)               the same for some of the B * S rows
+      _logits(state)                     fp32 logits of those rows
+    and raises the int32 `_id_error` on the GPU for a token id outside the vocabulary."""
+
+    ragged_prompts = True
+
+    def __init__(self, config, dtype):
+        self.config, self.dtype = config, dtype
+        self.slots: Optional[SequenceSlots] = None
+        self._id_error = torch.zeros(1, dtype=torch.int32, device="cuda")
+
+    def allocate(self, num_seqs: int, max_tokens: Optional[int] = None) -> None:
+        """Caches and states for `num_seqs` sequences of at most `max_tokens` tokens (None: of any length)."""
+        self.max_tokens = max_tokens
+        self.states = self.new_states(num_seqs, max_tokens)
+        self.slots = SequenceSlots(num_seqs, self.states)
+        self._all_slots = torch.arange(num_seqs, dtype=torch.int32, device="cuda")
+
+    @property
+    def seq_lens(self) -> torch.Tensor:
+        return self.slots.lens
+
+    def state_tensors(self):
+        return self.slots.tensors()
+
+    def _check_ids(self):
+        if int(self._id_error.item()) != 0:
+            self._id_error.zero_()
+            raise IndexError("token id out of range")
+
+    def extend(self, ids: torch.Tensor, slots: Sequence[int], want: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """The next S tokens of the sequences in `slots`, which all have seen equally many: ids (B, S) int32.  Returns the
+        fp32 logits of the rows `want` (indices into the B * S rows; None: the last row of every sequence)."""
+        B, S = ids.shape
+        flat = ids.reshape(-1).to(torch.int32).contiguous()
+        seq_ids = torch.tensor(list(slots), dtype=torch.int32, device="cuda")
+        positions = self.seq_lens.index_select(0, seq_ids)
+        seen = set(positions.tolist())
+        if len(seen) != 1:
+            raise RuntimeError("extend: the sequences of a portion must have equal lengths")
+        n_old = seen.pop()
+        if self.max_tokens is not None and n_old + S > self.max_tokens:
+            raise RuntimeError(f"extend: {n_old + S} tokens in a sequence; the caches were allocated for {self.max_tokens}")
+        state = self._forward(flat, B, S, seq_ids, positions, None if S == 1 else n_old)
+        self._check_ids()
+        self.seq_lens.index_add_(0, seq_ids, torch.full_like(seq_ids, S))
+        if want is None:
+            want = torch.arange(B, device="cuda") * S + S - 1
+        if want.numel() == 0:
+            return torch.empty((0, self.config.vocab_size), dtype=torch.float32, device="cuda")
+        if want.numel() != B * S or S > 1:
+            state = self._select(state, want)
+        return self._logits(state)
+
+    def prefill(self, input_ids, max_len: int) -> torch.Tensor:
+        """Prompts, (B, S) ids or a list of id lists of any lengths -> logits of each one's last position, (B, vocab)."""
+        prompts = list(input_ids)
+        self.allocate(len(prompts), max(max_len, max(len(p) for p in prompts)))
+        slots = [self.slots.acquire() for _ in prompts]
+        as_ids = lambda p: torch.as_tensor(p).to(device="cuda", dtype=torch.int32)     # noqa: E731
+        if len({len(p) for p in prompts}) == 1:
+            return self.extend(torch.stack([as_ids(p) for p in prompts]), slots)
+        return torch.cat([self.extend(as_ids(p)[None], [s]) for p, s in zip(prompts, slots)])
+
+    def decode_step(self, token_ids: torch.Tensor, check: bool = True, slots: Optional[Sequence[int]] = None) -> torch.Tensor:
+        """One new token for the sequences in `slots` (None: the first B slots), whatever their lengths."""
+        B = token_ids.numel()
+        seq_ids = self._all_slots[:B] if slots is None else torch.tensor(list(slots), dtype=torch.int32, device="cuda")
+        positions = self.seq_lens.index_select(0, seq_ids)
+        state = self._forward(token_ids.reshape(-1).to(torch.int32).contiguous(), B, 1, seq_ids, positions, None)
+        self.seq_lens.index_add_(0, seq_ids, torch.ones_like(seq_ids))
+        if check:
+            self._check_ids()
+        return self._logits(state)
+
+    def status(self) -> None:
+        """Raises if a kernel gave up a bounded wait since the last check.  Synchronises."""
+        ops.gemm_status()
 
 
 class LLaMAModelBF16(CausalLM):

@@ -3,6 +3,7 @@ used for device memory and streams only; all arithmetic is in libbn_attn.so).
 """
 from __future__ import annotations
 
+import ctypes as C
 from typing import Optional, Tuple
 
 import torch
@@ -410,7 +411,7 @@ def lse_combine(outs: torch.Tensor, lses: torch.Tensor, *, out_dtype=torch.float
 # Operators that exist in fp32 and in bf16 (dtype of the activations decides); row strides may exceed the row, so that
 # rows of any width start on 16-byte boundaries.
 # ---------------------------------------------------------------------------------------------------------------------
-ACTIVATIONS = {"none": _lib.BN_ACT_NONE, "silu": _lib.BN_ACT_SILU, "gelu_tanh": _lib.BN_ACT_GELU_TANH}
+ACTIVATIONS = {"none": _lib.BN_ACT_NONE, "silu": _lib.BN_ACT_SILU, "gelu_tanh": _lib.BN_ACT_GELU_TANH, "relu2": _lib.BN_ACT_RELU2}
 
 
 def round8(n: int) -> int:
@@ -436,12 +437,16 @@ def _rows(t: torch.Tensor, what: str) -> torch.Tensor:
 
 
 class Linear:
-    """y = x W^T for a weight (out, in): bf16 on the tensor cores, or true fp32 (`bn_mm_f32`).  Both sizes are rounded up to
-    multiples of 8 with zeros, so x may be passed with its padding columns (which must be finite) and y has them."""
+    """y = act(x W^T + bias) for a weight (out, in), bias (out) and act optional: bf16 on the tensor cores, or true fp32
+    (`bn_mm_f32`).  Both sizes are rounded up to multiples of 8 with zeros, so x may be passed with its padding columns (which
+    must be finite) and y has them."""
 
-    def __init__(self, weight: torch.Tensor, dtype, device="cuda"):
+    def __init__(self, weight: torch.Tensor, dtype, device="cuda", bias: Optional[torch.Tensor] = None, act: str = "none"):
         self.out_features, self.in_features = weight.shape
-        self.dtype = dtype
+        self.dtype, self.act, self.bias = dtype, act, None
+        if bias is not None:
+            self.bias = torch.zeros(round8(self.out_features), dtype=torch.float32, device=device)
+            self.bias[:self.out_features] = bias.to(device=device, dtype=torch.float32)
         self.n, self.k = round8(self.out_features), round8(self.in_features)
         self.weight = torch.zeros((self.n, self.k), dtype=dtype, device=device)
         self.weight[:self.out_features, :self.in_features] = weight.to(device)
@@ -468,10 +473,17 @@ class Linear:
         """(rows, in) -> (rows, out rounded up to a multiple of 8); `f32_out`: the fp32 accumulators themselves."""
         x = self._operand(x)
         rows = x.shape[0]
+        plain = self.bias is None and self.act == "none"
         if self.dtype == torch.float32:
-            return self._mm_f32(x, torch.empty((rows, self.n), dtype=torch.float32, device=x.device))
+            out = self._mm_f32(x, torch.empty((rows, self.n), dtype=torch.float32, device=x.device))
+            if not plain:
+                _lib.check(_lib.load().bn_bias_act_f32(out.data_ptr(), self.n, _ptr(self.bias), rows, self.n, ACTIVATIONS[self.act],
+                                                       _stream()))
+            return out
         if not f32_out:
-            return linear_bf16(x, self.weight)
+            return linear_bf16(x, self.weight) if plain else self._bias_act(x)
+        if not plain:
+            raise RuntimeError("linear: the fp32 result has neither a bias nor an activation")
         out = torch.empty((rows, self.n), dtype=torch.float32, device=x.device)
         lib = _lib.load()
         if skinny_any_k(rows, self.n, self.k):
@@ -486,8 +498,26 @@ class Linear:
                                                _gemm_error_ptr(x.device, None), _stream()))
         return out
 
+    def _bias_act(self, x: torch.Tensor) -> torch.Tensor:
+        rows, a, lib = x.shape[0], ACTIVATIONS[self.act], _lib.load()
+        out = torch.empty((rows, self.n), dtype=self.dtype, device=x.device)
+        if skinny_any_k(rows, self.n, self.k):
+            _lib.check(lib.bn_gemm_bias_act_bf16_nt_skinny(x.data_ptr(), self.weight.data_ptr(), _ptr(self.bias), out.data_ptr(), rows,
+                                                           self.n, self.k, a, _stream()))
+        elif small_m_ok(rows, self.n):
+            ws, n = _small_m_scratch(x.device, rows, self.n, self.k)
+            _lib.check(lib.bn_gemm_bias_act_bf16_nt_small_m(x.data_ptr(), self.weight.data_ptr(), _ptr(self.bias), out.data_ptr(), rows,
+                                                            self.n, self.k, a, ws.data_ptr(), n, _gemm_error_ptr(x.device, None),
+                                                            _stream()))
+        else:
+            _lib.check(lib.bn_gemm_bias_act_bf16_nt(x.data_ptr(), self.weight.data_ptr(), _ptr(self.bias), out.data_ptr(), rows, self.n,
+                                                    self.k, a, _gemm_error_ptr(x.device, None), _stream()))
+        return out
+
     def act_mul(self, x: torch.Tensor, mul: torch.Tensor, act: str) -> torch.Tensor:
         """act(x W^T) * mul, mul (rows, >= out rounded up) with any row stride that is a multiple of 8."""
+        if self.bias is not None or self.act != "none":
+            raise RuntimeError("act_mul: a product without a bias and an activation of its own")
         x = self._operand(x)
         rows, a = x.shape[0], ACTIVATIONS[act]
         _rows(mul, "act_mul(mul)")
@@ -608,6 +638,59 @@ def residual_norm(x: Optional[torch.Tensor], pending: Optional[Pending], dtype, 
         None if norm is None or norm.bias is None else norm.bias.data_ptr(), _ptr(y), 0 if y is None else y.stride(0),
         int(norm is not None and norm.center), _dt(dtype), rows, hidden, 0.0 if norm is None else norm.eps, _stream()))
     return (total if changed else x), y
+
+
+class StreamMix:
+    """How the fp32 streams of a residual that is kept several times go from one sublayer to the next: a matrix from the old
+    streams to the new ones, what each new stream takes of the pending sublayer output, and the weights of the sum that the
+    next sublayer reads.  With `keep` False the new streams are not wanted: the sum is folded into one."""
+
+    def __init__(self, mix, w_out, w_in, keep: bool = True):
+        n_in, n_out = len(mix), len(w_in)
+        if not keep:
+            mix = [[sum(m * w for m, w in zip(row, w_in))] for row in mix]
+            w_out, w_in, n_out = [sum(o * w for o, w in zip(w_out, w_in))], [1.0], 1
+        self.n_in, self.n_out, self.keep = n_in, n_out, keep
+        self.mix = (C.c_float * (n_in * n_out))(*[float(v) for row in mix for v in row])
+        self.w_out, self.w_in = (C.c_float * n_out)(*map(float, w_out)), (C.c_float * n_out)(*map(float, w_in))
+
+
+def hyper_norm(x: torch.Tensor, step: StreamMix, dtype, norm: NormWeight, *, delta: Optional[torch.Tensor] = None,
+               delta_scale: Optional[torch.Tensor] = None):
+    """x (rows, n_in, hidden) fp32 -> (the new streams (rows, n_out, hidden) or None, the RMS norm of their weighted sum in
+    `dtype`)."""
+    _need(x, torch.float32, "hyper_norm(x)")
+    rows, n_in, hidden = x.shape
+    if n_in != step.n_in or norm.center:
+        raise RuntimeError(f"hyper_norm: {n_in} streams where {step.n_in} are mixed, or a norm that is not an RMS norm")
+    if delta is not None and (_rows(delta, "hyper_norm(delta)").dtype != dtype or delta.shape[0] != rows or delta.shape[1] < hidden):
+        raise RuntimeError("hyper_norm: the sublayer's output must have the streams' rows and the activations' dtype")
+    out = torch.empty((rows, step.n_out, hidden), dtype=torch.float32, device=x.device) if step.keep else None
+    y = torch.empty((rows, round8(hidden)), dtype=dtype, device=x.device)
+    if y.shape[1] != hidden:
+        y[:, hidden:] = 0
+    _lib.check(_lib.load().bn_hyper_norm(
+        x.data_ptr(), n_in, step.n_out, step.mix, step.w_out, step.w_in, _ptr(delta), 0 if delta is None else delta.stride(0),
+        _ptr(delta_scale), _ptr(out), norm.weight.data_ptr(), y.data_ptr(), y.stride(0), _dt(dtype), rows, hidden, norm.eps, _stream()))
+    return out, y
+
+
+def tensors_of(value) -> list:
+    """The distinct tensors in a value: tensors themselves, sequences, and the attributes of this package's objects."""
+    out, seen = [], set()
+
+    def walk(v):
+        if isinstance(v, torch.Tensor):
+            if v.data_ptr() not in seen:
+                seen.add(v.data_ptr())
+                out.append(v)
+        elif isinstance(v, (list, tuple)):
+            for e in v:
+                walk(e)
+        elif type(v).__module__.startswith(__package__ + "."):
+            walk(list(vars(v).values()))
+    walk(value)
+    return out
 
 
 def rotation_frequencies(rot_dim: int, base: float, device="cuda") -> torch.Tensor:

@@ -36,8 +36,15 @@ def _soluzen(config: dict, weights: Optional[Weights], dtype):
     return SoluzenModel(SoluzenConfig.from_dict(config), weights, dtype)
 
 
+def _duponex(config: dict, weights: Optional[Weights], dtype):
+    from .duponex import DuponexConfig, DuponexModel
+    if weights is None:
+        raise RuntimeError("a Duponex model needs its checkpoint")
+    return DuponexModel(DuponexConfig.from_dict(config), weights, dtype)
+
+
 # architecture -> (family whose kernels it launches, constructor)
-ARCHITECTURES = {"LLaMA": ("llama", _llama), "Soluzen": ("soluzen", _soluzen)}
+ARCHITECTURES = {"LLaMA": ("llama", _llama), "Soluzen": ("soluzen", _soluzen), "Duponex": ("duponex", _duponex)}
 
 
 def build_model(config: dict, weights: Optional[Weights], dtype=torch.bfloat16):

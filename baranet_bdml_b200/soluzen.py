@@ -13,9 +13,8 @@ import torch
 
 from . import ops
 from .checkpoint import Weights
-from .kv_cache import SequenceSlots
 from .mixers import GatedMLP, LatentAttention, LatentAttentionConfig, Mamba2Config, Mamba2Mixer, TokenSide
-from .model import CausalLM
+from .model import SequenceLM
 from .ops import Pending, round8
 
 MIXERS = {"latent_attention": LatentAttention, "mamba2": Mamba2Mixer}
@@ -101,15 +100,13 @@ class SoluzenLayer:
         self.side = TokenSide(model.side_dim, model.width, model.eps, ACTIVATION, part("side"), dtype)
 
 
-class SoluzenModel(CausalLM):
+class SoluzenModel(SequenceLM):
     """The residual stream is fp32 in both dtypes; what reads it is normalised or rounded by the launch that adds the
     sublayer before it (ops.residual_norm)."""
 
-    ragged_prompts = True
-
     def __init__(self, config: SoluzenConfig, weights: Weights, dtype=torch.bfloat16):
+        super().__init__(config, dtype)
         c, w = config, weights
-        self.config, self.dtype = c, dtype
         n, width, w8 = len(c.layers), c.width, round8(c.width)
         self.embed_tokens = w("embed", c.vocab_size, width).to(device="cuda", dtype=dtype).contiguous()
         # each layer's part of the token input starts on a 16-byte boundary
@@ -133,22 +130,11 @@ class SoluzenModel(CausalLM):
         self.head = ops.Linear(w("head", c.vocab_size, width), dtype)
         if w.leftover():
             warnings.warn(f"checkpoint tensors that this design does not have: {w.leftover()[:5]}")
-        self.slots: Optional[SequenceSlots] = None
-        self._id_error = torch.zeros(1, dtype=torch.int32, device="cuda")
 
     # ------------------------------------------------------------------ sequences
-    def allocate(self, num_seqs: int) -> None:
-        """Caches and states for `num_seqs` sequences: one per layer run, so each pass of the loop has its own."""
-        self.states = [self.layers[i].mixer.new_state(num_seqs) for i, _ in self.runs]
-        self.slots = SequenceSlots(num_seqs, self.states)
-        self._all_slots = torch.arange(num_seqs, dtype=torch.int32, device="cuda")
-
-    @property
-    def seq_lens(self) -> torch.Tensor:
-        return self.slots.lens
-
-    def state_tensors(self):
-        return self.slots.tensors()
+    def new_states(self, num_seqs: int, max_tokens: Optional[int]):
+        """One per layer run, so each pass of the loop has its own; their size does not depend on a sequence's length."""
+        return [self.layers[i].mixer.new_state(num_seqs) for i, _ in self.runs]
 
     # -------------------------------------------------------------------- forward
     def _embed(self, ids: torch.Tensor):
@@ -171,7 +157,7 @@ class SoluzenModel(CausalLM):
         return x, side, cat
 
     def _forward(self, ids: torch.Tensor, B: int, S: int, seq_ids, positions, n_old: Optional[int]):
-        """All layers over B x S new tokens: the residual stream with its last addend still pending."""
+        """All layers over B x S new tokens: (the residual stream, its last addend, still pending)."""
         c, dt, width, w8, s8 = self.config, self.dtype, self.config.width, round8(self.config.width), self.side8
         x, side, cat = self._embed(ids)
         pending, row = None, None
@@ -191,75 +177,15 @@ class SoluzenModel(CausalLM):
             pending = layer.side(xb, side[:, i * s8:(i + 1) * s8])
         return x, pending
 
-    def _logits(self, x: torch.Tensor, pending: Pending) -> torch.Tensor:
+    def _select(self, state, rows: torch.Tensor):
+        x, pending = state
+        return x.index_select(0, rows), pending.select(rows)
+
+    def _logits(self, state) -> torch.Tensor:
+        x, pending = state
         _, h = ops.residual_norm(x, pending, self.dtype, self.config.width, norm=self.final_norm, keep_sum=False)
         return self.head(h, f32_out=True)[:, :self.config.vocab_size]
 
-    def _check_ids(self):
-        if int(self._id_error.item()) != 0:
-            self._id_error.zero_()
-            raise IndexError("token id out of range")
-
-    def extend(self, ids: torch.Tensor, slots: Sequence[int], want: Optional[torch.Tensor] = None) -> torch.Tensor:
-        """The next S tokens of the sequences in `slots`, which all have seen equally many: ids (B, S) int32.  Returns the
-        fp32 logits of the rows `want` (indices into the B * S rows; None: the last row of every sequence)."""
-        B, S = ids.shape
-        flat = ids.reshape(-1).to(torch.int32).contiguous()
-        seq_ids = torch.tensor(list(slots), dtype=torch.int32, device="cuda")
-        positions = self.seq_lens.index_select(0, seq_ids)
-        seen = set(positions.tolist())
-        if len(seen) != 1:
-            raise RuntimeError("extend: the sequences of a portion must have equal lengths")
-        x, pending = self._forward(flat, B, S, seq_ids, positions, None if S == 1 else seen.pop())
-        self._check_ids()
-        self.seq_lens.index_add_(0, seq_ids, torch.full_like(seq_ids, S))
-        if want is None:
-            want = torch.arange(B, device="cuda") * S + S - 1
-        if want.numel() == 0:
-            return torch.empty((0, self.config.vocab_size), dtype=torch.float32, device="cuda")
-        if want.numel() != B * S or S > 1:
-            x, pending = x.index_select(0, want), pending.select(want)
-        return self._logits(x, pending)
-
-    def prefill(self, input_ids, max_len: int) -> torch.Tensor:
-        """Prompts, (B, S) ids or a list of id lists of any lengths -> logits of each one's last position, (B, vocab)."""
-        prompts = list(input_ids)
-        self.allocate(len(prompts))
-        slots = [self.slots.acquire() for _ in prompts]
-        as_ids = lambda p: torch.as_tensor(p).to(device="cuda", dtype=torch.int32)     # noqa: E731
-        if len({len(p) for p in prompts}) == 1:
-            return self.extend(torch.stack([as_ids(p) for p in prompts]), slots)
-        return torch.cat([self.extend(as_ids(p)[None], [s]) for p, s in zip(prompts, slots)])
-
-    def decode_step(self, token_ids: torch.Tensor, check: bool = True, slots: Optional[Sequence[int]] = None) -> torch.Tensor:
-        """One new token for the sequences in `slots` (None: the first B slots), whatever their lengths."""
-        B = token_ids.numel()
-        seq_ids = self._all_slots[:B] if slots is None else torch.tensor(list(slots), dtype=torch.int32, device="cuda")
-        positions = self.seq_lens.index_select(0, seq_ids)
-        x, pending = self._forward(token_ids.reshape(-1).to(torch.int32).contiguous(), B, 1, seq_ids, positions, None)
-        self.seq_lens.index_add_(0, seq_ids, torch.ones_like(seq_ids))
-        if check:
-            self._check_ids()
-        return self._logits(x, pending)
-
-    def status(self) -> None:
-        """Raises if a kernel gave up a bounded wait since the last check.  Synchronises."""
-        ops.gemm_status()
-
     def parameters(self) -> List[torch.Tensor]:
-        out, seen = [], set()
-
-        def walk(v):
-            if isinstance(v, torch.Tensor):
-                if v.data_ptr() not in seen:
-                    seen.add(v.data_ptr())
-                    out.append(v)
-            elif isinstance(v, (list, tuple)):
-                for e in v:
-                    walk(e)
-            elif isinstance(v, (SoluzenLayer, LatentAttention, Mamba2Mixer, GatedMLP, TokenSide, ops.Linear, ops.GatedLinear,
-                                ops.NormWeight)):
-                walk(list(vars(v).values()))
-        walk([self.embed_tokens, self.side_embed, self.layers, getattr(self, "loop_in", None), getattr(self, "loop_step", None),
-              self.final_norm, self.head])
-        return out
+        return ops.tensors_of([self.embed_tokens, self.side_embed, self.layers, getattr(self, "loop_in", None),
+                               getattr(self, "loop_step", None), self.final_norm, self.head])

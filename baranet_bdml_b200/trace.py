@@ -10,6 +10,7 @@ import argparse
 import json
 import os
 import sys
+from typing import Optional
 
 import numpy as np
 import torch
@@ -18,9 +19,9 @@ import torch
 class TraceSession:
     """Requests of a trace by name, each in a slot of the model's caches and states."""
 
-    def __init__(self, model, max_requests: int):
+    def __init__(self, model, max_requests: int, max_tokens: Optional[int] = None):
         self.model = model
-        model.allocate(max_requests)
+        model.allocate(max_requests, max_tokens)
         self.slot_of = {}
 
     def run(self, entries) -> np.ndarray:
@@ -59,7 +60,7 @@ def main(argv=None) -> int:
     if not hasattr(model, "extend"):
         print("this model family takes whole prompts only", file=sys.stderr)
         return 2
-    session = TraceSession(model, a.max_requests)
+    session = TraceSession(model, a.max_requests, a.max_tokens or None)
     for line in sys.stdin:
         if not line.strip():
             continue

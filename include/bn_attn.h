@@ -56,7 +56,8 @@ extern "C" {
 #define BN_ACT_NONE 0
 #define BN_ACT_SILU 1
 #define BN_ACT_GELU_TANH 2
-#define BN_ACT_LAST 2
+#define BN_ACT_RELU2 3 /* max(z, 0)^2 */
+#define BN_ACT_LAST 3
 
 typedef void* bn_stream_t; /* a cudaStream_t */
 
@@ -474,6 +475,65 @@ BN_API int bn_mamba2_step(const void* proj, int64_t proj_ld, const float* conv_w
 BN_API int bn_gated_group_norm(const void* y, int64_t y_ld, int y_dtype, const void* z, int64_t z_ld, const float* w,
                                void* out, int64_t out_ld, int rows, int width, int groups, float eps, int dtype,
                                bn_stream_t stream);
+
+/* ------------------------------------------------------------------------
+ * c = act(a bt^T + bias), bias (N) fp32 or null, act one of BN_ACT_*; operands and limits as the plain products.
+ * bn_bias_act_f32: the same behind bn_mm_f32, in place.
+ * ------------------------------------------------------------------------ */
+BN_API int bn_gemm_bias_act_bf16_nt(const void* a, const void* bt, const float* bias, void* c, int M, int N, int K, int act,
+                                    int* error_word, bn_stream_t stream);
+BN_API int bn_gemm_bias_act_bf16_nt_small_m(const void* a, const void* bt, const float* bias, void* c, int M, int N, int K,
+                                            int act, void* workspace, size_t workspace_bytes, int* error_word,
+                                            bn_stream_t stream);
+BN_API int bn_gemm_bias_act_bf16_nt_skinny(const void* a, const void* bt, const float* bias, void* out, int M, int N, int K,
+                                           int act, bn_stream_t stream);
+BN_API int bn_bias_act_f32(float* x, int64_t ld, const float* bias, int rows, int cols, int act, bn_stream_t stream);
+
+/* ------------------------------------------------------------------------
+ * A residual stream in several fp32 copies: x (rows, n_in, hidden) -> x' (rows, n_out, hidden),
+ *   x'_t = sum_s mix[s * n_out + t] x_s + w_out[t] * delta * delta_scale   (delta in `dtype`, delta_scale (hidden); optional)
+ *   x_out = x' (optional);  y = RMS norm of sum_t w_in[t] x'_t with weight w, in `dtype` (w null: not wanted)
+ * mix, w_out (n_out) and w_in (n_out) are HOST pointers, read before the call returns; at most 16 streams.
+ * ------------------------------------------------------------------------ */
+BN_API int bn_hyper_norm(const float* x, int n_in, int n_out, const float* mix, const float* w_out, const float* w_in,
+                         const void* delta, int64_t delta_ld, const float* delta_scale, float* x_out, const float* w,
+                         void* y, int64_t y_ld, int dtype, int rows, int hidden, float eps, bn_stream_t stream);
+
+/* ------------------------------------------------------------------------
+ * Grouped-query attention in chunks (fp32 or bf16): query i sees key j if j <= i and both positions lie in the same chunk,
+ * position / chunk.  Rows are B sequences x S new tokens; sequence b occupies slot seq_ids[b] (null: b) and its first new
+ * token has position positions[b].  Head sizes dim_ld and vdim_ld are multiples of 8, zeros behind the values;
+ * rms_dim > 0: queries and keys are divided by sqrt(mean of squares + eps), the mean taken over rms_dim columns.
+ * ring_k[slot][kv_heads][ring_tokens][dim_ld], ring_v likewise with vdim_ld; the token of position p in row p % chunk.  A
+ * token whose row is not below ring_tokens is not kept, and its own result in bn_gqa_step is NaN.
+ * ------------------------------------------------------------------------ */
+/* k, v: the key and value columns of projection rows (ld); values become (1 - lambda) v + lambda v_first where v_first is
+ * given.  Written to row b * rows_per_seq + row_offset + s of k_out / v_out (both may be null) and into the ring */
+BN_API int bn_kv_prep(const void* k, const void* v, int64_t ld, const void* v_first, int64_t v_first_ld, float lambda,
+                      const int32_t* seq_ids, const int32_t* positions, int B, int S, int kv_heads, int dim_ld, int vdim_ld,
+                      int rms_dim, float eps, void* k_out, void* v_out, int rows_per_seq, int row_offset, void* ring_k,
+                      void* ring_v, int ring_tokens, int chunk, int dtype, bn_stream_t stream);
+/* the n_old = positions[b] % chunk tokens of the chunk before positions[b], from the ring to rows b * rows_per_seq + 0 .. */
+BN_API int bn_kv_gather(const void* ring_k, const void* ring_v, int ring_tokens, int chunk, int kv_heads, int dim_ld,
+                        int vdim_ld, const int32_t* seq_ids, const int32_t* positions, int B, int n_old, void* k_out,
+                        void* v_out, int rows_per_seq, int dtype, bn_stream_t stream);
+/* portions: key row b * rows_per_seq + n_old + s belongs to query s of sequence b, key row 0 to the first position of a
+ * chunk.  q (B*S, q_ld) as projected, k (rows, kv_heads * dim) prepared, v (rows, kv_heads * vdim); the result is multiplied
+ * by sigmoid(gate) where gate is given.  error_word (may be null) receives BN_ERR_TIMEOUT if a bounded wait runs out. */
+BN_API int bn_attn_chunked(const void* q, int64_t q_ld, const void* k, int64_t k_ld, const void* v, int64_t v_ld,
+                           const void* gate, int64_t gate_ld, void* out, int64_t out_ld, int B, int S, int n_old,
+                           int rows_per_seq, int H, int kv_heads, int dim, int vdim, int chunk, int rms_dim, float rms_eps,
+                           float scale, int* error_word, int dtype, bn_stream_t stream);
+/* one new token per row: prepares and appends its key and value, attends over the ring, gates; q, k, v and gate are columns
+ * of the same projection rows (ld).  partial holds B * kv_heads * ceil(H / kv_heads / 16) * splits * 16 * (vdim_ld + 2)
+ * floats (splits 1: may be null); tickets B * kv_heads * ceil(H / kv_heads / 16) ints, zero before the first call and left
+ * zero.  splits: bn_gqa_step_splits (a size, 0 for a bad shape), or any number up to 64 */
+BN_API int bn_gqa_step_splits(int B, int H, int kv_heads, int dim_ld, int vdim_ld, int ring_tokens, int dtype);
+BN_API int bn_gqa_step(const void* q, const void* k, const void* v, const void* gate, int64_t ld, const void* v_first,
+                       int64_t v_first_ld, float lambda, void* ring_k, void* ring_v, int num_slots, int ring_tokens,
+                       int chunk, const int32_t* seq_ids, const int32_t* positions, float* partial, int* tickets, int splits,
+                       void* out, int64_t out_ld, int B, int H, int kv_heads, int dim_ld, int vdim_ld, int rms_dim,
+                       float eps, float scale, int* error_word, int dtype, bn_stream_t stream);
 
 #ifdef __cplusplus
 }

@@ -69,7 +69,7 @@ def test_safetensors_round_trip(tmp_path):
 
 def test_registry_names_and_dtypes():
     from baranet_bdml_b200 import build, registry
-    assert set(registry.ARCHITECTURES) == {"LLaMA", "Soluzen"}
+    assert set(registry.ARCHITECTURES) == {"LLaMA", "Soluzen", "Duponex"}
     with pytest.raises(RuntimeError, match="unknown architecture"):
         registry.build_model({"architecture": "nothing"}, None)
     with pytest.raises(registry.UnsupportedDtype):
