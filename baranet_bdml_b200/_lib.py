@@ -96,7 +96,7 @@ SIGNATURES = {
     "bn_kv_prep": (_i, [_p, _p, _i64, _p, _i64, _f, _p, _p, _i, _i, _i, _i, _i, _i, _f, _p, _p, _i, _i, _p, _p, _i, _i, _i, _p]),
     "bn_kv_gather": (_i, [_p, _p, _i, _i, _i, _i, _i, _p, _p, _i, _i, _p, _p, _i, _i, _p]),
     "bn_attn_chunked": (_i, [_p, _i64, _p, _i64, _p, _i64, _p, _i64, _p, _i64, _i, _i, _i, _i, _i, _i, _i, _i, _i, _i, _f, _f,
-                             _p, _i, _p]),
+                             _f, _p, _i, _p]),
     "bn_gqa_step_splits": (_i, [_i, _i, _i, _i, _i, _i, _i]),
     "bn_gqa_step": (_i, [_p, _p, _p, _p, _i64, _p, _i64, _f, _p, _p, _i, _i, _i, _p, _p, _p, _p, _i, _p, _i64, _i, _i, _i, _i, _i,
                          _i, _f, _f, _p, _i, _p]),

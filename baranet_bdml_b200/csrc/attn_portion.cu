@@ -141,7 +141,7 @@ extern "C" int bn_attn_window(const void* q, int64_t q_ld, const void* k, const 
 extern "C" int bn_attn_chunked(const void* q, int64_t q_ld, const void* k, int64_t k_ld, const void* v, int64_t v_ld,
                                const void* gate, int64_t gate_ld, void* out, int64_t out_ld, int B, int S, int n_old,
                                int rows_per_seq, int H, int kv_heads, int dim, int vdim, int chunk, int rms_dim, float rms_eps,
-                               float scale, int* error_word, int dtype, bn_stream_t stream) {
+                               float scale, float score_bound, int* error_word, int dtype, bn_stream_t stream) {
     const char* what = "bn_attn_chunked";
     if (!q || !k || !v || !out) return fail(BN_ERR_INVALID_ARG, "%s: null pointer", what);
     if (B < 0 || S < 0 || n_old < 0 || n_old >= chunk || n_old + S > rows_per_seq || H <= 0 || kv_heads <= 0 || H % kv_heads || dim <= 0 ||
@@ -155,7 +155,8 @@ extern "C" int bn_attn_chunked(const void* q, int64_t q_ld, const void* k, int64
     p.q_ld = q_ld; p.k_ld = k_ld; p.v_ld = v_ld; p.gate_ld = gate_ld; p.out_ld = out_ld;
     p.k_head = dim; p.v_head = vdim; p.k_seq = rows_per_seq * k_ld; p.v_seq = rows_per_seq * v_ld;
     p.B = B; p.S = S; p.n_old = n_old; p.rows_per_seq = rows_per_seq; p.H = H; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim;
-    p.mask = MASK_CHUNK; p.span = chunk; p.rms_dim = rms_dim; p.rms_eps = rms_eps; p.scale = scale; p.error_word = error_word;
+    p.mask = MASK_CHUNK; p.span = chunk; p.rms_dim = rms_dim; p.rms_eps = rms_eps; p.scale = scale; p.score_bound = score_bound;
+    p.error_word = error_word;
     if (dtype == 1 && attn_window_sm100_ok(p)) return attn_window_sm100(p, as_stream(stream));
     return attn_any(p, dtype, as_stream(stream), what);
 }

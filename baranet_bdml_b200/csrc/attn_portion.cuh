@@ -26,6 +26,7 @@ struct AttnPortionParams {
     int B, S, n_old, rows_per_seq, H, kv_heads, dim, rot, vdim, mask, span;
     int rms_dim;                      // > 0: queries are divided by their root mean square, the mean taken over rms_dim columns
     float rms_eps, scale;
+    float score_bound;                // > 0: no scaled score is larger in magnitude
     int* error_word;                  // optional; set when a bounded wait ran out
 };
 

@@ -2,21 +2,23 @@
 // rotated part shared by all heads, values of another width, a sliding window or chunks, and keys that start before the
 // portion's first query (the fast path of bn_attn_window and bn_attn_chunked, bf16).
 //
-// Persistent, one CTA per SM, ten warps.  Work unit = (sequence, head, PAIR of 128-row query tiles); a unit walks the
+// Persistent, one CTA per SM, eleven warps.  Work unit = (sequence, head, PAIR of 128-row query tiles); a unit walks the
 // 64-key tiles from the first key that the pair's first row sees to the last row's own key:
 //   warps 0-3 / 4-7   softmax of query tile 0 / 1: thread = TMEM lane = query row, 64 scores of a step in registers
-//   warp 8            MMA issuer (one elected thread)
+//   warps 8 / 10      MMA issuer of query tile 0 / 1 (one elected thread each)
 //   warp 9            TMA producer
 // Shared memory holds blocks of 64 columns (128-byte swizzled rows): Q of both tiles, and a ring of K and V stages.  A
 // query or key row is ceil(dim / 64) unrotated blocks and ceil(rot / 64) rotated ones; the tensor maps end at dim (keys)
 // and at dim + rot (queries), so what a block holds beyond its part meets zeros on the other side.
-// Tensor memory: scores of tile 0 / 1 at columns [0, 64) / [64, 128), the bf16 weights written over the scores they came
-// from; outputs at [128, 320) / [320, 512), at most 192 value columns.
-// Step (tile u, key tile j): S = Q K^T, softmax with a running maximum that rescales O only when it has grown by 2^8,
-// O += P V.  The issuer's order is  PV(0,j) QK(0,j+1) PV(1,j) QK(1,j+1):  the tensor pipe executes in issue order, so new
-// scores never overtake the read of the weights they replace, and while one tile's softmax runs the other tile's products
-// do.  A commit covers everything issued before it, so the scores' barrier of step j also says that PV of step j - 1 has
-// landed and O may be rescaled.
+// Tensor memory, per query tile 256 columns: 4 - nb_v score buffers of 64 columns (nb_v = 64-column blocks of the values, at
+// most 3), the bf16 weights written over the scores they came from, then the output.
+// Step (tile u, key tile j): S = Q K^T, softmax, O += P V.  An issuer walks the sequence of all key tiles of all units twice,
+// Q K^T running as many key tiles ahead of P V as there are score buffers, across one unit's end too; per key tile its order
+// is P V(j), Q K^T(j + nbuf).  The tensor pipe executes a thread's products in issue order, so new scores never overtake the
+// read of the weights they replace.
+// Softmax: where the caller knows a bound on the scores (unit-RMS queries and keys: dim * scale), weights are exponentials of
+// the scores themselves, without a maximum; otherwise a running maximum that rescales O only when it has grown by 2^8, and
+// then after the P V of the step before has landed.
 // Optional: queries divided by their root mean square - a softmax thread sums its row's squares out of the Q tile and folds
 // the reciprocal into the row's score scale - and outputs multiplied by the sigmoid of a gate on their way out.
 // A key tile that a query tile does not see at all is skipped for that tile.  Masks are applied only by warps that have an
@@ -34,11 +36,11 @@ namespace bn {
 using namespace ptx;
 
 constexpr int WA_BM = 128, WA_BN = 64;
-constexpr int WA_THREADS = 320;
+constexpr int WA_THREADS = 352;
 constexpr int WA_QBLK = WA_BM * 128, WA_KBLK = WA_BN * 128;      // bytes of a 64-column block
 constexpr int WA_MAXSTAGE = 4;
-constexpr uint32_t WA_TMEM_COLS = 512, WA_COL_O = 128, WA_O_STRIDE = 192;
-constexpr int WA_MAXVB = 3;                                      // value blocks of 64 columns
+constexpr uint32_t WA_TMEM_COLS = 512, WA_TILE_COLS = 256;
+constexpr int WA_MAXVB = 3, WA_MAXBUF = 3;                       // value blocks of 64 columns, score buffers
 constexpr int WA_SMEM_LIMIT = 226 * 1024;
 constexpr float WA_LOG2E = 1.4426950408889634f;
 constexpr float WA_RESCALE_THRESHOLD = 8.0f;                     // log2 units
@@ -50,7 +52,7 @@ struct WaParams {
     int* error_word;
     int B, S, n_old, H, rep, dim, rot, vdim, mask, span, rms_dim;
     int nb_dim, nb_rot, nb_v, stages;        // 64-column blocks of the unrotated / rotated key parts and of the values
-    int n_pairs, n_units;
+    int n_pairs, n_units, nbuf;              // nbuf: score buffers in use
     float scale_log2, rms_eps;
 };
 
@@ -87,12 +89,37 @@ __device__ __forceinline__ int wa_unit_index(int round, int n_units) {
     return k < n_units ? k : -1;
 }
 
+// The key tiles of a CTA's units, one after the other
+struct WaCursor {
+    int round, j, n, first, last;            // first, last: of this cursor's query tile
+    bool live;
+    __device__ __forceinline__ void unit(const WaParams& p, int u) {
+        const int k = wa_unit_index(round, p.n_units);
+        live = k >= 0;
+        j = 0;
+        if (!live) return;
+        const WaUnit w = wa_unit(p, k);
+        n = w.n;
+        first = u ? w.first[1] : w.first[0];
+        last = u ? w.last[1] : w.last[0];
+    }
+    __device__ __forceinline__ void start(const WaParams& p, int u) { round = 0; unit(p, u); }
+    __device__ __forceinline__ void next(const WaParams& p, int u) {
+        if (++j < n) return;
+        ++round;
+        unit(p, u);
+    }
+    __device__ __forceinline__ bool active() const { return j >= first && j <= last; }
+};
+
+// NBK, NBV: 64-column blocks of keys and values, 0: any number
+template <bool BOUNDED, int NBK, int NBV>
 __global__ void __launch_bounds__(WA_THREADS, 1)
 attn_window_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                          const __grid_constant__ CUtensorMap tmap_r, const __grid_constant__ CUtensorMap tmap_v,
                          const WaParams p) {
     extern __shared__ uint8_t smem_raw[];
-    __shared__ __align__(8) uint64_t bar_q[2], bar_qfree[2], bar_s[2], bar_p[2], bar_o[2];
+    __shared__ __align__(8) uint64_t bar_q[2], bar_qfree[2], bar_s[2][WA_MAXBUF], bar_p[2][WA_MAXBUF], bar_o[2][WA_MAXBUF];
     __shared__ __align__(8) uint64_t bar_kfull[WA_MAXSTAGE], bar_kempty[WA_MAXSTAGE], bar_vfull[WA_MAXSTAGE], bar_vempty[WA_MAXSTAGE];
     __shared__ uint32_t s_tmem_base;
     __shared__ int s_abort;
@@ -106,15 +133,17 @@ attn_window_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
         for (int u = 0; u < 2; ++u) {
             mbar_init(smem_u32(&bar_q[u]), 1);
             mbar_init(smem_u32(&bar_qfree[u]), p.rms_dim ? 5 : 1);      // the last Q K^T, and the softmax warps that read Q
-            mbar_init(smem_u32(&bar_s[u]), 1);
-            mbar_init(smem_u32(&bar_p[u]), 128);
-            mbar_init(smem_u32(&bar_o[u]), 1);
+            for (int x = 0; x < WA_MAXBUF; ++x) {
+                mbar_init(smem_u32(&bar_s[u][x]), 1);
+                mbar_init(smem_u32(&bar_p[u][x]), 128);
+                mbar_init(smem_u32(&bar_o[u][x]), 1);
+            }
         }
         for (int s = 0; s < WA_MAXSTAGE; ++s) {
             mbar_init(smem_u32(&bar_kfull[s]), 1);
-            mbar_init(smem_u32(&bar_kempty[s]), 1);
+            mbar_init(smem_u32(&bar_kempty[s]), 2);               // both issuers
             mbar_init(smem_u32(&bar_vfull[s]), 1);
-            mbar_init(smem_u32(&bar_vempty[s]), 1);
+            mbar_init(smem_u32(&bar_vempty[s]), 2);
         }
         s_abort = 0;
         fence_mbar_init();
@@ -172,95 +201,129 @@ attn_window_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
                 }
             }
         }
-    } else if (warp == 8) {
-        // ------------------------------------------------------------ MMA issuer
+    } else if (warp >= 8) {
+        // ------------------------------------------------------------ MMA issuers
+        // one thread per query tile (a thread's issue rate, not the tensor pipe, would bound one thread for both); descriptors are
+        // stepped as their low words, block and step counts are compile-time for the common sizes
         constexpr uint32_t IDESC_QK = tc::idesc_bf16(WA_BM, WA_BN, 0), IDESC_PV = tc::idesc_bf16(WA_BM, 64, 1);
-        const uint64_t dZero = tc::smem_desc_sw128(0);               // descriptor = this + (address >> 4)
-        bool ok = true;
-        int kstage = 0, vstage = 0;
-        uint32_t kphase = 0, vphase = 0, nq[2] = {0, 0}, np[2] = {0, 0};
-        for (int round = 0; ok; ++round) {
-            const int k = wa_unit_index(round, p.n_units);
-            if (k < 0) break;
-            const WaUnit w = wa_unit(p, k);
-            for (int j = -1; ok && j < w.n; ++j) {
-                bool k_here = false, v_here = false;
+        constexpr uint32_t DESC_HI = (uint32_t)(tc::smem_desc_sw128(0) >> 32), DESC_LO = (uint32_t)tc::smem_desc_sw128(0);
+        if (elect_one()) {
+            const int u = warp == 8 ? 0 : 1;
+            const int nbv = NBV ? NBV : p.nb_v;
+            const uint32_t tT = tmem + u * WA_TILE_COLS, tO = tT + WA_TILE_COLS - nbv * 64;
+            const uint32_t dq = DESC_LO + (sQ >> 4) + u * nb * (WA_QBLK >> 4), dK = DESC_LO + (sK >> 4), dV = DESC_LO + (sV >> 4);
+            const uint32_t aS = smem_u32(bar_s[u]), aP = smem_u32(bar_p[u]), aO = smem_u32(bar_o[u]), aQ = smem_u32(&bar_q[u]),
+                           aQf = smem_u32(&bar_qfree[u]), aKf = smem_u32(bar_kfull), aKe = smem_u32(bar_kempty), aVf = smem_u32(bar_vfull),
+                           aVe = smem_u32(bar_vempty);
+            bool ok = true;
+            uint32_t kstage = 0, vstage = 0, kphase = 0, vphase = 0, qbuf = 0, pbuf = 0, pphase = 0, nq = 0;
+            WaCursor cq, cp;                                         // Q K^T, P V
+            cq.start(p, u);
+            cp.start(p, u);
+            int ahead = 0;                                           // key tiles with Q K^T issued and P V not
+            while (cq.live || ahead > 0) {
+                // Q K^T stays within one unit of P V: the queries of the unit after that are loaded only when the softmax warps
+                // have read this unit's, which they do after they have put out the unit before
+                const bool qk = cq.live && cq.round <= cp.round + 1, pv = ahead == p.nbuf || !qk;
+                if (pv) {                                            // O += P V
+                    // a tile also waits for key tiles that it does not see: a stage's release counts both tiles, once per filling
+                    ok = mbar_wait(aVf + vstage * 8, vphase, &s_abort);
+                    if (!ok) break;
+                    if (cp.active()) {
+                        ok = mbar_wait(aP + pbuf * 8, pphase, &s_abort);
+                        if (!ok) break;
+                        tc::fence_after_sync();
+                        const uint32_t tP = tT + pbuf * WA_BN, more = cp.j > cp.first;
+                        const uint32_t dv = dV + vstage * nbv * (WA_KBLK >> 4);
+                        if (NBV) {
 #pragma unroll
-                for (int u = 0; u < 2; ++u) {
-                    if (!ok) continue;
-                    const uint32_t tS = tmem + u * WA_BN, tO = tmem + WA_COL_O + u * WA_O_STRIDE;
-                    if (j >= w.first[u] && j <= w.last[u]) {          // O += P V of key tile j
-                        ok = mbar_wait(smem_u32(&bar_p[u]), np[u] & 1u, &s_abort);
-                        ++np[u];
-                        if (ok && !v_here) {
-                            ok = mbar_wait(smem_u32(&bar_vfull[vstage]), vphase, &s_abort);
-                            v_here = true;
-                        }
-                        if (!ok) continue;
-                        if (elect_one()) {
-                            tc::fence_after_sync();
-                            for (int x = 0; x < p.nb_v; ++x) {
-                                const uint32_t v = sV + (vstage * p.nb_v + x) * WA_KBLK;
+                            for (int x = 0; x < NBV; ++x)
 #pragma unroll
                                 for (int kk = 0; kk < WA_BN / 16; ++kk)
-                                    tc::mma_ts(tO + x * 64, tS + kk * 8, dZero + (uint64_t)((v >> 4) + kk * 128), IDESC_PV,
-                                               j > w.first[u] || kk > 0);
-                            }
-                            if (j == w.last[u]) tc::commit(smem_u32(&bar_o[u]));
+                                    tc::mma_ts_lohi(tO + x * 64, tP + kk * 8, dv + x * (WA_KBLK >> 4) + kk * 128, DESC_HI, IDESC_PV,
+                                                    kk > 0 ? 1u : more);
+                        } else {
+                            for (int x = 0; x < nbv; ++x)
+#pragma unroll
+                                for (int kk = 0; kk < WA_BN / 16; ++kk)
+                                    tc::mma_ts_lohi(tO + x * 64, tP + kk * 8, dv + x * (WA_KBLK >> 4) + kk * 128, DESC_HI, IDESC_PV,
+                                                    kk > 0 ? 1u : more);
                         }
-                        __syncwarp();
+                        if (BOUNDED) {
+                            if (cp.j == cp.last) tc::commit(aO);
+                        } else {
+                            tc::commit(aO + pbuf * 8);
+                        }
+                        if (++pbuf == p.nbuf) { pbuf = 0; pphase ^= 1u; }
                     }
-                    if (j + 1 >= w.first[u] && j + 1 <= w.last[u]) {  // S = Q K^T of key tile j + 1
-                        if (j + 1 == w.first[u]) {
-                            ok = mbar_wait(smem_u32(&bar_q[u]), nq[u] & 1u, &s_abort);
-                            ++nq[u];
+                    tc::commit(aVe + vstage * 8);
+                    if (++vstage == p.stages) { vstage = 0; vphase ^= 1u; }
+                    cp.next(p, u);
+                }
+                if (qk) {                                            // S = Q K^T
+                    ok = mbar_wait(aKf + kstage * 8, kphase, &s_abort);
+                    if (!ok) break;
+                    if (cq.active()) {
+                        if (cq.j == cq.first) {
+                            ok = mbar_wait(aQ, nq & 1u, &s_abort);
+                            ++nq;
+                            if (!ok) break;
                         }
-                        if (ok && !k_here) {
-                            ok = mbar_wait(smem_u32(&bar_kfull[kstage]), kphase, &s_abort);
-                            k_here = true;
-                        }
-                        if (!ok) continue;
-                        if (elect_one()) {
-                            tc::fence_after_sync();
-                            bool more = false;
+                        tc::fence_after_sync();
+                        const uint32_t tS = tT + qbuf * WA_BN, dk = dK + kstage * nb * (WA_KBLK >> 4);
+                        if (NBK) {
+                            // what a block holds beyond its part is zero, or meets zeros: every block takes four steps
+#pragma unroll
+                            for (int x = 0; x < NBK; ++x)
+#pragma unroll
+                                for (int kk = 0; kk < 4; ++kk)
+                                    tc::mma_ss_lohi(tS, dq + x * (WA_QBLK >> 4) + kk * 2, dk + x * (WA_KBLK >> 4) + kk * 2, DESC_HI, IDESC_QK,
+                                                    x > 0 || kk > 0);
+                        } else {
+                            uint32_t more = 0;
                             for (int x = 0; x < nb; ++x) {
                                 const int cols = x < p.nb_dim ? p.dim - x * 64 : p.rot - (x - p.nb_dim) * 64;
                                 const int steps = cols >= 64 ? 4 : (cols + 15) / 16;
-                                const uint32_t qa = sQ + (u * nb + x) * WA_QBLK, ka = sK + (kstage * nb + x) * WA_KBLK;
                                 for (int kk = 0; kk < steps; ++kk) {
-                                    tc::mma_ss(tS, dZero + (uint64_t)((qa >> 4) + kk * 2), dZero + (uint64_t)((ka >> 4) + kk * 2),
-                                               IDESC_QK, more);
-                                    more = true;
+                                    tc::mma_ss_lohi(tS, dq + x * (WA_QBLK >> 4) + kk * 2, dk + x * (WA_KBLK >> 4) + kk * 2, DESC_HI, IDESC_QK,
+                                                    more);
+                                    more = 1;
                                 }
                             }
-                            tc::commit(smem_u32(&bar_s[u]));
-                            if (j + 1 == w.last[u]) tc::commit(smem_u32(&bar_qfree[u]));
                         }
-                        __syncwarp();
+                        tc::commit(aS + qbuf * 8);
+                        if (cq.j == cq.last) tc::commit(aQf);
+                        if (++qbuf == p.nbuf) qbuf = 0;
                     }
+                    tc::commit(aKe + kstage * 8);
+                    if (++kstage == p.stages) { kstage = 0; kphase ^= 1u; }
+                    cq.next(p, u);
                 }
-                if (!ok) break;
-                if (elect_one()) {
-                    if (j >= 0) tc::commit(smem_u32(&bar_vempty[vstage]));
-                    if (j + 1 < w.n) tc::commit(smem_u32(&bar_kempty[kstage]));
-                }
-                __syncwarp();
-                if (j >= 0 && ++vstage == p.stages) { vstage = 0; vphase ^= 1u; }
-                if (j + 1 < w.n && ++kstage == p.stages) { kstage = 0; kphase ^= 1u; }
+                ahead += (int)qk - (int)pv;
             }
         }
+        __syncwarp();
     } else {
         // ---------------------------------------------------------- softmax warps
         const int u = warp / 4;
         const uint32_t lane_base = ((uint32_t)((warp % 4) * 32)) << 16;
-        const uint32_t tS = tmem + lane_base + u * WA_BN, tO = tmem + lane_base + WA_COL_O + u * WA_O_STRIDE;
+        const uint32_t tT = tmem + lane_base + u * WA_TILE_COLS, tO = tT + WA_TILE_COLS - p.nb_v * 64;
         bool ok = true;
-        uint32_t ns = 0, no = 0, nq = 0;                             // steps and tiles of this query tile so far
+        int buf = 0;
+        uint32_t phase = 0, nu = 0, nq = 0;                          // nu: units so far
+        // the latest P V that this query tile has handed its weights to: an output barrier per score buffer where every step
+        // may have to wait for one (two phases of a barrier are then never outstanding), else one per unit
+        auto wait_pv = [&]() {
+            if (BOUNDED) return mbar_wait(smem_u32(&bar_o[u][0]), nu & 1u, &s_abort);
+            return buf == 0 ? mbar_wait(smem_u32(&bar_o[u][p.nbuf - 1]), phase ^ 1u, &s_abort)
+                            : mbar_wait(smem_u32(&bar_o[u][buf - 1]), phase, &s_abort);
+        };
         for (int round = 0; ok; ++round) {
             const int k = wa_unit_index(round, p.n_units);
             if (k < 0) break;
             const WaUnit w = wa_unit(p, k);
-            if (w.last[u] < w.first[u]) continue;
+            const int first = u ? w.first[1] : w.first[0], last = u ? w.last[1] : w.last[0];
+            if (last < first) continue;
             const int row0 = w.i0 + u * WA_BM + (warp % 4) * 32;     // the warp's first row
             const int gi = row0 + lane;
             const int own = p.n_old + gi, oldest = mask_oldest(p.mask, p.span, own);         // the keys this row sees
@@ -286,11 +349,13 @@ attn_window_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
                 __syncwarp();
                 if (lane == 0) mbar_arrive(smem_u32(&bar_qfree[u]));
             }
-            float m_ref = -INFINITY, l_run = 0.f;
-            for (int j = w.first[u]; j <= w.last[u]; ++j, ++ns) {
-                ok = mbar_wait(smem_u32(&bar_s[u]), ns & 1u, &s_abort);
+            float m_ref = -INFINITY;
+            float l0 = 0.f, l1 = 0.f, l2 = 0.f, l3 = 0.f;
+            for (int j = first; j <= last; ++j) {
+                ok = mbar_wait(smem_u32(&bar_s[u][buf]), phase, &s_abort);
                 if (!ok) break;
                 tc::fence_after_sync();
+                const uint32_t tS = tT + buf * WA_BN;
                 const int key = w.key0 + j * WA_BN;
                 const bool masked = key + WA_BN - 1 > warp_own0 || key < warp_oldest1;
                 uint32_t r[2][32];
@@ -307,89 +372,120 @@ attn_window_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const __gri
                             if (kk > own || kk < oldest) r[c][i] = 0xff800000u;          // -inf
                         }
                 }
-                float t0 = -INFINITY, t1 = -INFINITY, t2 = -INFINITY, t3 = -INFINITY;
-#pragma unroll
-                for (int i = 0; i < 32; i += 2) {
-                    t0 = fmaxf(t0, __uint_as_float(r[0][i]));
-                    t1 = fmaxf(t1, __uint_as_float(r[0][i + 1]));
-                    t2 = fmaxf(t2, __uint_as_float(r[1][i]));
-                    t3 = fmaxf(t3, __uint_as_float(r[1][i + 1]));
-                }
-                const float m_new = fmaxf(m_ref, fmaxf(fmaxf(t0, t1), fmaxf(t2, t3)));
-                const bool grow = (m_new - m_ref) * scale_log2 > WA_RESCALE_THRESHOLD;   // NaN (both -inf) is false
-                if (__any_sync(0xffffffffu, grow)) {
-                    if (j > w.first[u]) {
-                        const float alpha = m_ref == -INFINITY ? 0.f : ex2((m_ref - m_new) * scale_log2);
-                        l_run *= alpha;
-                        for (int c = 0; c < 2 * p.nb_v; ++c) {
-                            uint32_t o[32];
-                            tc::ld32(tO + c * 32, o);
-                            tc::wait_ld(o);
-#pragma unroll
-                            for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * alpha);
-                            tc::st32(tO + c * 32, o);
-                        }
-                    }
-                    m_ref = m_new;
-                }
-                // a row that has seen no key yet has only -inf scores: any finite reference gives zero weights
-                const float mneg = m_ref == -INFINITY ? 0.f : -m_ref * scale_log2;
-                float l0 = 0.f, l1 = 0.f;
-#pragma unroll
-                for (int c = 0; c < 2; ++c) {
-                    uint32_t pk[16];
+                float mneg = 0.f;
+                if (!BOUNDED) {
+                    float t0 = -INFINITY, t1 = -INFINITY, t2 = -INFINITY, t3 = -INFINITY;
 #pragma unroll
                     for (int i = 0; i < 32; i += 2) {
-                        const float p0 = ex2(fmaf(__uint_as_float(r[c][i]), scale_log2, mneg));
-                        const float p1 = ex2(fmaf(__uint_as_float(r[c][i + 1]), scale_log2, mneg));
-                        l0 += p0;
-                        l1 += p1;
-                        pk[i / 2] = pack_bf16(p0, p1);
+                        t0 = fmaxf(t0, __uint_as_float(r[0][i]));
+                        t1 = fmaxf(t1, __uint_as_float(r[0][i + 1]));
+                        t2 = fmaxf(t2, __uint_as_float(r[1][i]));
+                        t3 = fmaxf(t3, __uint_as_float(r[1][i + 1]));
                     }
-                    tc::st16(tS + c * 16, pk);
+                    const float m_new = fmaxf(m_ref, fmaxf(fmaxf(t0, t1), fmaxf(t2, t3)));
+                    const bool grow = (m_new - m_ref) * scale_log2 > WA_RESCALE_THRESHOLD;   // NaN (both -inf) is false
+                    if (__any_sync(0xffffffffu, grow)) {
+                        if (j > first) {
+                            ok = wait_pv();                          // of the step before
+                            if (!ok) break;
+                            tc::fence_after_sync();
+                            const float alpha = m_ref == -INFINITY ? 0.f : ex2((m_ref - m_new) * scale_log2);
+                            l0 *= alpha; l1 *= alpha; l2 *= alpha; l3 *= alpha;
+#pragma unroll 1
+                            for (int c = 0; c < 4 * p.nb_v; ++c) {
+                                uint32_t o[16];
+                                tc::ld16(tO + c * 16, o);
+                                tc::wait_ld(o);
+#pragma unroll
+                                for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * alpha);
+                                tc::st16(tO + c * 16, o);
+                            }
+                        }
+                        m_ref = m_new;
+                    }
+                    // a row that has seen no key yet has only -inf scores: any finite reference gives zero weights
+                    mneg = m_ref == -INFINITY ? 0.f : -m_ref * scale_log2;
                 }
-                l_run += l0 + l1;
+                if (BOUNDED) {
+                    const uint64_t sc2 = pack_f32x2(scale_log2, scale_log2), zero2 = pack_f32x2(0.f, 0.f);
+                    uint64_t la = pack_f32x2(l0, l1), lb = pack_f32x2(l2, l3);
+#pragma unroll
+                    for (int c = 0; c < 2; ++c) {
+                        uint32_t pk[16];
+#pragma unroll
+                        for (int i = 0; i < 32; i += 2) {
+                            float p0, p1;
+                            unpack_f32x2(fma_f32x2(pack_f32x2(__uint_as_float(r[c][i]), __uint_as_float(r[c][i + 1])), sc2, zero2), p0, p1);
+                            p0 = ex2(p0);
+                            p1 = ex2(p1);
+                            if (i & 2) lb = add_f32x2(lb, pack_f32x2(p0, p1));
+                            else la = add_f32x2(la, pack_f32x2(p0, p1));
+                            pk[i / 2] = pack_bf16(p0, p1);
+                        }
+                        tc::st16(tS + c * 16, pk);
+                    }
+                    unpack_f32x2(la, l0, l1);
+                    unpack_f32x2(lb, l2, l3);
+                } else {
+#pragma unroll
+                    for (int c = 0; c < 2; ++c) {
+                        uint32_t pk[16];
+#pragma unroll
+                        for (int i = 0; i < 32; i += 2) {
+                            const float p0 = ex2(fmaf(__uint_as_float(r[c][i]), scale_log2, mneg));
+                            const float p1 = ex2(fmaf(__uint_as_float(r[c][i + 1]), scale_log2, mneg));
+                            l0 += p0;
+                            l1 += p1;
+                            pk[i / 2] = pack_bf16(p0, p1);
+                        }
+                        tc::st16(tS + c * 16, pk);
+                    }
+                }
                 tc::wait_st();
                 tc::fence_before_sync();
-                mbar_arrive(smem_u32(&bar_p[u]));
+                mbar_arrive(smem_u32(&bar_p[u][buf]));
+                if (++buf == p.nbuf) { buf = 0; phase ^= 1u; }
             }
             if (!ok) break;
-            // O / l -> bf16 -> global
-            ok = mbar_wait(smem_u32(&bar_o[u]), no & 1u, &s_abort);
-            ++no;
+            // O / l, gated -> bf16 -> global
+            const float l_run = (l0 + l1) + (l2 + l3);
+            const __nv_bfloat16* gate = p.gate && gi < p.S ? p.gate + ((int64_t)w.b * p.S + gi) * p.gate_ld + w.h * p.vdim : nullptr;
+            uint4 g4[4];
+            auto load_gate = [&](int c) {                            // of 32 columns, requested before they are needed
+#pragma unroll
+                for (int v = 0; v < 4; ++v)
+                    if (gate && c * 32 + v * 8 < p.vdim) g4[v] = *reinterpret_cast<const uint4*>(gate + c * 32 + v * 8);
+            };
+            load_gate(0);
+            ok = wait_pv();
+            ++nu;
             if (!ok) break;
             tc::fence_after_sync();
             const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
             __nv_bfloat16* dst = p.out + ((int64_t)w.b * p.S + gi) * p.out_ld + w.h * p.vdim;
-            const __nv_bfloat16* gate = p.gate ? p.gate + ((int64_t)w.b * p.S + gi) * p.gate_ld + w.h * p.vdim : nullptr;
             for (int c = 0; c < 2 * p.nb_v; ++c) {
                 uint32_t o[32];
                 tc::ld32(tO + c * 32, o);
                 tc::wait_ld(o);
                 if (gi < p.S) {
-                    if (gate) {
-#pragma unroll
-                        for (int v = 0; v < 4; ++v)
-                            if (c * 32 + v * 8 < p.vdim) {
-                                const uint4 g4 = *reinterpret_cast<const uint4*>(gate + c * 32 + v * 8);
-                                const uint32_t* gw = reinterpret_cast<const uint32_t*>(&g4);
-#pragma unroll
-                                for (int e = 0; e < 4; ++e) {
-                                    o[v * 8 + 2 * e] = __float_as_uint(__uint_as_float(o[v * 8 + 2 * e]) * sigmoid_fast(bf16_lo(gw[e])));
-                                    o[v * 8 + 2 * e + 1] = __float_as_uint(__uint_as_float(o[v * 8 + 2 * e + 1]) * sigmoid_fast(bf16_hi(gw[e])));
-                                }
-                            }
-                    }
 #pragma unroll
                     for (int v = 0; v < 4; ++v)
                         if (c * 32 + v * 8 < p.vdim) {                 // vdim is a multiple of 8
-                            uint4 o4;
-                            o4.x = pack_bf16(__uint_as_float(o[v * 8 + 0]) * inv, __uint_as_float(o[v * 8 + 1]) * inv);
-                            o4.y = pack_bf16(__uint_as_float(o[v * 8 + 2]) * inv, __uint_as_float(o[v * 8 + 3]) * inv);
-                            o4.z = pack_bf16(__uint_as_float(o[v * 8 + 4]) * inv, __uint_as_float(o[v * 8 + 5]) * inv);
-                            o4.w = pack_bf16(__uint_as_float(o[v * 8 + 6]) * inv, __uint_as_float(o[v * 8 + 7]) * inv);
-                            *reinterpret_cast<uint4*>(dst + c * 32 + v * 8) = o4;
+                            float f[8];
+#pragma unroll
+                            for (int e = 0; e < 8; ++e) f[e] = __uint_as_float(o[v * 8 + e]) * inv;
+                            if (gate) {
+                                const uint32_t gw[4] = {g4[v].x, g4[v].y, g4[v].z, g4[v].w};
+#pragma unroll
+                                for (int e = 0; e < 4; ++e) {
+                                    f[2 * e] *= sigmoid_fast(bf16_lo(gw[e]));
+                                    f[2 * e + 1] *= sigmoid_fast(bf16_hi(gw[e]));
+                                }
+                            }
+                            *reinterpret_cast<uint4*>(dst + c * 32 + v * 8) =
+                                make_uint4(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]), pack_bf16(f[4], f[5]), pack_bf16(f[6], f[7]));
                         }
+                    load_gate(c + 1);
                 }
             }
             // the next unit's first PV overwrites O: it waits for this warp's next arrival on bar_p, which follows
@@ -430,6 +526,20 @@ static int wa_map(CUtensorMap* m, const void* base, int inner, int heads, int64_
     return make_tensor_map(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, base, dims, strides, box, CU_TENSOR_MAP_SWIZZLE_128B);
 }
 
+template <bool BOUNDED, int NBK, int NBV>
+static int wa_launch(unsigned grid, size_t smem, cudaStream_t st, const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mr,
+                     const CUtensorMap& mv, const WaParams& p, int dev, const char* what) {
+    static thread_local int configured_dev = -1;
+    if (configured_dev != dev) {
+        cudaError_t e = cudaFuncSetAttribute(attn_window_sm100_kernel<BOUNDED, NBK, NBV>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                             WA_SMEM_LIMIT);
+        if (e != cudaSuccess) return fail(BN_ERR_CUDA, "%s: %s", what, cudaGetErrorString(e));
+        configured_dev = dev;
+    }
+    attn_window_sm100_kernel<BOUNDED, NBK, NBV><<<grid, WA_THREADS, smem, st>>>(mq, mk, mr, mv, p);
+    return launch_status(what);
+}
+
 int attn_window_sm100(const AttnPortionParams& a, cudaStream_t st) {
     const char* what = "portion attention";
     CUtensorMap mq, mk, mr, mv;
@@ -455,21 +565,24 @@ int attn_window_sm100(const AttnPortionParams& a, cudaStream_t st) {
     const long long units = (long long)a.B * a.H * p.n_pairs;
     if (units > (1 << 30)) return fail(BN_ERR_UNSUPPORTED, "%s: too many query tiles", what);
     p.n_units = (int)units;
+    p.nbuf = 4 - p.nb_v < p.stages ? 4 - p.nb_v : p.stages;
     p.scale_log2 = a.scale * WA_LOG2E;
+    // the weights of a row are at most 2^60 and at least 2^-60, their sums far from either end of fp32
+    const bool bounded = a.score_bound > 0.f && a.score_bound * WA_LOG2E <= 60.f;
     const int nb = p.nb_dim + p.nb_rot;
     const size_t smem = 1024 + (size_t)2 * nb * WA_QBLK + (size_t)p.stages * (nb + p.nb_v) * WA_KBLK;
     int dev = 0, sms = 0;
     cudaGetDevice(&dev);
     cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev);
-    static thread_local int configured_dev = -1;
-    if (configured_dev != dev) {
-        cudaError_t e = cudaFuncSetAttribute(attn_window_sm100_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, WA_SMEM_LIMIT);
-        if (e != cudaSuccess) return fail(BN_ERR_CUDA, "%s: %s", what, cudaGetErrorString(e));
-        configured_dev = dev;
-    }
     const unsigned grid = (unsigned)(p.n_units < sms ? p.n_units : sms);
-    attn_window_sm100_kernel<<<grid, WA_THREADS, smem, st>>>(mq, mk, mr, mv, p);
-    return launch_status(what);
+    const int sizes = nb * 4 + p.nb_v;
+    if (bounded && sizes == 1 * 4 + 1) return wa_launch<true, 1, 1>(grid, smem, st, mq, mk, mr, mv, p, dev, what);
+    if (bounded && sizes == 2 * 4 + 2) return wa_launch<true, 2, 2>(grid, smem, st, mq, mk, mr, mv, p, dev, what);
+    if (bounded) return wa_launch<true, 0, 0>(grid, smem, st, mq, mk, mr, mv, p, dev, what);
+    if (sizes == 1 * 4 + 1) return wa_launch<false, 1, 1>(grid, smem, st, mq, mk, mr, mv, p, dev, what);
+    if (sizes == 2 * 4 + 2) return wa_launch<false, 2, 2>(grid, smem, st, mq, mk, mr, mv, p, dev, what);
+    if (sizes == 3 * 4 + 2) return wa_launch<false, 3, 2>(grid, smem, st, mq, mk, mr, mv, p, dev, what);
+    return wa_launch<false, 0, 0>(grid, smem, st, mq, mk, mr, mv, p, dev, what);
 }
 
 }  // namespace bn

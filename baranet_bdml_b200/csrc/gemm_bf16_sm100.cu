@@ -85,6 +85,7 @@ gemm_bf16_nt_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
     __shared__ __align__(8) uint64_t bar_full[GM_NSTAGE], bar_empty[GM_NSTAGE], bar_acc_full[2], bar_acc_empty[2];
     __shared__ uint32_t s_tmem_base;
     __shared__ int s_abort;
+    __shared__ __align__(16) float s_bias[EPI == EPI_BIAS ? 4 : 1][EPI == EPI_BIAS ? GM_BN : 4];      // a copy per epilogue warp
 
     const int tid = threadIdx.x, warp = tid / 32, lane = tid % 32;
     const uint32_t smem0 = (smem_u32(smem_raw) + 1023u) & ~1023u;
@@ -186,6 +187,11 @@ gemm_bf16_nt_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
         for (int t = blockIdx.x; ok && t < n_tiles; t += gridDim.x, ++local) {
             const uint32_t acc = local & 1u;
             const int m0 = (t % tiles_m) * GM_BM, n0 = ((t / tiles_m) % tiles_n) * GM_BN;
+            if (EPI == EPI_BIAS) {                // the tile's bias, fetched while its products run
+                __syncwarp();
+                for (int c = lane; c < GM_BN; c += 32) s_bias[warp][c] = p.bias && n0 + c < p.n_out ? __ldg(p.bias + n0 + c) : 0.f;
+                __syncwarp();
+            }
             ok = mbar_wait(smem_u32(&bar_acc_full[acc]), (local >> 1) & 1u, &s_abort);
             if (!ok) break;
             tc::fence_after_sync();
@@ -224,8 +230,9 @@ gemm_bf16_nt_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_con
                         for (int v = 0; v < 4; ++v) {
                             const int col = n0 + c * 32 + v * 8;
                             if (col < p.n_out) {
-                                float h[8], b4[4] = {0.f, 0.f, 0.f, 0.f}, b8[4] = {0.f, 0.f, 0.f, 0.f};
-                                if (p.bias) { load4(p.bias + col, b4); load4(p.bias + col + 4, b8); }
+                                float h[8], b4[4], b8[4];
+                                load4(&s_bias[warp][c * 32 + v * 8], b4);
+                                load4(&s_bias[warp][c * 32 + v * 8 + 4], b8);
 #pragma unroll
                                 for (int e = 0; e < 4; ++e) {
                                     h[e] = activation_fast(p.act, __uint_as_float(r[v * 8 + e]) + b4[e]);

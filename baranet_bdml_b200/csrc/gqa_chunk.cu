@@ -43,88 +43,140 @@ struct KvPrepParams {
     float lambda, eps;
 };
 
-constexpr int KP_WARPS = 8;
+constexpr int KP_THREADS = 256;
 
-template <typename T>
-__global__ void __launch_bounds__(KP_WARPS * 32)
+// 8 values, one 16-byte piece in bf16 and two in fp32
+__device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
+    load4(p, *reinterpret_cast<float(*)[4]>(v));
+    load4(p + 4, *reinterpret_cast<float(*)[4]>(v + 4));
+}
+__device__ __forceinline__ void store8(float* p, const float (&v)[8]) {
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
+}
+__device__ __forceinline__ void unpack8(const uint4& u, float (&f)[8]) {
+    f[0] = bf16_lo(u.x); f[1] = bf16_hi(u.x); f[2] = bf16_lo(u.y); f[3] = bf16_hi(u.y);
+    f[4] = bf16_lo(u.z); f[5] = bf16_hi(u.z); f[6] = bf16_lo(u.w); f[7] = bf16_hi(u.w);
+}
+__device__ __forceinline__ uint4 pack8(const float (&f)[8]) {
+    return make_uint4(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]), pack_bf16(f[4], f[5]), pack_bf16(f[6], f[7]));
+}
+__device__ __forceinline__ void load8(const __nv_bfloat16* p, float (&v)[8]) { unpack8(*reinterpret_cast<const uint4*>(p), v); }
+__device__ __forceinline__ void store8(__nv_bfloat16* p, const float (&v)[8]) { *reinterpret_cast<uint4*>(p) = pack8(v); }
+
+// LANES lanes (a power of two) for each (token, key head); a lane's first pieces of key, value and first value are requested
+// together, heads wider than 8 LANES go round
+template <typename T, int LANES>
+__global__ void __launch_bounds__(KP_THREADS)
 kv_prep_kernel(const KvPrepParams p) {
     grid_dependency_wait();
     grid_launch_dependents();
-    const int lane = threadIdx.x % 32;
-    const long long n = (long long)p.B * p.S * p.G;
-    for (long long item = (long long)blockIdx.x * KP_WARPS + threadIdx.x / 32; item < n; item += (long long)gridDim.x * KP_WARPS) {
-        const int g = (int)(item % p.G);
-        const long long r = item / p.G;
-        const int b = (int)(r / p.S), s = (int)(r - (long long)b * p.S);
-        const int pos = p.positions[b] + s, last = p.positions[b] + p.S - 1, slot = p.seq_ids ? p.seq_ids[b] : b;
+    constexpr int PER_BLOCK = KP_THREADS / LANES;
+    const int lane = threadIdx.x % LANES;
+    const unsigned n = (unsigned)p.B * p.S * p.G;
+    for (unsigned at = blockIdx.x * PER_BLOCK; at < n; at += gridDim.x * PER_BLOCK) {
+        const unsigned item = at + threadIdx.x / LANES;
+        const bool here = item < n;                       // the whole warp takes part in the sums
+        const int g = here ? (int)(item % p.G) : 0, r = here ? (int)(item / p.G) : 0;
+        const int b = r / p.S, s = r - b * p.S;
         const T* k = static_cast<const T*>(p.k) + r * p.ld + g * p.dim_ld;
         const T* v = static_cast<const T*>(p.v) + r * p.ld + g * p.vdim_ld;
+        const T* vf = p.v_first ? static_cast<const T*>(p.v_first) + r * p.v_first_ld + g * p.vdim_ld : nullptr;
+        float k8[8] = {}, v8[8] = {}, f8[8] = {};
+        const int c0 = lane * 8;
+        if (here && c0 < p.dim_ld) load8(k + c0, k8);
+        if (here && c0 < p.vdim_ld) {
+            load8(v + c0, v8);
+            if (vf) load8(vf + c0, f8);
+        }
+        const int start = p.positions[b], pos = start + s, last = start + p.S - 1, slot = p.seq_ids ? p.seq_ids[b] : b;
         const int64_t out_row = (int64_t)b * p.rows_per_seq + p.row_offset + s;
         T* ko = p.k_out ? static_cast<T*>(p.k_out) + (out_row * p.G + g) * p.dim_ld : nullptr;
         T* vo = p.v_out ? static_cast<T*>(p.v_out) + (out_row * p.G + g) * p.vdim_ld : nullptr;
         // only the chunk that the portion ends in is kept, so no cache row is written twice
-        const int row = pos % p.chunk;
-        const bool keep = row < p.ring_tokens && pos / p.chunk == last / p.chunk;
+        const int row = pos % p.chunk, first_kept = last - last % p.chunk;
+        const bool keep = row < p.ring_tokens && pos >= first_kept;
         const int64_t ring_row = ((int64_t)slot * p.G + g) * p.ring_tokens + row;
         T* kr = keep ? static_cast<T*>(p.ring_k) + ring_row * p.dim_ld : nullptr;
         T* vr = keep ? static_cast<T*>(p.ring_v) + ring_row * p.vdim_ld : nullptr;
         float inv = 1.f;
         if (p.rms_dim) {
             float ss = 0.f;
-            for (int i = lane * 4; i < p.dim_ld; i += 128) {
-                float x[4];
-                load4(k + i, x);
 #pragma unroll
-                for (int e = 0; e < 4; ++e) ss = fmaf(x[e], x[e], ss);
+            for (int e = 0; e < 8; ++e) ss = fmaf(k8[e], k8[e], ss);
+            for (int c = c0 + 8 * LANES; here && c < p.dim_ld; c += 8 * LANES) {
+                float x[8];
+                load8(k + c, x);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) ss = fmaf(x[e], x[e], ss);
             }
 #pragma unroll
-            for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+            for (int o = LANES / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
             inv = rsqrtf(ss / (float)p.rms_dim + p.eps);
         }
-        for (int i = lane * 4; i < p.dim_ld; i += 128) {
-            float x[4];
-            load4(k + i, x);
+        if (!here) continue;
+        for (int c = c0; c < p.dim_ld; c += 8 * LANES) {
+            if (c > c0) load8(k + c, k8);
 #pragma unroll
-            for (int e = 0; e < 4; ++e) x[e] *= inv;
-            if (ko) store4(ko + i, x);
-            if (kr) store4(kr + i, x);
+            for (int e = 0; e < 8; ++e) k8[e] *= inv;
+            if (ko) store8(ko + c, k8);
+            if (kr) store8(kr + c, k8);
         }
-        const T* vf = p.v_first ? static_cast<const T*>(p.v_first) + r * p.v_first_ld + g * p.vdim_ld : nullptr;
-        for (int i = lane * 4; i < p.vdim_ld; i += 128) {
-            float x[4];
-            load4(v + i, x);
-            if (vf) {
-                float f[4];
-                load4(vf + i, f);
-#pragma unroll
-                for (int e = 0; e < 4; ++e) x[e] = fmaf(p.lambda, f[e], (1.f - p.lambda) * x[e]);
+        for (int c = c0; c < p.vdim_ld; c += 8 * LANES) {
+            if (c > c0) {
+                load8(v + c, v8);
+                if (vf) load8(vf + c, f8);
             }
-            if (vo) store4(vo + i, x);
-            if (vr) store4(vr + i, x);
+            if (vf) {
+#pragma unroll
+                for (int e = 0; e < 8; ++e) v8[e] = fmaf(p.lambda, f8[e], (1.f - p.lambda) * v8[e]);
+            }
+            if (vo) store8(vo + c, v8);
+            if (vr) store8(vr + c, v8);
         }
     }
 }
 
+template <typename T>
+static void kv_prep_launch(const KvPrepParams& p, cudaStream_t st) {
+    const int widest = p.dim_ld > p.vdim_ld ? p.dim_ld : p.vdim_ld;
+    const int lanes = widest <= 64 ? 8 : widest <= 128 ? 16 : 32;
+    const long long per = KP_THREADS / lanes, blocks = ((long long)p.B * p.S * p.G + per - 1) / per, cap = (long long)sm_count() * 16;
+    const unsigned grid = (unsigned)(blocks < cap ? blocks : cap);
+    if (lanes == 8) launch_dependent(kv_prep_kernel<T, 8>, grid, KP_THREADS, 0, st, p);
+    else if (lanes == 16) launch_dependent(kv_prep_kernel<T, 16>, grid, KP_THREADS, 0, st, p);
+    else launch_dependent(kv_prep_kernel<T, 32>, grid, KP_THREADS, 0, st, p);
+}
+
 // the n_old tokens of the chunk before positions[b], out of the cache, to rows 0 .. n_old - 1 of each sequence's block of
-// rows; rows are moved in 16-byte pieces
-__global__ void __launch_bounds__(128)
+// rows; a thread moves GA_BATCH 16-byte pieces, all requested before the first is stored.  Block (pieces, key head, sequence)
+constexpr int GA_THREADS = 256, GA_BATCH = 4;
+
+__global__ void __launch_bounds__(GA_THREADS)
 kv_gather_kernel(const uint4* ring_k, const uint4* ring_v, int ring_tokens, int G, int k16, int v16, const int32_t* seq_ids,
-                 const int32_t* positions, int chunk, int B, int n_old, uint4* k_out, uint4* v_out, int rows_per_seq) {
+                 const int32_t* positions, int chunk, int n_old, uint4* k_out, uint4* v_out, int rows_per_seq, int blocks) {
     grid_dependency_wait();
     grid_launch_dependents();
-    const long long n = (long long)B * n_old * G;
-    const int per = k16 + v16, lanes = 128 / per > 0 ? per : 128;           // several (token, head) pairs per block where they fit
-    const int sub = threadIdx.x / lanes, subs = 128 / lanes;
-    if (sub >= subs) return;
-    for (long long item = (long long)blockIdx.x * subs + sub; item < n; item += (long long)gridDim.x * subs) {
-        const int g = (int)(item % G), i = (int)(item / G % n_old), b = (int)(item / ((long long)G * n_old));
-        const int slot = seq_ids ? seq_ids[b] : b;
-        if (i >= positions[b] % chunk || i >= ring_tokens) continue;        // the host sized n_old by the same positions
-        const int64_t src = ((int64_t)slot * G + g) * ring_tokens + i, dst = ((int64_t)b * rows_per_seq + i) * G + g;
-        for (int j = threadIdx.x - sub * lanes; j < per; j += lanes) {
-            if (j < k16) k_out[dst * k16 + j] = ring_k[src * k16 + j];
-            else v_out[dst * v16 + j - k16] = ring_v[src * v16 + j - k16];
-        }
+    const int part = blockIdx.x % blocks, g = blockIdx.x / blocks % G, b = blockIdx.x / (blocks * G);
+    const int slot = seq_ids ? seq_ids[b] : b, n = min(min(n_old, positions[b] % chunk), ring_tokens);    // the host sized n_old by the same positions
+    const uint4* ks = ring_k + ((int64_t)slot * G + g) * ring_tokens * k16;
+    const uint4* vs = ring_v + ((int64_t)slot * G + g) * ring_tokens * v16;
+    uint4* kd = k_out + ((int64_t)b * rows_per_seq * G + g) * k16;
+    uint4* vd = v_out + ((int64_t)b * rows_per_seq * G + g) * v16;
+    const long long nk = (long long)n * k16, all = nk + (long long)n * v16;
+    uint4 u[GA_BATCH];
+    const long long i0 = (long long)part * GA_THREADS * GA_BATCH + threadIdx.x;
+#pragma unroll
+    for (int x = 0; x < GA_BATCH; ++x) {
+        const long long i = i0 + x * GA_THREADS;
+        if (i < all) u[x] = i < nk ? ks[i] : vs[i - nk];
+    }
+#pragma unroll
+    for (int x = 0; x < GA_BATCH; ++x) {
+        const long long i = i0 + x * GA_THREADS;
+        if (i >= all) break;
+        const unsigned j = (unsigned)(i < nk ? i : i - nk), w = i < nk ? k16 : v16, row = j / w;
+        (i < nk ? kd : vd)[(int64_t)row * G * w + (j - row * w)] = u[x];
     }
 }
 
@@ -177,14 +229,6 @@ struct GqaStepParams {
     float lambda, eps, scale_log2;
 };
 
-// 8 bf16 of `piece` as floats
-__device__ __forceinline__ void unpack8(const uint4& u, float (&f)[8]) {
-    f[0] = bf16_lo(u.x); f[1] = bf16_hi(u.x); f[2] = bf16_lo(u.y); f[3] = bf16_hi(u.y);
-    f[4] = bf16_lo(u.z); f[5] = bf16_hi(u.z); f[6] = bf16_lo(u.w); f[7] = bf16_hi(u.w);
-}
-__device__ __forceinline__ uint4 pack8(const float (&f)[8]) {
-    return make_uint4(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]), pack_bf16(f[4], f[5]), pack_bf16(f[6], f[7]));
-}
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
@@ -549,10 +593,9 @@ extern "C" int bn_kv_prep(const void* k, const void* v, int64_t ld, const void* 
     if (B == 0 || S == 0) return BN_OK;
     KvPrepParams p{k, v, v_first, ld, v_first_ld, seq_ids, positions, k_out, v_out, ring_k, ring_v, B, S, kv_heads, dim_ld, vdim_ld,
                    rms_dim, rows_per_seq, row_offset, ring_tokens, chunk, lambda, eps};
-    const long long blocks = ((long long)B * S * kv_heads + KP_WARPS - 1) / KP_WARPS, cap = (long long)sm_count() * 16;
-    const unsigned grid = (unsigned)(blocks < cap ? blocks : cap);
-    if (dtype == 0) launch_dependent(kv_prep_kernel<float>, grid, KP_WARPS * 32, 0, as_stream(stream), p);
-    else launch_dependent(kv_prep_kernel<__nv_bfloat16>, grid, KP_WARPS * 32, 0, as_stream(stream), p);
+    if ((long long)B * S * kv_heads >= (1LL << 31)) return fail(BN_ERR_UNSUPPORTED, "%s: too many rows", what);
+    if (dtype == 0) kv_prep_launch<float>(p, as_stream(stream));
+    else kv_prep_launch<__nv_bfloat16>(p, as_stream(stream));
     return launch_status(what);
 }
 
@@ -569,11 +612,12 @@ extern "C" int bn_kv_gather(const void* ring_k, const void* ring_v, int ring_tok
         return fail(BN_ERR_INVALID_ARG, "%s: pointers must be 16-byte aligned", what);
     if (int rc = require_sm100()) return rc;
     if (B == 0 || n_old == 0) return BN_OK;
-    const int per = dtype == 0 ? 4 : 8;                   // elements of a 16-byte piece
-    const long long n = (long long)B * n_old * kv_heads, cap = (long long)sm_count() * 16;
-    launch_dependent(kv_gather_kernel, (unsigned)(n < cap ? n : cap), 128, 0, as_stream(stream), static_cast<const uint4*>(ring_k),
-                     static_cast<const uint4*>(ring_v), ring_tokens, kv_heads, dim_ld / per, vdim_ld / per, seq_ids, positions, chunk, B,
-                     n_old, static_cast<uint4*>(k_out), static_cast<uint4*>(v_out), rows_per_seq);
+    const int per = dtype == 0 ? 4 : 8, k16 = dim_ld / per, v16 = vdim_ld / per;          // 16-byte pieces of a row
+    const long long pieces = (long long)n_old * (k16 + v16), blocks = (pieces + GA_THREADS * GA_BATCH - 1) / (GA_THREADS * GA_BATCH);
+    if (pieces >= (1LL << 31) || blocks * B * kv_heads >= (1LL << 31)) return fail(BN_ERR_UNSUPPORTED, "%s: too many rows", what);
+    launch_dependent(kv_gather_kernel, (unsigned)(blocks * B * kv_heads), GA_THREADS, 0, as_stream(stream), static_cast<const uint4*>(ring_k),
+                     static_cast<const uint4*>(ring_v), ring_tokens, kv_heads, k16, v16, seq_ids, positions, chunk, n_old,
+                     static_cast<uint4*>(k_out), static_cast<uint4*>(v_out), rows_per_seq, (int)blocks);
     return launch_status(what);
 }
 

@@ -158,6 +158,7 @@ class ChunkedAttention:
             self.cols.append(self.cols[-1] + part.shape[0])
         o = weight("o", width, c.heads * c.vdim)
         self.o = ops.Linear(pad_heads(o.t(), c.heads, c.vdim).t(), dtype, bias=weight("o.b", width))
+        self.score_bound = 1.02 * c.dim * abs(c.scale)          # unit-RMS queries and keys, the keys rounded to bf16
         self.mix = float(weight("vmix").reshape(-1)[0]) if c.mixes_values else 0.0
 
     def new_state(self, num_seqs: int, max_tokens: Optional[int] = None) -> ChunkCache:
@@ -199,7 +200,7 @@ class ChunkedAttention:
         _lib.check(lib.bn_attn_chunked(
             q, proj.stride(0), keys.data_ptr(), keys.stride(0), values.data_ptr(), values.stride(0), g, proj.stride(0), out.data_ptr(),
             out.stride(0), B, S, n_old, n, c.heads, c.kv_heads, self.dim_ld, self.vdim_ld, c.chunk, c.dim, self.eps, float(c.scale),
-            ops.status_word(dev).data_ptr(), dt, s))
+            self.score_bound, ops.status_word(dev).data_ptr(), dt, s))
 
     def _one_token(self, proj, B, S, cache, seq_ids, positions, n_old, v_first, out):
         c, dev, dt, lib = self.cfg, proj.device, _dt(self.dtype), _lib.load()

@@ -1153,13 +1153,14 @@ def run_ours(args):
         dist.destroy_process_group()
 
 
-def run_soluzen(args):
+def run_design(name, args):
+    """A model design's own measurements (bench_<name>.py) with the clocks seen meanwhile."""
+    import importlib
     import torch
-    import bench_soluzen
     torch.cuda.set_device(0)
     sampler = ClockSampler(0)
     sampler.start()
-    res = bench_soluzen.run(peaks(), max(10, args.steps))
+    res = importlib.import_module("bench_" + name).run(peaks(), max(10, args.steps))
     res["clocks"] = sampler.stop()
     _emit(json.dumps(res))
 
@@ -1193,10 +1194,12 @@ def main():
     ap.add_argument("--soluzen", action="store_true",
                     help="measure the Soluzen design (whole models beside LLaMA, and its kernels one by one) instead of the "
                          "default workload; prints its object alone")
+    ap.add_argument("--duponex", action="store_true", help="the same for the Duponex design")
     args = ap.parse_args()
-    if args.soluzen:
-        run_soluzen(args)
-        return
+    for design in ("soluzen", "duponex"):
+        if getattr(args, design):
+            run_design(design, args)
+            return
     if args.warmup < 3 and args.impl == "ours":
         args.warmup = 3
     if args.impl == "reference":

@@ -519,11 +519,12 @@ BN_API int bn_kv_gather(const void* ring_k, const void* ring_v, int ring_tokens,
                         void* v_out, int rows_per_seq, int dtype, bn_stream_t stream);
 /* portions: key row b * rows_per_seq + n_old + s belongs to query s of sequence b, key row 0 to the first position of a
  * chunk.  q (B*S, q_ld) as projected, k (rows, kv_heads * dim) prepared, v (rows, kv_heads * vdim); the result is multiplied
- * by sigmoid(gate) where gate is given.  error_word (may be null) receives BN_ERR_TIMEOUT if a bounded wait runs out. */
+ * by sigmoid(gate) where gate is given.  score_bound > 0 promises that no scaled score is larger in magnitude (queries and keys
+ * of unit RMS: rms_dim * |scale|), which spares the softmax its maximum.  error_word (may be null) receives BN_ERR_TIMEOUT if a bounded wait runs out. */
 BN_API int bn_attn_chunked(const void* q, int64_t q_ld, const void* k, int64_t k_ld, const void* v, int64_t v_ld,
                            const void* gate, int64_t gate_ld, void* out, int64_t out_ld, int B, int S, int n_old,
                            int rows_per_seq, int H, int kv_heads, int dim, int vdim, int chunk, int rms_dim, float rms_eps,
-                           float scale, int* error_word, int dtype, bn_stream_t stream);
+                           float scale, float score_bound, int* error_word, int dtype, bn_stream_t stream);
 /* one new token per row: prepares and appends its key and value, attends over the ring, gates; q, k, v and gate are columns
  * of the same projection rows (ld).  partial holds B * kv_heads * ceil(H / kv_heads / 16) * splits * 16 * (vdim_ld + 2)
  * floats (splits 1: may be null); tickets B * kv_heads * ceil(H / kv_heads / 16) ints, zero before the first call and left

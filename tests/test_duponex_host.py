@@ -98,7 +98,7 @@ def test_bad_arguments_come_back_as_status(lib):
     p = ctypes.addressof(buf) // 16 * 16 + 16
     # a portion whose old tokens reach behind the chunk's start; more tokens than rows
     for n_old, rows in ((7, 20), (0, 3)):
-        assert lib.bn_attn_chunked(p, 8, p, 8, p, 8, None, 0, p, 8, 1, 4, n_old, rows, 1, 1, 8, 8, 7, 0, 0.0, 1.0, None, 0, None) == \
+        assert lib.bn_attn_chunked(p, 8, p, 8, p, 8, None, 0, p, 8, 1, 4, n_old, rows, 1, 1, 8, 8, 7, 0, 0.0, 1.0, 0.0, None, 0, None) == \
             _lib.BN_ERR_INVALID_ARG
 
 

@@ -290,7 +290,7 @@ def _unpad(t, heads, d):
     return f64(t).reshape(t.shape[:-1] + (heads, -1))[..., :d]
 
 
-def _chunked_attention(q, k, v, gate, n_old, chunk, scale, eps, dtype):
+def _chunked_attention(q, k, v, gate, n_old, chunk, scale, eps, dtype, bound=0.0):
     """bn_attn_chunked on (T, heads, .) arrays whose first n_old keys have no query; queries as projected, keys prepared."""
     from baranet_bdml_b200 import _lib
     n, G, E = k.shape
@@ -300,7 +300,8 @@ def _chunked_attention(q, k, v, gate, n_old, chunk, scale, eps, dtype):
     word = torch.zeros(1, dtype=torch.int32, device="cuda")
     _lib.check(_lib.load().bn_attn_chunked(
         qg.data_ptr(), qg.stride(0), kg.data_ptr(), kg.stride(0), vg.data_ptr(), vg.stride(0), gg.data_ptr(), gg.stride(0), out.data_ptr(),
-        out.stride(0), 1, S, n_old, n, H, G, kg.shape[1] // G, vg.shape[1] // G, chunk, E, eps, scale, word.data_ptr(), code(dtype), stream()))
+        out.stride(0), 1, S, n_old, n, H, G, kg.shape[1] // G, vg.shape[1] // G, chunk, E, eps, scale, bound, word.data_ptr(), code(dtype),
+        stream()))
     torch.cuda.synchronize()
     assert int(word.item()) == 0
     Q = np.concatenate([np.zeros((n_old, H, E)), R.unit_rms(_unpad(qg, H, E), eps)])
@@ -317,9 +318,10 @@ def test_chunked_attention(lib, dtype, H, G, E, V, S, n_old, chunk):
     rng = np.random.default_rng(S + chunk + E)
     n = S + n_old
     q, k = 3.0 * rng.standard_normal((S, H, E)) * rng.uniform(0.1, 2.0, (S, H, 1)), R.unit_rms(rng.standard_normal((n, G, E)), 1e-5)
-    got, want = _chunked_attention(q, k, rng.standard_normal((n, G, V)), 2 * rng.standard_normal((S, H, V)), n_old, chunk, 4.0 * E ** -0.5,
-                                   1e-5, dtype)
-    assert np.abs(got - want).max() <= (2e-5 if dtype == torch.float32 else 3e-2)
+    v, g, scale = rng.standard_normal((n, G, V)), 2 * rng.standard_normal((S, H, V)), 4.0 * E ** -0.5
+    for bound in (0.0, 1.02 * E * scale):
+        got, want = _chunked_attention(q, k, v, g, n_old, chunk, scale, 1e-5, dtype, bound)
+        assert np.abs(got - want).max() <= (2e-5 if dtype == torch.float32 else 3e-2), bound
 
 
 @DTYPES
@@ -338,7 +340,7 @@ def test_keys_just_inside_and_outside_a_chunk(lib, dtype, chunk, n_old):
         v = rng.standard_normal((n, G, V)) * 0.1
         v[key] = 5.0
         q = np.tile(u * 0.3, (S, H, 1)) + 0.001 * rng.standard_normal((S, H, E))
-        got, want = _chunked_attention(q, k, v, np.full((S, H, V), 20.0), n_old, chunk, 10.0 / E, 1e-5, dtype)
+        got, want = _chunked_attention(q, k, v, np.full((S, H, V), 20.0), n_old, chunk, 10.0 / E, 1e-5, dtype, bound=10.2)
         assert np.abs(got - want).max() <= (5e-5 if dtype == torch.float32 else 3e-2), key
         seen = np.array([i >= key and i // chunk == key // chunk for i in range(n_old, n)])
         if seen.any():
