@@ -134,7 +134,7 @@ extern "C" int bn_attn_window(const void* q, int64_t q_ld, const void* k, const 
     p.k_head = dim; p.v_head = vdim; p.k_seq = p.v_seq = rows_per_seq * kv_ld;
     p.B = B; p.S = S; p.n_old = n_old; p.rows_per_seq = rows_per_seq; p.H = p.kv_heads = H; p.dim = dim; p.rot = rot; p.vdim = vdim;
     p.mask = MASK_WINDOW; p.span = window; p.scale = scale; p.error_word = error_word;
-    if (dtype == 1 && attn_window_sm100_ok(p)) return attn_window_sm100(p, as_stream(stream));
+    if (dtype == 1 && attn_portion_sm100_ok(p)) return attn_portion_sm100(p, as_stream(stream));
     return attn_any(p, dtype, as_stream(stream), what);
 }
 
@@ -157,6 +157,6 @@ extern "C" int bn_attn_chunked(const void* q, int64_t q_ld, const void* k, int64
     p.B = B; p.S = S; p.n_old = n_old; p.rows_per_seq = rows_per_seq; p.H = H; p.kv_heads = kv_heads; p.dim = dim; p.vdim = vdim;
     p.mask = MASK_CHUNK; p.span = chunk; p.rms_dim = rms_dim; p.rms_eps = rms_eps; p.scale = scale; p.score_bound = score_bound;
     p.error_word = error_word;
-    if (dtype == 1 && attn_window_sm100_ok(p)) return attn_window_sm100(p, as_stream(stream));
+    if (dtype == 1 && attn_portion_sm100_ok(p)) return attn_portion_sm100(p, as_stream(stream));
     return attn_any(p, dtype, as_stream(stream), what);
 }

@@ -30,8 +30,8 @@ struct AttnPortionParams {
     int* error_word;                  // optional; set when a bounded wait ran out
 };
 
-bool attn_window_sm100_ok(const AttnPortionParams& p);
-int attn_window_sm100(const AttnPortionParams& p, cudaStream_t stream);
+bool attn_portion_sm100_ok(const AttnPortionParams& p);
+int attn_portion_sm100(const AttnPortionParams& p, cudaStream_t stream);
 // the kernel for any sizes; also one-token rows over a cache (positions set)
 int attn_any(const AttnPortionParams& p, int dtype, cudaStream_t stream, const char* what);
 

@@ -115,7 +115,7 @@ struct WaCursor {
 // NBK, NBV: 64-column blocks of keys and values, 0: any number
 template <bool BOUNDED, int NBK, int NBV>
 __global__ void __launch_bounds__(WA_THREADS, 1)
-attn_window_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
+attn_portion_sm100_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                          const __grid_constant__ CUtensorMap tmap_r, const __grid_constant__ CUtensorMap tmap_v,
                          const WaParams p) {
     extern __shared__ uint8_t smem_raw[];
@@ -510,7 +510,7 @@ static int wa_stages(int nb, int nb_v) {
     return s > WA_MAXSTAGE ? WA_MAXSTAGE : s;
 }
 
-bool attn_window_sm100_ok(const AttnPortionParams& p) {
+bool attn_portion_sm100_ok(const AttnPortionParams& p) {
     const int nb = (p.dim + 63) / 64 + (p.rot + 63) / 64, nb_v = (p.vdim + 63) / 64;
     const uintptr_t bases = reinterpret_cast<uintptr_t>(p.q) | reinterpret_cast<uintptr_t>(p.k) | reinterpret_cast<uintptr_t>(p.v) |
                             reinterpret_cast<uintptr_t>(p.krot) | reinterpret_cast<uintptr_t>(p.gate) | reinterpret_cast<uintptr_t>(p.out);
@@ -531,16 +531,16 @@ static int wa_launch(unsigned grid, size_t smem, cudaStream_t st, const CUtensor
                      const CUtensorMap& mv, const WaParams& p, int dev, const char* what) {
     static thread_local int configured_dev = -1;
     if (configured_dev != dev) {
-        cudaError_t e = cudaFuncSetAttribute(attn_window_sm100_kernel<BOUNDED, NBK, NBV>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+        cudaError_t e = cudaFuncSetAttribute(attn_portion_sm100_kernel<BOUNDED, NBK, NBV>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                              WA_SMEM_LIMIT);
         if (e != cudaSuccess) return fail(BN_ERR_CUDA, "%s: %s", what, cudaGetErrorString(e));
         configured_dev = dev;
     }
-    attn_window_sm100_kernel<BOUNDED, NBK, NBV><<<grid, WA_THREADS, smem, st>>>(mq, mk, mr, mv, p);
+    attn_portion_sm100_kernel<BOUNDED, NBK, NBV><<<grid, WA_THREADS, smem, st>>>(mq, mk, mr, mv, p);
     return launch_status(what);
 }
 
-int attn_window_sm100(const AttnPortionParams& a, cudaStream_t st) {
+int attn_portion_sm100(const AttnPortionParams& a, cudaStream_t st) {
     const char* what = "portion attention";
     CUtensorMap mq, mk, mr, mv;
     if (int rc = wa_map(&mq, a.q, a.dim + a.rot, a.H, a.dim + a.rot, a.S, a.q_ld, a.B, WA_BM)) return rc;

@@ -186,35 +186,35 @@ kv_gather_kernel(const uint4* ring_k, const uint4* ring_v, int ring_tokens, int 
 constexpr int ST_KEYS = 32, ST_BLK = ST_KEYS * 128;       // a 64-column block of a warp's tile: 4 KB
 constexpr int ST_MAXSTAGE = 4, ST_MAXWARPS = 4, ST_MAXSPLITS = 64;
 constexpr int ST_MAXDIM = 256;
-constexpr size_t ST_SMEM_ONE = 220 * 1024, ST_SMEM_TWO = 107 * 1024;      // dynamic, for one or two CTAs per SM beside 5 KB static
+constexpr int ST_SMEM_ONE = 220 * 1024, ST_SMEM_TWO = 107 * 1024;      // dynamic, for one or two CTAs per SM beside 5 KB static
 constexpr float ST_LOG2E = 1.4426950408889634f;
 
 struct StLayout {
     int nbk, nbv, warps, stages, ctas;                    // ctas: resident per SM
-    size_t tile, q, knew, vnew, gate, ring, total;        // byte sizes and offsets
+    int tile, q, knew, vnew, gate, ring, total;           // byte sizes and offsets
 };
 
-__host__ __device__ inline StLayout st_layout(int dim_ld, int vdim_ld) {
+static StLayout st_layout(int dim_ld, int vdim_ld) {
     StLayout L;
     L.nbk = (dim_ld + 63) / 64;
     L.nbv = (vdim_ld + 63) / 64;
-    L.tile = (size_t)(L.nbk + L.nbv) * ST_BLK;
+    L.tile = (L.nbk + L.nbv) * ST_BLK;
     L.q = 0;                                              // [16][nbk * 64 + 8] bf16
-    L.knew = L.q + (size_t)16 * (L.nbk * 64 + 8) * 2;     // [nbk * 64] bf16
-    L.vnew = L.knew + (size_t)L.nbk * 128;                // [nbv * 64] bf16
-    L.gate = L.vnew + (size_t)L.nbv * 128;                // [16][vdim_ld] bf16
-    L.ring = (L.gate + (size_t)32 * vdim_ld + 1023) / 1024 * 1024;
-    const size_t fixed = 1024 + L.ring;
+    L.knew = L.q + 16 * (L.nbk * 64 + 8) * 2;             // [nbk * 64] bf16
+    L.vnew = L.knew + L.nbk * 128;                        // [nbv * 64] bf16
+    L.gate = L.vnew + L.nbv * 128;                        // [16][vdim_ld] bf16
+    L.ring = (L.gate + 32 * vdim_ld + 1023) / 1024 * 1024;
+    const int fixed = 1024 + L.ring;
     L.warps = ST_MAXWARPS;
     for (;; L.warps /= 2) {
-        const size_t stage = (size_t)L.warps * L.tile;
-        const int two = (int)((ST_SMEM_TWO - fixed) / stage), one = (int)((ST_SMEM_ONE - fixed) / stage);
+        const int stage = L.warps * L.tile;
+        const int two = (ST_SMEM_TWO - fixed) / stage, one = (ST_SMEM_ONE - fixed) / stage;
         L.ctas = two >= 3 ? 2 : 1;
         L.stages = two >= 3 ? two : one;
         if (L.stages >= 2 || L.warps == 1) break;
     }
     if (L.stages > ST_MAXSTAGE) L.stages = ST_MAXSTAGE;
-    L.total = fixed + (size_t)L.warps * L.stages * L.tile;
+    L.total = fixed + L.warps * L.stages * L.tile;
     return L;
 }
 
@@ -227,6 +227,7 @@ struct GqaStepParams {
     int *tickets, *error_word;
     int G, rep, groups, dim_ld, vdim_ld, rms_dim, ring_tokens, chunk, splits;
     float lambda, eps, scale_log2;
+    StLayout L;
 };
 
 __device__ __forceinline__ float warp_sum(float v) {
@@ -235,23 +236,26 @@ __device__ __forceinline__ float warp_sum(float v) {
     return v;
 }
 
-// NVP: 8-column pieces of the values a warp accumulates, vdim_ld <= 8 NVP
-template <int NVP>
-__global__ void __launch_bounds__(ST_MAXWARPS * 32)
+// NVP: 8-column pieces of the values a warp accumulates, vdim_ld <= 8 NVP.  KS: dim_ld is 16 KS and vdim_ld is 8 NVP exactly;
+// 0: any sizes
+template <int NVP, int KS>
+__global__ void __launch_bounds__(ST_MAXWARPS * 32, 2)
 gqa_step_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constant__ CUtensorMap tmap_v, const GqaStepParams p) {
     extern __shared__ uint8_t smem_raw[];
     __shared__ __align__(8) uint64_t bar[ST_MAXWARPS][ST_MAXSTAGE];
     __shared__ float s_scale[16], s_ml[ST_MAXWARPS][16][2], s_w[16][ST_MAXSPLITS];
     __shared__ int s_abort, s_last;
     const int tid = threadIdx.x, warp = tid / 32, lane = tid % 32, nw = blockDim.x / 32;
-    const StLayout L = st_layout(p.dim_ld, p.vdim_ld);
+    const StLayout& L = p.L;
+    const int nbk = KS ? (KS + 3) / 4 : L.nbk, nbv = KS ? (NVP + 7) / 8 : L.nbv, tile = (nbk + nbv) * ST_BLK;
+    const int dim_ld = KS ? KS * 16 : p.dim_ld, vdim_ld = KS ? NVP * 8 : p.vdim_ld;
     uint8_t* base = smem_raw + (((smem_u32(smem_raw) + 1023u) & ~1023u) - smem_u32(smem_raw));
     __nv_bfloat16* sq = reinterpret_cast<__nv_bfloat16*>(base + L.q);
     __nv_bfloat16* sknew = reinterpret_cast<__nv_bfloat16*>(base + L.knew);
     __nv_bfloat16* svnew = reinterpret_cast<__nv_bfloat16*>(base + L.vnew);
     __nv_bfloat16* sgate = reinterpret_cast<__nv_bfloat16*>(base + L.gate);
-    const int q_ld = L.nbk * 64 + 8;
-    uint8_t* ring = base + L.ring + (size_t)warp * L.stages * L.tile;     // this warp's stages
+    const int q_ld = nbk * 64 + 8;
+    uint8_t* ring = base + L.ring + warp * L.stages * tile;     // this warp's stages
     const uint32_t ring_u = smem_u32(ring);
     const int split = blockIdx.x % p.splits, item = blockIdx.x / p.splits;
     const int grp = item % p.groups, g = item / p.groups % p.G, b = item / (p.groups * p.G);
@@ -268,81 +272,101 @@ gqa_step_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constan
     __syncthreads();
     grid_dependency_wait();
     grid_launch_dependents();
-    const int pos = p.positions[b], slot = p.seq_ids ? p.seq_ids[b] : b, local = pos % p.chunk;
+    const int pos = p.positions[b], slot = p.seq_ids ? p.seq_ids[b] : b;
+    // This warp's part of the projection row is requested before the cache is streamed, or it would arrive behind the stream.
+    // A lane has 8 columns of a head.  Queries as they are (zeros beyond the group's heads and their columns), their norms go
+    // into the score scale; key and value of the new token where this part may hold it
+    const int c8 = lane * 8;
+    const uint4 z = make_uint4(0, 0, 0, 0);
+    const __nv_bfloat16* qrow = p.q + b * p.ld + h0 * dim_ld + c8;
+    const __nv_bfloat16* grow = p.gate + b * p.ld + h0 * vdim_ld + c8;
+    uint4 uk = z, uv = z, uf = z, uq[4], ug[4];
+    auto load_heads = [&](int r0) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            uq[i] = r0 + i < nh && c8 < dim_ld ? *reinterpret_cast<const uint4*>(qrow + (r0 + i) * dim_ld) : z;
+            ug[i] = p.gate && r0 + i < nh && c8 < vdim_ld ? *reinterpret_cast<const uint4*>(grow + (r0 + i) * vdim_ld) : z;
+        }
+    };
+    load_heads(warp * 4);
+    if (warp == 0 && c8 < dim_ld) uk = *reinterpret_cast<const uint4*>(p.k + b * p.ld + g * dim_ld + c8);
+    if (warp == nw - 1 && c8 < vdim_ld) {
+        uv = *reinterpret_cast<const uint4*>(p.v + b * p.ld + g * vdim_ld + c8);
+        if (p.v_first) uf = *reinterpret_cast<const uint4*>(p.v_first + b * p.v_first_ld + g * vdim_ld + c8);
+    }
+
+    const int local = pos % p.chunk;
     const int n = local < p.ring_tokens ? local + 1 : 0;                  // keys; none: the cache has no room, the result is NaN
     const int tiles = (n + ST_KEYS - 1) / ST_KEYS, rounds = (tiles + nw - 1) / nw;
     const int per = (rounds + p.splits - 1) / p.splits * nw;
     const int t_begin = min(tiles, split * per), t_end = min(tiles, t_begin + per);
     const int row0 = (slot * p.G + g) * p.ring_tokens;
     const bool owner = t_begin < tiles && t_end == tiles;                 // this part holds the new token
+    const bool new_k = owner && warp == 0, new_v = owner && warp == nw - 1;
 
     auto issue = [&](int t, int stage) {
-        const uint32_t full = smem_u32(&bar[warp][stage]), dst = ring_u + stage * (uint32_t)L.tile;
-        mbar_arrive_expect_tx(full, (uint32_t)L.tile);
-        for (int x = 0; x < L.nbk; ++x) tma_load_2d(dst + x * ST_BLK, &tmap_k, x * 64, row0 + t * ST_KEYS, full);
-        for (int x = 0; x < L.nbv; ++x) tma_load_2d(dst + (L.nbk + x) * ST_BLK, &tmap_v, x * 64, row0 + t * ST_KEYS, full);
+        const uint32_t full = smem_u32(&bar[warp][stage]), dst = ring_u + stage * tile;
+        mbar_arrive_expect_tx(full, (uint32_t)tile);
+        for (int x = 0; x < nbk; ++x) tma_load_2d(dst + x * ST_BLK, &tmap_k, x * 64, row0 + t * ST_KEYS, full);
+        for (int x = 0; x < nbv; ++x) tma_load_2d(dst + (nbk + x) * ST_BLK, &tmap_v, x * 64, row0 + t * ST_KEYS, full);
     };
     if (lane == 0)
         for (int s = 0; s < L.stages; ++s)
             if (t_begin + warp + s * nw < t_end) issue(t_begin + warp + s * nw, s);
 
-    // queries of the group as they are, zeros beyond its heads and their columns; their norms go into the score scale
-    for (int h = warp; h < 16; h += nw) {
-        float ss = 0.f;
-        for (int c = lane * 8; c < q_ld; c += 256) {
-            uint4 u = make_uint4(0, 0, 0, 0);
-            if (h < nh && c < p.dim_ld) u = *reinterpret_cast<const uint4*>(p.q + b * p.ld + (h0 + h) * p.dim_ld + c);
-            *reinterpret_cast<uint4*>(sq + h * q_ld + c) = u;
+    for (int r0 = warp * 4; r0 < 16; r0 += nw * 4) {
+        if (r0 > warp * 4) load_heads(r0);
+        float ss[4];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
             float f[8];
-            unpack8(u, f);
+            unpack8(uq[i], f);
+            ss[i] = 0.f;
 #pragma unroll
-            for (int e = 0; e < 8; ++e) ss = fmaf(f[e], f[e], ss);
+            for (int e = 0; e < 8; ++e) ss[i] = fmaf(f[e], f[e], ss[i]);
+            if (c8 < q_ld) *reinterpret_cast<uint4*>(sq + (r0 + i) * q_ld + c8) = uq[i];
+            if (c8 < vdim_ld) *reinterpret_cast<uint4*>(sgate + (r0 + i) * vdim_ld + c8) = ug[i];
         }
-        if (p.rms_dim) ss = rsqrtf(warp_sum(ss) / (float)p.rms_dim + p.eps);
-        if (lane == 0) s_scale[h] = p.rms_dim ? p.scale_log2 * ss : p.scale_log2;
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], o);
+        if (lane < 4) {
+            const float t = lane == 0 ? ss[0] : lane == 1 ? ss[1] : lane == 2 ? ss[2] : ss[3];
+            s_scale[r0 + lane] = p.rms_dim ? p.scale_log2 * rsqrtf(t / (float)p.rms_dim + p.eps) : p.scale_log2;
+        }
     }
-    if (p.gate)
-        for (int i = tid; i < nh * (p.vdim_ld / 8); i += blockDim.x) {
-            const int h = i / (p.vdim_ld / 8), c = (i - h * (p.vdim_ld / 8)) * 8;
-            *reinterpret_cast<uint4*>(sgate + h * p.vdim_ld + c) =
-                *reinterpret_cast<const uint4*>(p.gate + b * p.ld + (h0 + h) * p.vdim_ld + c);
-        }
-    if (owner && warp == 0) {
-        const int c = lane * 8;
-        float f[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f}, ss = 0.f;
-        if (c < p.dim_ld) unpack8(*reinterpret_cast<const uint4*>(p.k + b * p.ld + g * p.dim_ld + c), f);
+    if (new_k) {
         if (p.rms_dim) {
+            float f[8], t = 0.f;
+            unpack8(uk, f);
 #pragma unroll
-            for (int e = 0; e < 8; ++e) ss = fmaf(f[e], f[e], ss);
-            const float inv = rsqrtf(warp_sum(ss) / (float)p.rms_dim + p.eps);
+            for (int e = 0; e < 8; ++e) t = fmaf(f[e], f[e], t);
+            const float inv = rsqrtf(warp_sum(t) / (float)p.rms_dim + p.eps);
 #pragma unroll
             for (int e = 0; e < 8; ++e) f[e] *= inv;
+            uk = pack8(f);
         }
-        const uint4 u = pack8(f);
-        if (c < L.nbk * 64) *reinterpret_cast<uint4*>(sknew + c) = u;
-        if (grp == 0 && c < p.dim_ld) *reinterpret_cast<uint4*>(p.ring_k + (int64_t)(row0 + local) * p.dim_ld + c) = u;
+        if (c8 < nbk * 64) *reinterpret_cast<uint4*>(sknew + c8) = uk;
+        if (grp == 0 && c8 < dim_ld) *reinterpret_cast<uint4*>(p.ring_k + (int64_t)(row0 + local) * dim_ld + c8) = uk;
     }
-    if (owner && warp == nw - 1) {
-        const int c = lane * 8;
-        float f[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-        if (c < p.vdim_ld) {
-            unpack8(*reinterpret_cast<const uint4*>(p.v + b * p.ld + g * p.vdim_ld + c), f);
-            if (p.v_first) {
-                float a[8];
-                unpack8(*reinterpret_cast<const uint4*>(p.v_first + b * p.v_first_ld + g * p.vdim_ld + c), a);
+    if (new_v) {
+        if (p.v_first) {
+            float f[8], a[8];
+            unpack8(uv, f);
+            unpack8(uf, a);
 #pragma unroll
-                for (int e = 0; e < 8; ++e) f[e] = fmaf(p.lambda, a[e], (1.f - p.lambda) * f[e]);
-            }
+            for (int e = 0; e < 8; ++e) f[e] = fmaf(p.lambda, a[e], (1.f - p.lambda) * f[e]);
+            uv = pack8(f);
         }
-        const uint4 u = pack8(f);
-        if (c < L.nbv * 64) *reinterpret_cast<uint4*>(svnew + c) = u;
-        if (grp == 0 && c < p.vdim_ld) *reinterpret_cast<uint4*>(p.ring_v + (int64_t)(row0 + local) * p.vdim_ld + c) = u;
+        if (c8 < nbv * 64) *reinterpret_cast<uint4*>(svnew + c8) = uv;
+        if (grp == 0 && c8 < vdim_ld) *reinterpret_cast<uint4*>(p.ring_v + (int64_t)(row0 + local) * vdim_ld + c8) = uv;
     }
     __syncthreads();
 
     const int gq = lane / 4, j = lane % 4;
     const float sc_lo = s_scale[gq], sc_hi = s_scale[gq + 8];
-    const int k_steps = (p.dim_ld + 15) / 16, npc = p.vdim_ld / 8;
+    const int k_steps = KS ? KS : (dim_ld + 15) / 16, npc = KS ? NVP : vdim_ld / 8;
     const uint32_t qa = smem_u32(sq) + ((lane % 16) * q_ld + (lane / 16) * 8) * 2;
     float acc[NVP][4];
 #pragma unroll
@@ -350,7 +374,7 @@ gqa_step_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constan
     float m_lo = -INFINITY, m_hi = -INFINITY, l_lo = 0.f, l_hi = 0.f;
     for (int t = t_begin + warp, it = 0; t < t_end; t += nw, ++it) {
         const int stage = it % L.stages;
-        const uint32_t tk = ring_u + stage * (uint32_t)L.tile, tv = tk + L.nbk * ST_BLK;
+        const uint32_t tk = ring_u + stage * tile, tv = tk + nbk * ST_BLK;
         if (__any_sync(0xffffffffu, !mbar_wait(smem_u32(&bar[warp][stage]), (it / L.stages) & 1u, &s_abort))) {
             for (int k = 1; k < L.stages && t + k * nw < t_end; ++k)        // what else is in flight, as far as it arrives
                 mbar_wait(smem_u32(&bar[warp][(it + k) % L.stages]), ((it + k) / L.stages) & 1u, &s_abort);
@@ -358,9 +382,9 @@ gqa_step_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constan
         }
         if (t == tiles - 1) {                             // the new token's row, whatever the cache still held there
             const int r = local % ST_KEYS;
-            uint8_t* at = ring + stage * L.tile + r * 128;
-            for (int c = lane; c < (L.nbk + L.nbv) * 8; c += 32) {
-                const uint4 u = c < L.nbk * 8 ? reinterpret_cast<const uint4*>(sknew)[c] : reinterpret_cast<const uint4*>(svnew)[c - L.nbk * 8];
+            uint8_t* at = ring + stage * tile + r * 128;
+            for (int c = lane; c < (nbk + nbv) * 8; c += 32) {
+                const uint4 u = c < nbk * 8 ? reinterpret_cast<const uint4*>(sknew)[c] : reinterpret_cast<const uint4*>(svnew)[c - nbk * 8];
                 *reinterpret_cast<uint4*>(at + (c / 8) * ST_BLK + (((c % 8) ^ (r & 7)) << 4)) = u;
             }
             __syncwarp();
@@ -370,8 +394,7 @@ gqa_step_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constan
 #pragma unroll
         for (int i = 0; i < 4; ++i) c[i][0] = c[i][1] = c[i][2] = c[i][3] = 0.f;
         const int row = (lane / 16) * 8 + lane % 8, kpart = (lane / 8) % 2;          // B fragments: keys (0-7 | 8-15) x columns (0-7 | 8-15)
-#pragma unroll 4
-        for (int ks = 0; ks < k_steps; ++ks) {
+        auto score_step = [&](int ks) {
             uint32_t a0, a1, a2, a3;
             ldmatrix_x4(qa + ks * 32, a0, a1, a2, a3);
             const int chunk = ks * 2 + kpart;
@@ -383,6 +406,13 @@ gqa_step_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constan
                 mma_bf16_16816(c[2 * half], a0, a1, a2, a3, b0, b1);
                 mma_bf16_16816(c[2 * half + 1], a0, a1, a2, a3, b2, b3);
             }
+        };
+        if (KS) {
+#pragma unroll
+            for (int ks = 0; ks < KS; ++ks) score_step(ks);
+        } else {
+#pragma unroll 4
+            for (int ks = 0; ks < k_steps; ++ks) score_step(ks);
         }
         float x_lo = -INFINITY, x_hi = -INFINITY;
 #pragma unroll
@@ -432,7 +462,7 @@ gqa_step_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constan
         }
 #pragma unroll
         for (int i = 0; i < NVP; ++i) {
-            if (i >= npc) break;
+            if (!KS && i >= npc) break;
             uint32_t b0, b1, b2, b3;                      // 32 keys: four 8 x 8 matrices, transposed
             ldmatrix_x4_trans(tv + (i / 8) * ST_BLK + lane * 128 + (((i % 8) ^ (lane & 7)) << 4), b0, b1, b2, b3);
             mma_bf16_16816(acc[i], a[0][0], a[0][1], a[0][2], a[0][3], b0, b1);
@@ -448,12 +478,12 @@ gqa_step_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constan
     }
     // ---- the CTA's part: the warps' sums through shared memory (a warp's own stages; everything it asked for has arrived)
     __syncwarp();
-    const int o_ld = p.vdim_ld + 8;
+    const int o_ld = vdim_ld + 8;
     if (s_abort == 0) {
         float* so = reinterpret_cast<float*>(ring);
 #pragma unroll
         for (int i = 0; i < NVP; ++i) {
-            if (i >= npc) break;
+            if (!KS && i >= npc) break;
             *reinterpret_cast<float2*>(so + gq * o_ld + i * 8 + 2 * j) = make_float2(acc[i][0], acc[i][1]);
             *reinterpret_cast<float2*>(so + (gq + 8) * o_ld + i * 8 + 2 * j) = make_float2(acc[i][2], acc[i][3]);
         }
@@ -466,16 +496,16 @@ gqa_step_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constan
     const bool bad = s_abort != 0;
     const float nan = __int_as_float(0x7fc00000);
     if (bad && tid == 0 && p.error_word) atomicExch(p.error_word, BN_ERR_TIMEOUT);
-    const int quads = p.vdim_ld / 4;
+    const int quads = vdim_ld / 4;
     auto emit = [&](int r, int c4, float4 o) {            // four output columns of head r
         float f[4] = {o.x, o.y, o.z, o.w};
         if (p.gate) {
             float gt[4];
-            load4(sgate + r * p.vdim_ld + c4, gt);
+            load4(sgate + r * vdim_ld + c4, gt);
 #pragma unroll
             for (int e = 0; e < 4; ++e) f[e] *= sigmoid_fast(gt[e]);
         }
-        store4(p.out + b * p.out_ld + (h0 + r) * p.vdim_ld + c4, f);
+        store4(p.out + b * p.out_ld + (h0 + r) * vdim_ld + c4, f);
     };
     for (int i = tid; i < nh * quads; i += blockDim.x) {
         const int r = i / quads, c4 = (i - r * quads) * 4;
@@ -484,7 +514,7 @@ gqa_step_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constan
         for (int w = 0; w < nw; ++w) M = fmaxf(M, s_ml[w][r][0]);
         for (int w = 0; w < nw && !bad; ++w) {
             const float f = M == -INFINITY ? 0.f : ex2(s_ml[w][r][0] - M);
-            const float4 u = *reinterpret_cast<const float4*>(base + L.ring + (size_t)w * L.stages * L.tile + ((size_t)r * o_ld + c4) * 4);
+            const float4 u = *reinterpret_cast<const float4*>(base + L.ring + w * L.stages * tile + (r * o_ld + c4) * 4);
             l = fmaf(s_ml[w][r][1], f, l);
             o.x = fmaf(u.x, f, o.x); o.y = fmaf(u.y, f, o.y); o.z = fmaf(u.z, f, o.z); o.w = fmaf(u.w, f, o.w);
         }
@@ -493,7 +523,7 @@ gqa_step_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constan
             emit(r, c4, make_float4(o.x * inv, o.y * inv, o.z * inv, o.w * inv));
         } else {
             const int64_t part = ((int64_t)item * p.splits + split) * 16 + r;
-            *reinterpret_cast<float4*>(p.part_o + part * p.vdim_ld + c4) = o;
+            *reinterpret_cast<float4*>(p.part_o + part * vdim_ld + c4) = o;
             if (c4 == 0) *reinterpret_cast<float2*>(p.part_ml + part * 2) = make_float2(M, bad ? nan : l);
         }
     }
@@ -537,10 +567,10 @@ gqa_step_kernel(const __grid_constant__ CUtensorMap tmap_k, const __grid_constan
     for (int i = tid; i < nh * quads; i += blockDim.x) {
         const int r = i / quads, c4 = (i - r * quads) * 4;
         float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
-        const float4* src = reinterpret_cast<const float4*>(p.part_o + ((int64_t)item * p.splits * 16 + r) * p.vdim_ld + c4);
+        const float4* src = reinterpret_cast<const float4*>(p.part_o + ((int64_t)item * p.splits * 16 + r) * vdim_ld + c4);
 #pragma unroll 8
         for (int s = 0; s < p.splits; ++s) {
-            const float4 u = __ldcg(src + (int64_t)s * 4 * p.vdim_ld);
+            const float4 u = __ldcg(src + (int64_t)s * 4 * vdim_ld);
             const float f = s_w[r][s];
             o.x = fmaf(u.x, f, o.x); o.y = fmaf(u.y, f, o.y); o.z = fmaf(u.z, f, o.z); o.w = fmaf(u.w, f, o.w);
         }
@@ -556,18 +586,18 @@ static bool sizes_ok(int H, int G, int dim_ld, int vdim_ld) {
     return H > 0 && G > 0 && H % G == 0 && dim_ld > 0 && vdim_ld > 0 && dim_ld % 8 == 0 && vdim_ld % 8 == 0;
 }
 
-template <int NVP>
-static int gqa_step_launch(const CUtensorMap& mk, const CUtensorMap& mv, const GqaStepParams& p, const StLayout& L, unsigned grid,
-                           cudaStream_t st, const char* what) {
+template <int NVP, int KS>
+static int gqa_step_launch(const CUtensorMap& mk, const CUtensorMap& mv, const GqaStepParams& p, unsigned grid, cudaStream_t st,
+                           const char* what) {
     int dev = 0;
     cudaGetDevice(&dev);
     static thread_local int configured_dev = -1;
     if (configured_dev != dev) {
-        cudaError_t e = cudaFuncSetAttribute(gqa_step_kernel<NVP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)ST_SMEM_ONE);
+        cudaError_t e = cudaFuncSetAttribute(gqa_step_kernel<NVP, KS>, cudaFuncAttributeMaxDynamicSharedMemorySize, ST_SMEM_ONE);
         if (e != cudaSuccess) return fail(BN_ERR_CUDA, "%s: %s", what, cudaGetErrorString(e));
         configured_dev = dev;
     }
-    launch_dependent(gqa_step_kernel<NVP>, grid, L.warps * 32, L.total, st, mk, mv, p);
+    launch_dependent(gqa_step_kernel<NVP, KS>, grid, p.L.warps * 32, p.L.total, st, mk, mv, p);
     return launch_status(what);
 }
 
@@ -621,7 +651,8 @@ extern "C" int bn_kv_gather(const void* ring_k, const void* ring_v, int ring_tok
     return launch_status(what);
 }
 
-// CTAs of a part cost their rounds of tiles plus about two for their start and end: the cut whose waves take the least time
+// A CTA costs its rounds of tiles plus about seven for its start and end, merging parts about five: the cut whose waves take
+// the least time
 extern "C" int bn_gqa_step_splits(int B, int H, int kv_heads, int dim_ld, int vdim_ld, int ring_tokens, int dtype) {
     if (B <= 0 || !sizes_ok(H, kv_heads, dim_ld, vdim_ld) || ring_tokens <= 0) return 0;
     if (!gqa_step_mma_ok(dim_ld, vdim_ld, dtype)) return 1;
@@ -632,7 +663,7 @@ extern "C" int bn_gqa_step_splits(int B, int H, int kv_heads, int dim_ld, int vd
     double best_cost = 1e30;
     for (int s = 1; s <= rounds && s <= ST_MAXSPLITS; ++s) {
         const long long waves = (items * s + slots - 1) / slots;
-        const double cost = (double)waves * ((rounds + s - 1) / s + 2.0) + (s > 1 ? 1.0 : 0.0) + 0.05 * s;
+        const double cost = (double)waves * ((rounds + s - 1) / s + 7.0) + (s > 1 ? 5.0 : 0.0) + 0.05 * s;
         if (cost < best_cost) { best_cost = cost; best = s; }
     }
     return best;
@@ -701,9 +732,11 @@ extern "C" int bn_gqa_step(const void* q, const void* k, const void* v, const vo
     const int64_t items = (int64_t)B * kv_heads * p.groups;
     p.part_o = partial;                                   // items * splits * 16 rows of vdim_ld, then of 2
     p.part_ml = partial ? partial + items * splits * 16 * vdim_ld : nullptr;
-    const StLayout L = st_layout(dim_ld, vdim_ld);
+    p.L = st_layout(dim_ld, vdim_ld);
     const unsigned grid = (unsigned)(items * splits);
-    if (vdim_ld <= 64) return gqa_step_launch<8>(mk, mv, p, L, grid, st, what);
-    if (vdim_ld <= 128) return gqa_step_launch<16>(mk, mv, p, L, grid, st, what);
-    return gqa_step_launch<32>(mk, mv, p, L, grid, st, what);
+    if (dim_ld == 64 && vdim_ld == 64) return gqa_step_launch<8, 4>(mk, mv, p, grid, st, what);
+    if (dim_ld == 128 && vdim_ld == 128) return gqa_step_launch<16, 8>(mk, mv, p, grid, st, what);
+    if (vdim_ld <= 64) return gqa_step_launch<8, 0>(mk, mv, p, grid, st, what);
+    if (vdim_ld <= 128) return gqa_step_launch<16, 0>(mk, mv, p, grid, st, what);
+    return gqa_step_launch<32, 0>(mk, mv, p, grid, st, what);
 }

@@ -159,7 +159,7 @@ class ChunkedAttention:
         o = weight("o", width, c.heads * c.vdim)
         self.o = ops.Linear(pad_heads(o.t(), c.heads, c.vdim).t(), dtype, bias=weight("o.b", width))
         self.score_bound = 1.02 * c.dim * abs(c.scale)          # unit-RMS queries and keys, the keys rounded to bf16
-        self.mix = float(weight("vmix").reshape(-1)[0]) if c.mixes_values else 0.0
+        self.mix = float(weight("vmix").reshape(())) if c.mixes_values else 0.0      # one number
 
     def new_state(self, num_seqs: int, max_tokens: Optional[int] = None) -> ChunkCache:
         c = self.cfg

@@ -87,9 +87,9 @@ def prompt_kernels(pk, B=8, S=2048):
                                           dim, dim, 1e-5, keys.data_ptr(), vals.data_ptr(), S, 0, cache.k.data_ptr(), cache.v.data_ptr(),
                                           cache.ring_tokens, chunk, 1, _stream()))
             kept = B * ((S - 1) % chunk + 1)
-            K.hbm(f"kv_prep, {kv} x {dim}, chunk {chunk}", timed(prep), (T * 5 + kept * 2) * kv * dim * 2)
+            K.hbm(f"kv_prep, {kv} x {dim}, chunk {chunk}", timed_graph(prep), (T * 5 + kept * 2) * kv * dim * 2)
             pos = torch.full((B,), chunk - 1, dtype=torch.int32, device="cuda")
-            K.hbm(f"kv_gather, {kv} x {dim}, {chunk - 1} tokens", timed(lambda i: cache.gather(seq, pos, chunk - 1, keys, vals, chunk - 1)),
+            K.hbm(f"kv_gather, {kv} x {dim}, {chunk - 1} tokens", timed_graph(lambda i: cache.gather(seq, pos, chunk - 1, keys, vals, chunk - 1)),
                   B * (chunk - 1) * kv * dim * 8)
             if chunk == 512:
                 K.tensor(f"product q|k|v|gate, {heads} x {dim}", timed(lambda i: m.project(h)), 2.0 * T * m.proj.n * m.proj.k)
@@ -114,12 +114,14 @@ def prompt_kernels(pk, B=8, S=2048):
 def llama_prompt_kernels(pk, B=8, S=2048):
     from baranet_bdml_b200 import ops
     K, bf, T = Kernels(pk), torch.bfloat16, B * S
-    q, k, v = _rnd(B, S, HEADS, DIM), _rnd(B, S, KV_HEADS, DIM), _rnd(B, S, KV_HEADS, DIM)
-    ws = ops.prefill_workspace(B, S, HEADS, KV_HEADS, DIM)
-    out = torch.empty_like(q)
-    ops.attn_prefill_bf16(q, k, v, out=out, workspace=ws)
-    K.tensor("prefill_kernel, causal", timed(lambda i: ops.attn_prefill_bf16(q, None, v, out=out, workspace=ws, reuse_rotated_k=True)),
-             2.0 * B * HEADS * (S * (S + 1) / 2) * 2 * DIM)
+    for b, s in ((B, S), (T // 512, 512)):
+        q, k, v = _rnd(b, s, HEADS, DIM), _rnd(b, s, KV_HEADS, DIM), _rnd(b, s, KV_HEADS, DIM)
+        ws = ops.prefill_workspace(b, s, HEADS, KV_HEADS, DIM)
+        out = torch.empty_like(q)
+        ops.attn_prefill_bf16(q, k, v, out=out, workspace=ws)
+        K.tensor(f"prefill_kernel, causal, {b} x {s}",
+                 timed(lambda i: ops.attn_prefill_bf16(q, None, v, out=out, workspace=ws, reuse_rotated_k=True)),
+                 2.0 * b * HEADS * (s * (s + 1) / 2) * 2 * DIM)
     h, w = _rnd(T, WIDTH), torch.ones(WIDTH, device="cuda", dtype=bf)
     for name, n, kk in (("product 2048 x 2048", 2048, 2048), ("product 5120 x 2048", 5120, 2048), (f"product {FF} x 2048", FF, 2048),
                         (f"product 2048 x {FF}", 2048, FF)):

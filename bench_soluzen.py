@@ -145,7 +145,7 @@ def prompt_kernels(pk, B=8, S=2048, window=1024):
         _lib.check(lib.bn_attn_window(q.data_ptr(), q.stride(0), kv.data_ptr(), kv.data_ptr() + c.heads * c.dim * 2, kv.stride(0),
                                       key.data_ptr(), at.rot_ld, out.data_ptr(), out.stride(0), B, S, 0, S, c.heads, c.dim, c.rot_dim, c.vdim,
                                       window, float(c.scale), ops.status_word("cuda").data_ptr(), 1, st()))
-    K.tensor(f"attn_window_sm100, window {window}", timed(attn), 2.0 * B * c.heads * seen * (c.dim + c.rot_dim + c.vdim))
+    K.tensor(f"attn_portion_sm100, window {window}", timed(attn), 2.0 * B * c.heads * seen * (c.dim + c.rot_dim + c.vdim))
 
     # mamba2
     pin = rnd(T, mb.proj_in.n)

@@ -325,6 +325,38 @@ def test_chunked_attention(lib, dtype, H, G, E, V, S, n_old, chunk):
 
 
 @DTYPES
+@pytest.mark.parametrize("B,H,G,E,V", [(16, 32, 4, 64, 64), (9, 40, 8, 128, 128), (20, 16, 2, 40, 136)])
+@pytest.mark.parametrize("S,n_old,chunk", [(40, 0, 16), (130, 0, 500), (2, 9, 12), (300, 63, 64), (257, 0, 1)])
+def test_many_short_units(lib, dtype, B, H, G, E, V, S, n_old, chunk):
+    """More (sequence, head, query tile) units than the GPU has SMs, each of one or a few key tiles: the persistent kernel goes
+    from unit to unit while the one before is still being put out."""
+    from baranet_bdml_b200 import _lib
+    rng = np.random.default_rng(B + S)
+    n, eps, scale = S + n_old, 1e-5, 4.0 * E ** -0.5
+    q, k = rng.standard_normal((B, S, H, E)), R.unit_rms(rng.standard_normal((B, n, G, E)), eps)
+    qg, kg, vg = _pad(q, dtype), _pad(k, dtype), _pad(rng.standard_normal((B, n, G, V)), dtype)
+    V8, E8 = vg.shape[-1] // G, kg.shape[-1] // G
+    seqs = [0, B // 2, B - 1]
+    heads = [0, H // 2, H - 1]
+    for bound in (0.0, 1.02 * E * scale):
+        out = torch.full((B, S, H * V8), 7.0, dtype=dtype, device="cuda")
+        word = torch.zeros(1, dtype=torch.int32, device="cuda")
+        for _ in range(3):
+            _lib.check(_lib.load().bn_attn_chunked(
+                qg.data_ptr(), H * E8, kg.data_ptr(), G * E8, vg.data_ptr(), G * V8, None, 0, out.data_ptr(), H * V8, B, S, n_old, n, H, G, E8,
+                V8, chunk, E, eps, scale, bound, word.data_ptr(), code(dtype), stream()))
+        torch.cuda.synchronize()
+        assert int(word.item()) == 0
+        Q, K_, V_, got = R.unit_rms(_unpad(qg, H, E), eps), _unpad(kg, G, E), _unpad(vg, G, V), _unpad(out, H, V)
+        for b in seqs:
+            for h in heads:
+                g = h // (H // G)
+                Qb = np.concatenate([np.zeros((n_old, 1, E)), Q[b, :, h:h + 1]])
+                want = R.chunked_attention(Qb, K_[b, :, g:g + 1], V_[b, :, g:g + 1], scale, chunk)[n_old:, 0]
+                assert np.abs(got[b, :, h] - want).max() <= (2e-5 if dtype == torch.float32 else 3e-2), (bound, b, h)
+
+
+@DTYPES
 @pytest.mark.parametrize("chunk,n_old", [(70, 0), (70, 69), (128, 5), (200, 131)])
 def test_keys_just_inside_and_outside_a_chunk(lib, dtype, chunk, n_old):
     """One key that every query of its chunk picks out (its score is 8 standard deviations up): the first and the last of a

@@ -333,6 +333,31 @@ def test_window_attention(lib, dtype, H, dim, rot, vd, S, n_old, window):
     assert np.abs(got - want).max() <= (2e-5 if dtype == torch.float32 else 3e-2)
 
 
+@pytest.mark.parametrize("H,dim,rot,vd", [(20, 128, 64, 128), (32, 40, 16, 72), (16, 128, 64, 192)])
+@pytest.mark.parametrize("S,window", [(70, 30), (130, 500), (300, 64)])
+def test_window_attention_many_short_units(lib, H, dim, rot, vd, S, window):
+    """More (sequence, head, query tile) units than the GPU has SMs, each of a few key tiles."""
+    from baranet_bdml_b200 import _lib
+    rng = np.random.default_rng(S + H)
+    B, scale, bf = 12, 4.0 * (dim + rot) ** -0.5, torch.bfloat16
+    q, kn = gpu(rng.standard_normal((B, S, H, dim + rot)), bf), gpu(rng.standard_normal((B, S, H, dim)), bf)
+    kr, v = gpu(rng.standard_normal((B, S, rot)), bf), gpu(rng.standard_normal((B, S, H, vd)), bf)
+    kv = torch.cat([kn.reshape(B * S, -1), v.reshape(B * S, -1)], dim=1).contiguous()
+    out, word = torch.zeros((B, S, H, vd), dtype=bf, device="cuda"), torch.zeros(1, dtype=torch.int32, device="cuda")
+    for _ in range(3):
+        _lib.check(_lib.load().bn_attn_window(
+            q.data_ptr(), H * (dim + rot), kv.data_ptr(), kv.data_ptr() + H * dim * 2, kv.stride(0), kr.data_ptr(), rot, out.data_ptr(), H * vd,
+            B, S, 0, S, H, dim, rot, vd, window, scale, word.data_ptr(), 1, torch.cuda.current_stream().cuda_stream))
+    torch.cuda.synchronize()
+    assert int(word.item()) == 0
+    up = lambda t: t.double().cpu().numpy()              # noqa: E731
+    for b in (0, B - 1):
+        for h in (0, H - 1):
+            key = np.concatenate([up(kn[b, :, h]), up(kr[b])], axis=1)[:, None]
+            want = R.windowed_softmax_attention(up(q[b, :, h])[:, None], key, up(v[b, :, h])[:, None], scale, window)[:, 0]
+            assert np.abs(up(out[b, :, h]) - want).max() <= 3e-2
+
+
 @pytest.mark.parametrize("S", [64, 300])
 def test_window_attention_growing_scores(lib, S):
     """Scores that rise along the keys by far more than the rescale threshold, and rows whose first key tile they cannot see."""
