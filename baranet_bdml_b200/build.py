@@ -25,8 +25,8 @@ SOURCES = ["api.cu", "tma.cu", "attn_f32.cu", "rmsnorm.cu", "embed_argmax.cu", "
 FAMILIES = {
     "soluzen": ["api.cu", "tma.cu", "mm_f32.cu", "embed_argmax.cu", "gemm_bf16_sm100.cu", "gemm_skinny.cu", "residual_norm.cu",
                 "attn_portion.cu", "attn_portion_sm100.cu", "latent_attn.cu", "latent_decode.cu", "mamba2.cu", "ssd_scan.cu"],
-    "duponex": ["api.cu", "tma.cu", "mm_f32.cu", "embed_argmax.cu", "gemm_bf16_sm100.cu", "gemm_skinny.cu", "residual_norm.cu",
-                "hyper_norm.cu", "attn_portion.cu", "attn_portion_sm100.cu", "gqa_chunk.cu"],
+    "duponex": ["api.cu", "tma.cu", "mm_f32.cu", "embed_argmax.cu", "gemm_bf16_sm100.cu", "gemm_skinny.cu", "hyper_norm.cu",
+                "attn_portion.cu", "attn_portion_sm100.cu", "gqa_chunk.cu"],
 }
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "--expt-relaxed-constexpr", "-Xcompiler", "-fPIC,-fvisibility=hidden",

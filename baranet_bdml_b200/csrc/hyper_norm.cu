@@ -32,7 +32,7 @@ struct HyperParams {
 };
 
 // NV = float4 pieces per thread: hidden <= 1024 * NV, hidden % 4 == 0, every row start 16-byte (bf16: 8-byte) aligned
-template <typename T, typename TD, int NV, int NI, int NO>
+template <typename T, int NV, int NI, int NO>
 __global__ void __launch_bounds__(HY_THREADS)
 hyper_norm_regs_kernel(const __grid_constant__ HyperParams p) {
     __shared__ float sh[HY_THREADS / 32];
@@ -43,7 +43,7 @@ hyper_norm_regs_kernel(const __grid_constant__ HyperParams p) {
     for (int r = blockIdx.x; r < p.rows; r += gridDim.x) {
         float xv[NV][NI][4], d[NV][4];
         const float* xr = p.x + (int64_t)r * NI * p.hidden;
-        const TD* dr = static_cast<const TD*>(p.delta) + (int64_t)r * p.delta_ld;
+        const T* dr = static_cast<const T*>(p.delta) + (int64_t)r * p.delta_ld;
 #pragma unroll
         for (int k = 0; k < NV; ++k) {
             const int c = threadIdx.x + k * HY_THREADS;
@@ -100,7 +100,7 @@ hyper_norm_regs_kernel(const __grid_constant__ HyperParams p) {
 }
 
 // any hidden, any number of streams up to HY_MAX, any strides
-template <typename T, typename TD>
+template <typename T>
 __global__ void __launch_bounds__(HY_THREADS)
 hyper_norm_any_kernel(const __grid_constant__ HyperParams p) {
     extern __shared__ float row_buf[];
@@ -111,7 +111,7 @@ hyper_norm_any_kernel(const __grid_constant__ HyperParams p) {
     ptx::grid_dependency_wait();
     ptx::grid_launch_dependents();
     for (int r = blockIdx.x; r < p.rows; r += gridDim.x) {
-        const TD* dr = p.delta ? static_cast<const TD*>(p.delta) + (int64_t)r * p.delta_ld : nullptr;
+        const T* dr = p.delta ? static_cast<const T*>(p.delta) + (int64_t)r * p.delta_ld : nullptr;
         float ss = 0.f;
         for (int i = threadIdx.x; i < p.hidden; i += HY_THREADS) {
             float d = dr ? to_f(dr[i]) : 0.f;
@@ -135,7 +135,7 @@ hyper_norm_any_kernel(const __grid_constant__ HyperParams p) {
 
 template <int NV, int NI, int NO>
 static void hyper_launch(unsigned grid, cudaStream_t st, const HyperParams& p) {
-    launch_dependent(hyper_norm_regs_kernel<__nv_bfloat16, __nv_bfloat16, NV, NI, NO>, grid, HY_THREADS, 0, st, p);
+    launch_dependent(hyper_norm_regs_kernel<__nv_bfloat16, NV, NI, NO>, grid, HY_THREADS, 0, st, p);
 }
 
 // the stream counts that have a register form; false: none
@@ -162,10 +162,10 @@ static int hyper_any(unsigned grid, cudaStream_t st, const HyperParams& p) {
     const size_t smem = (size_t)p.hidden * sizeof(float);
     if (smem > 200 * 1024) return fail(BN_ERR_UNSUPPORTED, "%s: hidden=%d (at most 51200)", what, p.hidden);
     if (smem > 40 * 1024) {
-        cudaError_t e = cudaFuncSetAttribute(hyper_norm_any_kernel<T, T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaError_t e = cudaFuncSetAttribute(hyper_norm_any_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return fail(BN_ERR_CUDA, "%s: %s", what, cudaGetErrorString(e));
     }
-    launch_dependent(hyper_norm_any_kernel<T, T>, grid, HY_THREADS, smem, st, p);
+    launch_dependent(hyper_norm_any_kernel<T>, grid, HY_THREADS, smem, st, p);
     return launch_status(what);
 }
 

@@ -1,6 +1,7 @@
 // fp32 matrix product in the reference's own arithmetic order: one FMA chain per output, k ascending (reference:
 // src/ops/op_mm_optimized.cuh:35-62).
 #include "common.cuh"
+#include "hybrid.cuh"
 
 namespace bn {
 
@@ -65,6 +66,15 @@ mm_f32_kernel(const float* __restrict__ A, int64_t a_rs, int64_t a_cs, const flo
     }
 }
 
+// x = act(x + bias) in place, fp32 rows (the unfused form of the products with a bias or an activation)
+__global__ void __launch_bounds__(256)
+bias_act_kernel(float* x, int64_t ld, const float* bias, long long n, int cols, int act) {
+    for (long long i = (long long)blockIdx.x * 256 + threadIdx.x; i < n; i += (long long)gridDim.x * 256) {
+        const int64_t r = i / cols, c = i - r * cols;
+        x[r * ld + c] = activation_exact(act, x[r * ld + c] + (bias ? bias[c] : 0.f));
+    }
+}
+
 }  // namespace bn
 
 using namespace bn;
@@ -79,4 +89,15 @@ extern "C" int bn_mm_f32(const float* A, int64_t a_rs, int64_t a_cs, const float
     if (grid.y > 65535) return fail(BN_ERR_UNSUPPORTED, "bn_mm_f32: M=%d too large", M);
     mm_f32_kernel<<<grid, 256, 0, as_stream(stream)>>>(A, a_rs, a_cs, B, b_rs, b_cs, C, c_rs, c_cs, M, K, N);
     return launch_status("bn_mm_f32");
+}
+
+extern "C" int bn_bias_act_f32(float* x, int64_t ld, const float* bias, int rows, int cols, int act, bn_stream_t stream) {
+    if (!x) return fail(BN_ERR_INVALID_ARG, "bn_bias_act_f32: null pointer");
+    if (rows < 0 || cols < 0 || act < 0 || act > BN_ACT_LAST) return fail(BN_ERR_INVALID_ARG, "bn_bias_act_f32: bad shape or activation");
+    if (int rc = require_sm100()) return rc;
+    const long long n = (long long)rows * cols;
+    if (n == 0) return BN_OK;
+    const long long blocks = (n + 255) / 256;
+    bias_act_kernel<<<(unsigned)(blocks < 4096 ? blocks : 4096), 256, 0, as_stream(stream)>>>(x, ld, bias, n, cols, act);
+    return launch_status("bn_bias_act_f32");
 }

@@ -229,15 +229,6 @@ act_mul_kernel(const float* a, int64_t a_ld, const float* b, int64_t b_ld, float
     }
 }
 
-// x = act(x + bias) in place, fp32 rows (the unfused form of the products with a bias or an activation)
-__global__ void __launch_bounds__(256)
-bias_act_kernel(float* x, int64_t ld, const float* bias, long long n, int cols, int act) {
-    for (long long i = (long long)blockIdx.x * 256 + threadIdx.x; i < n; i += (long long)gridDim.x * 256) {
-        const int64_t r = i / cols, c = i - r * cols;
-        x[r * ld + c] = activation_exact(act, x[r * ld + c] + (bias ? bias[c] : 0.f));
-    }
-}
-
 }  // namespace bn
 
 using namespace bn;
@@ -272,15 +263,4 @@ extern "C" int bn_act_mul_f32(const float* a, int64_t a_ld, const float* b, int6
     act_mul_kernel<<<(unsigned)(blocks < 4096 ? blocks : 4096), 256, 0, as_stream(stream)>>>(a, a_ld, b, b_ld, out, out_ld, n,
                                                                                        cols, act);
     return launch_status("bn_act_mul_f32");
-}
-
-extern "C" int bn_bias_act_f32(float* x, int64_t ld, const float* bias, int rows, int cols, int act, bn_stream_t stream) {
-    if (!x) return fail(BN_ERR_INVALID_ARG, "bn_bias_act_f32: null pointer");
-    if (rows < 0 || cols < 0 || act < 0 || act > BN_ACT_LAST) return fail(BN_ERR_INVALID_ARG, "bn_bias_act_f32: bad shape or activation");
-    if (int rc = require_sm100()) return rc;
-    const long long n = (long long)rows * cols;
-    if (n == 0) return BN_OK;
-    const long long blocks = (n + 255) / 256;
-    bias_act_kernel<<<(unsigned)(blocks < 4096 ? blocks : 4096), 256, 0, as_stream(stream)>>>(x, ld, bias, n, cols, act);
-    return launch_status("bn_bias_act_f32");
 }
